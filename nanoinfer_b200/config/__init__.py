@@ -4,6 +4,7 @@ from .vadonex import VadonexConfig
 from .kemuzen import KemuzenConfig
 from .mulavik import MulavikConfig
 from .nagilix import NagilixConfig
+from .dedunex import DedunexConfig
 
 __all__ = ["ConfigError", "ModelConfig", "field", "read_config_json", "architecture_name", "GPT2Config", "VadonexConfig",
-           "MulavikConfig", "KemuzenConfig", "NagilixConfig"]
+           "MulavikConfig", "KemuzenConfig", "NagilixConfig", "DedunexConfig"]

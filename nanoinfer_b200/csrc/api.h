@@ -24,7 +24,9 @@
 //                 the sequence);
 //   head_scale:   one number per query head that multiplies the scale (a temperature);
 //   sinks:        with `sink` set, one number per query head: the denominator's extra term is exp(sinks[h]) instead
-//                 of exp(0).
+//                 of exp(0);
+//   out32:        `out` holds 32-bit floats whatever the dtype of queries and cache (what follows the attention
+//                 subtracts or norms its results before they are rounded).
 struct AttnExtras {
   float softcap;
   int keep_first;
@@ -35,6 +37,7 @@ struct AttnExtras {
   int span;
   const float* head_scale;
   const float* sinks;
+  int out32;
 };
 
 #ifdef __cplusplus
@@ -111,7 +114,7 @@ int nib_attention_simt(int dtype, const void* q, int ldq, const void* cache, voi
                        const int* block_table, int max_blocks, const int* rows, const int* row_entry,
                        const int* positions, int T, int n_head, int n_kv_head, int head_dim,
                        int page_size, int n_pages, float scale, int window, int sink, float softcap,
-                       int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int* status,
+                       int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
                        cudaStream_t stream);
 
 // tcgen05 attention for prompt portions (bfloat16, head size 64, page size a multiple of 16): tiles of
@@ -122,7 +125,7 @@ int nib_attention_prefill_tc(const void* q, int ldq, int T, const void* cache, v
                              const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                              const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head, int head_dim,
                              int page_size, int n_pages, float scale, int window, int sink, float softcap, int keep_first,
-                             const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int* status,
+                             const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
                              cudaStream_t stream);
 
 // Split-KV attention for single decoded tokens (float32 or bfloat16, head sizes up to 128 in steps
@@ -132,7 +135,7 @@ int nib_attention_decode(int dtype, const void* q, int ldq, const void* cache, f
                          int ldo, const int* block_table, int max_blocks, const int* rows,
                          const int* row_entry, const int* positions, int n_rows, int n_head, int n_kv_head,
                          int head_dim, int page_size, int n_pages, float scale, int window, int sink, float softcap,
-                         int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int chunk,
+                         int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int chunk,
                          int n_splits, int* counters, int* status, cudaStream_t stream);
 
 // Tiled tensor-core attention for prompt portions (bfloat16, head sizes 16..128 in steps of 16), with the options of
@@ -142,7 +145,7 @@ int nib_attention_prefill(const void* q, int ldq, const void* cache, void* out, 
                           const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                           const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head,
                           int head_dim, int page_size, int n_pages, float scale, int window, int sink, float softcap,
-                          int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int* status,
+                          int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
                           cudaStream_t stream);
 
 // Loading: src holds [rows, cols] values as a checkpoint stores them (src_dtype 0: 32-bit floats, 1:
@@ -201,19 +204,20 @@ int nib_mlstm(int dtype, const float* proj, int ld, int q_off, int k_off, int v_
               const int* entry_start, const int* entry_slot, int n_entries, int n_rows, int n_head, int dim, int vdim,
               float eps, float* gates, float* num, int ld_num, float* den, void* out, int ldo, cudaStream_t stream);
 
-// ---- attention through a shared low-rank latent (latent_attention.cu)
+// ---- attention through a shared low-rank latent (latent_attention.cu); halves: the layout of the rotation (0: pairs
+// (2i, 2i + 1), 1: i with i + rot_dims / 2); gate (may be null): head h's output times sigmoid(gate[t * ldg + h])
 int nib_latent_prep(int dtype, const float* proj, int ld, int q_rank, int kv_rank, int rot_dim, int rot_dims,
                     const double* freqs, const float* wq, const float* wkv, float eps, void* cq, int ld_cq,
                     void* cache, const int* block_table, int max_blocks, const int* row_entry,
-                    const int* positions, int T, int page_size, int n_pages, int has_kv, int* status,
+                    const int* positions, int T, int page_size, int n_pages, int has_kv, int halves, int* status,
                     cudaStream_t stream);
 int nib_rope_heads(int dtype, const void* q, int ldq, int nope, int rot_dim, int rot_dims, const double* freqs,
-                   const int* positions, float* out, int out_dim, int out_off, int n_head, int T,
+                   const int* positions, float* out, int out_dim, int out_off, int n_head, int T, int halves,
                    cudaStream_t stream);
 int nib_latent_attention(int dtype, const float* q, const void* cache, void* out, int ldo, const int* block_table,
                          int max_blocks, const int* rows, const int* row_entry, const int* positions, int n_rows,
                          int n_head, int kv_rank, int D, int page_size, int n_pages, float scale, int window,
-                         int* status, int n_splits, float* partials, cudaStream_t stream);
+                         const float* gate, int ldg, int* status, int n_splits, float* partials, cudaStream_t stream);
 
 // ---- a product per head (linear_heads.cu): out[t, h, :N] = a[t, h, :K] . w[h]^T, w [n_head, N, K]
 int nib_linear_heads(int dtype, int out_dtype, const void* a, int lda, int a_head_stride, const void* w, void* out,
@@ -309,6 +313,36 @@ int nib_selective_scan(int out_dtype, const float* dtp, int ld_dt, const float* 
                        int b_off, int c_off, const float* z, int ldz, const float* A_log, const float* D, float* state,
                        long long state_stride, long long s_off, const int* entry_start, const int* entry_slot,
                        int n_entries, int inner, int N, void* out, int ldo, cudaStream_t stream);
+
+// ---- norms in groups (group_norm.cu): every row is cut into `groups` equal consecutive parts, each divided by its own
+// root mean square (eps inside the root), and the whole multiplied by w.
+// out[r] = norm(x[rows[r]] (+ add)); with `add` (one vector of C floats) the sum is also written back to x (rows null
+// then).  out may be null: the sum only.
+int nib_group_norm(int out_dtype, float* x, const int* rows, const float* add, const float* w, void* out, int n_rows,
+                   int C, int groups, float eps, cudaStream_t stream);
+// x[t] = norm(table[token_t] * scale) in 32-bit (tokens as in nib_embed).
+int nib_embed_group_norm(int dtype, const int* tokens, const int* feedback, const void* table, float scale,
+                         const float* w, float* x, int T, int C, int groups, float eps, cudaStream_t stream);
+
+// ---- differential attention (differential.cu, rope.cu)
+// Queries [n_head][maps][dim] and keys [n_kv_head][maps][dim] of the 32-bit projection, every (head, map) divided by
+// its root mean square and times a shared weight (null: no norm), the first rot_dims values turned in the halves layout
+// with cosine and sine times `amp`; keys go to plane 0 of the row's cache slot, the maps of a head side by side, values
+// [n_kv_head][vdim] to plane 1; a query of map m goes to head (h * maps + m) of q_out at the place where the cache
+// holds that map's key, zeros elsewhere in its hd values.
+int nib_norm_rope_maps_append(int dtype, const float* proj, int ld, int q_off, int k_off, int v_off, int n_head,
+                              int n_kv_head, int maps, int dim, int vdim, int hd, const float* wq, const float* wk,
+                              float eps, int rot_dims, const double* freqs, float amp, const int* positions,
+                              const int* row_entry, void* q_out, int ldq, void* cache, const int* block_table,
+                              int max_blocks, int page_size, int n_pages, int T, int* status, cudaStream_t stream);
+// out[t, h, :vdim] = mul * o / sqrt(mean(o^2) + eps) with o = a[t, 2h] - lambda * a[t, 2h + 1], a 32-bit heads of hd.
+int nib_diff_combine(int out_dtype, const float* a, int lda, int n_head, int hd, int vdim, float lambda, float eps,
+                     float mul, void* out, int ldo, int T, cudaStream_t stream);
+
+// ---- the minimal gated recurrent unit (min_gru.cu): z, u and g logits at three column offsets of the 32-bit proj.
+int nib_min_gru(int out_dtype, const float* proj, int ld, int z_off, int u_off, int g_off, int width, float* state,
+                long long state_stride, const int* entry_start, const int* entry_slot, int n_entries, int n_rows,
+                void* out, int ldo, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -257,9 +257,11 @@ attention_decode_kernel(const T* q, int ldq, const T* cache, float* part_o,
   for (int d = threadIdx.x; d < head_dim; d += blockDim.x) {
     float acc = 0.0f;
     for (int w = 0; w < ALL_GROUPS; ++w) acc += (gm[w] == -INFINITY) ? 0.0f : go[w * head_dim + d] * pow2<T>(gm[w] - M);
-    if (n_splits == 1)
-      out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(acc / L1 * mul1);
-    else if (cluster_merge)
+    if (n_splits == 1) {
+      const float y = acc / L1 * mul1;
+      if (ex.out32) reinterpret_cast<float*>(out)[(size_t)t * ldo + h * head_dim + d] = y;
+      else out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(y);
+    } else if (cluster_merge)
       store_to_rank(xo + split * head_dim + d, 0, acc);
     else
       part_o[pidx * head_dim + d] = acc;
@@ -312,7 +314,9 @@ attention_decode_kernel(const T* q, int ldq, const T* cache, float* part_o,
       const float ls = part_ml[2 * (base + sp) + 1];
       if (ls > 0.0f) acc += part_o[(base + sp) * head_dim + d] * pow2<T>(part_ml[2 * (base + sp)] - Mx);
     }
-    out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(acc / Lx * mulx);
+    const float y = acc / Lx * mulx;
+    if (ex.out32) reinterpret_cast<float*>(out)[(size_t)t * ldo + h * head_dim + d] = y;
+    else out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(y);
   }
 }
 
@@ -361,10 +365,10 @@ extern "C" int nib_attention_decode(int dtype, const void* q, int ldq, const voi
                                     const int* row_entry, const int* positions, int n_rows, int n_head,
                                     int n_kv_head, int head_dim, int page_size, int n_pages, float scale,
                                     int window, int sink, float softcap, int keep_first, const float* slopes,
-                                    const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int chunk, int n_splits,
+                                    const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int chunk, int n_splits,
                                     int* counters, int* status, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks};
+  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32};
   if (head_dim <= 0 || head_dim > DEC_MAX_HD || (head_dim & 7)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (page_size % 16 != 0 || chunk <= 0 || chunk % 16 != 0 || n_splits <= 0) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_kv_head <= 0 || n_head % n_kv_head != 0) return NIB_ERR_BAD_ARGUMENT;
@@ -440,5 +444,5 @@ extern "C" int nib_attention_decode_static(int dtype, const void* q, int ldq, co
   if (e != cudaSuccess) return (int)e;
   return nib_attention_decode(dtype, q, ldq, cache, scratch, out, ldo, block_table, max_blocks, rows, row_entry,
                               positions, n_rows, n_head, n_kv_head, head_dim, page_size, n_pages, scale, window,
-                              0, 0.0f, 0, nullptr, nullptr, 0, 1.0f, 0, nullptr, nullptr, chunk, n_splits, counters, status, stream);
+                              0, 0.0f, 0, nullptr, nullptr, 0, 1.0f, 0, nullptr, nullptr, 0, chunk, n_splits, counters, status, stream);
 }

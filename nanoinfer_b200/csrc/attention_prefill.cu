@@ -314,6 +314,12 @@ attention_prefill_kernel(const bf16* q, int ldq, const bf16* cache, bf16* out,
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) {
     const int d = h * HD + i * 8 + (lane & 3) * 2;
+    if (EX && ex.out32) {
+      float* o32 = reinterpret_cast<float*>(out);
+      if (r0 < n_rows) *reinterpret_cast<float2*>(o32 + (size_t)(row0 + r0) * ldo + d) = make_float2(o[i][0] * i0, o[i][1] * i0);
+      if (r1 < n_rows) *reinterpret_cast<float2*>(o32 + (size_t)(row0 + r1) * ldo + d) = make_float2(o[i][2] * i1, o[i][3] * i1);
+      continue;
+    }
     if (r0 < n_rows)
       *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + r0) * ldo + d) = pack2(o[i][0] * i0, o[i][1] * i0);
     if (r1 < n_rows)
@@ -357,16 +363,16 @@ extern "C" int nib_attention_prefill(const void* q, int ldq, const void* cache, 
                                      const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head,
                                      int head_dim, int page_size, int n_pages, float scale, int window,
                                      int sink, float softcap, int keep_first, const float* slopes,
-                                     const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int* status, cudaStream_t stream) {
+                                     const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
-  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks};
+  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32};
   const bool plain = !(softcap > 0.0f) && (keep_first <= 0 || window <= 0) && !slopes && !gate && out_scale == 1.0f &&
-                     span <= 0 && !head_scale && !sinks;
+                     span <= 0 && !head_scale && !sinks && !out32;
   if (span < 0) return NIB_ERR_BAD_ARGUMENT;
   if (softcap < 0.0f || keep_first < 0) return NIB_ERR_BAD_ARGUMENT;
   if (!nib_attention_prefill_supported(head_dim)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_kv_head <= 0 || n_head % n_kv_head != 0 || !(scale > 0.0f)) return NIB_ERR_BAD_ARGUMENT;
-  if ((ldq & 7) || ((uintptr_t)q & 15) || (ldo & 1) || ((uintptr_t)out & 3)) return NIB_ERR_UNSUPPORTED_SIZE;
+  if ((ldq & 7) || ((uintptr_t)q & 15) || (ldo & 1) || ((uintptr_t)out & (out32 ? 7 : 3))) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_tiles > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
 #define NIB_PF_CASE(D)                                                                                         \
   case D:                                                                                                      \

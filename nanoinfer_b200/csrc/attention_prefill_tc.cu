@@ -377,7 +377,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       for (int c = 0; c < AT_HD / 32; ++c) {
         float t[32];
         tmem_ld32(lane_addr + O_COL + (uint32_t)(c * 32), t);
-        if (r < n_rows) {
+        if (EX && prm.ex.out32) {
+          float* dst32 = reinterpret_cast<float*>(prm.out) + (size_t)(row0 + r) * prm.ldo + h * AT_HD;
+          if (r < n_rows) {
+#pragma unroll
+            for (int g = 0; g < 8; ++g)
+              *reinterpret_cast<float4*>(dst32 + c * 32 + 4 * g) =
+                  make_float4(t[4 * g] * inv, t[4 * g + 1] * inv, t[4 * g + 2] * inv, t[4 * g + 3] * inv);
+          }
+        } else if (r < n_rows) {
 #pragma unroll
           for (int g = 0; g < 4; ++g)
             *reinterpret_cast<uint4*>(dst + c * 32 + 8 * g) = make_uint4(
@@ -413,11 +421,11 @@ extern "C" int nib_attention_prefill_tc(const void* q, int ldq, int T, const voi
                                         const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head,
                                         int head_dim, int page_size, int n_pages, float scale, int window,
                                         int sink, float softcap, int keep_first, const float* slopes, const float* gate,
-                                        int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int* status, cudaStream_t stream) {
+                                        int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (softcap < 0.0f || keep_first < 0) return NIB_ERR_BAD_ARGUMENT;
   const bool plain = !(softcap > 0.0f) && (keep_first <= 0 || window <= 0) && !slopes && !gate && out_scale == 1.0f &&
-                     span <= 0 && !head_scale && !sinks;
+                     span <= 0 && !head_scale && !sinks && !out32;
   if (span < 0) return NIB_ERR_BAD_ARGUMENT;
   if (!nib_attention_prefill_tc_supported(head_dim, page_size)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_kv_head <= 0 || n_head % n_kv_head != 0 || !(scale > 0.0f) || T <= 0) return NIB_ERR_BAD_ARGUMENT;
@@ -434,7 +442,7 @@ extern "C" int nib_attention_prefill_tc(const void* q, int ldq, int T, const voi
   prm.entry_start = entry_start; prm.entry_pos0 = entry_pos0;
   prm.n_head = n_head; prm.n_kv_head = n_kv_head; prm.page_size = page_size; prm.n_pages = n_pages;
   prm.scale = scale; prm.window = window; prm.sink = sink; prm.out = (bf16*)out; prm.ldo = ldo; prm.status = status;
-  prm.ex = AttnExtras{softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks};
+  prm.ex = AttnExtras{softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32};
   // 128 keys a tile, one block an SM: measured a little faster than 64 keys a tile and two blocks
   constexpr int BN = 128;
   static bool attr_set = false;

@@ -111,7 +111,9 @@ attention_simt_kernel(const T* q, int ldq, const T* cache,
 #pragma unroll
   for (int i = 0; i < ATT_MAX_ND; ++i) {
     const int d = lane + 32 * i;
-    if (d < head_dim) out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(o[i] * inv);
+    if (d >= head_dim) continue;
+    if (ex.out32) reinterpret_cast<float*>(out)[(size_t)t * ldo + h * head_dim + d] = o[i] * inv;
+    else out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(o[i] * inv);
   }
 }
 
@@ -124,10 +126,10 @@ extern "C" int nib_attention_simt(int dtype, const void* q, int ldq, const void*
                                   const int* row_entry, const int* positions, int T, int n_head,
                                   int n_kv_head, int head_dim, int page_size, int n_pages,
                                   float scale, int window, int sink, float softcap, int keep_first,
-                                  const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int* status,
+                                  const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
                                   cudaStream_t stream) {
   if (T <= 0) return 0;
-  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks};
+  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32};
   if (head_dim <= 0 || head_dim > 32 * ATT_MAX_ND || (head_dim & 1)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_kv_head <= 0 || n_head % n_kv_head != 0) return NIB_ERR_BAD_ARGUMENT;
   if (T > 65535) return NIB_ERR_UNSUPPORTED_SIZE;

@@ -14,9 +14,10 @@
 //   rope_heads       : rotates the rot part of every head's query and writes it behind the absorbed part
 //   latent_attention : softmax attention of rows over the cache, causal, with an optional window
 //                      (position i sees j with 0 <= i - j < window)
-// Rotation: pairs (2i, 2i+1) of the first rot_dims values, angle = position * freq[i]; the angle and its
-// sine and cosine are computed in double precision from a table of frequencies made on the host, the
-// rest in 32-bit.  Scores, softmax and the weighted sums are 32-bit.
+// Rotation: pairs (2i, 2i+1) of the first rot_dims values or, with `halves`, value i with value i + rot_dims / 2;
+// angle = position * freq[i]; the angle and its sine and cosine are computed in double precision from a table of frequencies made on the host, the
+// rest in 32-bit.  An output gate per head (optional, logits in 32-bit): the head's output times sigmoid(gate[t, h]),
+// applied to the weighted sum of latents, which the map to the head's values leaves linear.  Scores, softmax and the weighted sums are 32-bit.
 #include "api.h"
 #include "common.cuh"
 
@@ -28,7 +29,7 @@ latent_prep_kernel(const float* proj, int ld, int q_rank, int kv_rank, int rot_d
                    const double* __restrict__ freqs, const float* __restrict__ wq, const float* __restrict__ wkv,
                    float eps, T* cq, int ld_cq, T* cache, const int* __restrict__ block_table, int max_blocks,
                    const int* __restrict__ row_entry, const int* __restrict__ positions, int page_size,
-                   int n_pages, int has_kv, int* status) {
+                   int n_pages, int has_kv, int halves, int* status) {
   pdl_trigger();
   __shared__ float scratch[32];
   const int t = blockIdx.x;
@@ -56,9 +57,10 @@ latent_prep_kernel(const float* proj, int ld, int q_rank, int kv_rank, int rot_d
   for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
     double sn, cs;
     sincos((double)pos * freqs[i], &sn, &cs);
-    const float u = kr[2 * i], v = kr[2 * i + 1], c = (float)cs, sf = (float)sn;
-    dst[kv_rank + 2 * i] = from_float<T>(u * c - v * sf);
-    dst[kv_rank + 2 * i + 1] = from_float<T>(v * c + u * sf);
+    const int iu = halves ? i : 2 * i, iv = halves ? i + rot_dims / 2 : 2 * i + 1;
+    const float u = kr[iu], v = kr[iv], c = (float)cs, sf = (float)sn;
+    dst[kv_rank + iu] = from_float<T>(u * c - v * sf);
+    dst[kv_rank + iv] = from_float<T>(v * c + u * sf);
   }
   for (int c = rot_dims + threadIdx.x; c < rot_dim; c += blockDim.x) dst[kv_rank + c] = from_float<T>(kr[c]);
 }
@@ -68,7 +70,7 @@ latent_prep_kernel(const float* proj, int ld, int q_rank, int kv_rank, int rot_d
 template <typename T>
 __global__ void __launch_bounds__(128)
 rope_heads_kernel(const T* q, int ldq, int nope, int rot_dim, int rot_dims, const double* __restrict__ freqs,
-                  const int* __restrict__ positions, float* out, int out_dim, int out_off, int n_head) {
+                  const int* __restrict__ positions, float* out, int out_dim, int out_off, int n_head, int halves) {
   pdl_trigger();
   extern __shared__ float cs[];   // cos, sin per pair
   const int t = blockIdx.x, half = rot_dims / 2;
@@ -87,9 +89,10 @@ rope_heads_kernel(const T* q, int ldq, int nope, int rot_dim, int rot_dims, cons
     const T* src = q + (size_t)t * ldq + (size_t)h * (nope + rot_dim) + nope;
     float* dst = out + ((size_t)t * n_head + h) * out_dim + out_off;
     if (i < half) {
-      const float u = to_float(src[2 * i]), v = to_float(src[2 * i + 1]), c = cs[2 * i], s = cs[2 * i + 1];
-      dst[2 * i] = u * c - v * s;
-      dst[2 * i + 1] = v * c + u * s;
+      const int iu = halves ? i : 2 * i, iv = halves ? i + half : 2 * i + 1;
+      const float u = to_float(src[iu]), v = to_float(src[iv]), c = cs[2 * i], s = cs[2 * i + 1];
+      dst[iu] = u * c - v * s;
+      dst[iv] = v * c + u * s;
     } else {
       const int d = rot_dims + (i - half);
       dst[d] = to_float(src[d]);
@@ -109,7 +112,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32)
 latent_attention_kernel(const float* q, const T* cache, T* out, int ldo, const int* __restrict__ block_table,
                         int max_blocks, const int* __restrict__ rows, const int* __restrict__ row_entry,
                         const int* __restrict__ positions, int n_head, int kv_rank, int D, int page_size,
-                        int n_pages, float scale, int window, int* status, int n_splits, float* partials) {
+                        int n_pages, float scale, int window, const float* gate, int ldg, int* status, int n_splits, float* partials) {
   pdl_trigger();
   extern __shared__ float smem[];
   const int Dp = D | 1;
@@ -206,7 +209,8 @@ latent_attention_kernel(const float* q, const T* cache, T* out, int ldo, const i
       if (d < kv_rank) dst[2 + d] = acc[k];
     }
   } else if (live) {
-    const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
     T* o = out + (size_t)t * ldo + (size_t)h * kv_rank;
 #pragma unroll
     for (int k = 0; k < NACC; ++k) {
@@ -221,7 +225,7 @@ latent_attention_kernel(const float* q, const T* cache, T* out, int ldo, const i
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* partials, T* out, int ldo, const int* __restrict__ rows,
-                    const int* __restrict__ row_entry, int n_head, int kv_rank, int n_splits) {
+                    const int* __restrict__ row_entry, int n_head, int kv_rank, const float* gate, int ldg, int n_splits) {
   pdl_trigger();
   const int t = rows ? rows[blockIdx.x] : blockIdx.x, h = blockIdx.y;
   if (row_entry[t] < 0) return;
@@ -234,7 +238,8 @@ latent_merge_kernel(const float* partials, T* out, int ldo, const int* __restric
     const float ms = src[(size_t)s * (kv_rank + 2)];
     if (ms != -INFINITY) l += src[(size_t)s * (kv_rank + 2) + 1] * expf(ms - m);
   }
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
   for (int d = threadIdx.x; d < kv_rank; d += blockDim.x) {
     float a = 0.0f;
     for (int s = 0; s < n_splits; ++s) {
@@ -249,18 +254,18 @@ template <typename T, int NACC>
 static int launch_latent_attention(const float* q, const T* cache, T* out, int ldo, const int* block_table,
                                    int max_blocks, const int* rows, const int* row_entry, const int* positions,
                                    int n_rows, int n_head, int kv_rank, int D, int page_size, int n_pages,
-                                   float scale, int window, int* status, int n_splits, float* partials,
-                                   cudaStream_t stream) {
+                                   float scale, int window, const float* gate, int ldg, int* status, int n_splits,
+                                   float* partials, cudaStream_t stream) {
   const size_t smem = ((size_t)LA_TILE * (D | 1) + (size_t)LA_WARPS * D) * sizeof(float);
   if (smem > 200 * 1024) return NIB_ERR_UNSUPPORTED_SIZE;
   if (smem > 48 * 1024)
     cudaFuncSetAttribute(latent_attention_kernel<T, NACC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   launch_pdl(latent_attention_kernel<T, NACC>, dim3(n_rows, (n_head + LA_WARPS - 1) / LA_WARPS, n_splits),
              dim3(LA_WARPS * 32), smem, stream, q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-             n_head, kv_rank, D, page_size, n_pages, scale, window, status, n_splits, partials);
+             n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status, n_splits, partials);
   if (n_splits > 1)
     launch_pdl(latent_merge_kernel<T>, dim3(n_rows, n_head), dim3(128), 0, stream, (const float*)partials, out, ldo,
-               rows, row_entry, n_head, kv_rank, n_splits);
+               rows, row_entry, n_head, kv_rank, gate, ldg, n_splits);
   NIB_LAUNCH_CHECK();
 }
 
@@ -268,12 +273,12 @@ template <typename T>
 static int pick_latent_attention(const float* q, const void* cache, void* out, int ldo, const int* block_table,
                                  int max_blocks, const int* rows, const int* row_entry, const int* positions,
                                  int n_rows, int n_head, int kv_rank, int D, int page_size, int n_pages,
-                                 float scale, int window, int* status, int n_splits, float* partials,
-                                 cudaStream_t stream) {
+                                 float scale, int window, const float* gate, int ldg, int* status, int n_splits,
+                                 float* partials, cudaStream_t stream) {
 #define NIB_LA(N)                                                                                              \
   return launch_latent_attention<T, N>(q, (const T*)cache, (T*)out, ldo, block_table, max_blocks, rows,       \
                                        row_entry, positions, n_rows, n_head, kv_rank, D, page_size, n_pages,  \
-                                       scale, window, status, n_splits, partials, stream)
+                                       scale, window, gate, ldg, status, n_splits, partials, stream)
   const int n = (kv_rank + 31) / 32;
   if (n <= 2) NIB_LA(2);
   if (n <= 4) NIB_LA(4);
@@ -292,18 +297,18 @@ extern "C" int nib_latent_prep(int dtype, const float* proj, int ld, int q_rank,
                                int rot_dims, const double* freqs, const float* wq, const float* wkv, float eps,
                                void* cq, int ld_cq, void* cache, const int* block_table, int max_blocks,
                                const int* row_entry, const int* positions, int T, int page_size, int n_pages,
-                               int has_kv, int* status, cudaStream_t stream) {
+                               int has_kv, int halves, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (q_rank <= 0 || (has_kv && (kv_rank <= 0 || rot_dim < 0 || rot_dims > rot_dim || (rot_dims & 1))))
     return NIB_ERR_BAD_ARGUMENT;
   if (dtype == DT_F32)
     launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(128), 0, stream, proj, ld, q_rank, kv_rank, rot_dim, rot_dims,
                freqs, wq, wkv, eps, (float*)cq, ld_cq, (float*)cache, block_table, max_blocks, row_entry, positions,
-               page_size, n_pages, has_kv, status);
+               page_size, n_pages, has_kv, halves, status);
   else if (dtype == DT_BF16)
     launch_pdl(latent_prep_kernel<bf16>, dim3(T), dim3(128), 0, stream, proj, ld, q_rank, kv_rank, rot_dim, rot_dims,
                freqs, wq, wkv, eps, (bf16*)cq, ld_cq, (bf16*)cache, block_table, max_blocks, row_entry, positions,
-               page_size, n_pages, has_kv, status);
+               page_size, n_pages, has_kv, halves, status);
   else
     return NIB_ERR_BAD_ARGUMENT;
   NIB_LAUNCH_CHECK();
@@ -311,16 +316,16 @@ extern "C" int nib_latent_prep(int dtype, const float* proj, int ld, int q_rank,
 
 extern "C" int nib_rope_heads(int dtype, const void* q, int ldq, int nope, int rot_dim, int rot_dims,
                               const double* freqs, const int* positions, float* out, int out_dim, int out_off,
-                              int n_head, int T, cudaStream_t stream) {
+                              int n_head, int T, int halves, cudaStream_t stream) {
   if (T <= 0 || rot_dim <= 0) return 0;
   if (rot_dims > rot_dim || (rot_dims & 1)) return NIB_ERR_BAD_ARGUMENT;
   const size_t smem = (size_t)(rot_dims + 2) * sizeof(float);
   if (dtype == DT_F32)
     launch_pdl(rope_heads_kernel<float>, dim3(T), dim3(128), smem, stream, (const float*)q, ldq, nope, rot_dim,
-               rot_dims, freqs, positions, out, out_dim, out_off, n_head);
+               rot_dims, freqs, positions, out, out_dim, out_off, n_head, halves);
   else if (dtype == DT_BF16)
     launch_pdl(rope_heads_kernel<bf16>, dim3(T), dim3(128), smem, stream, (const bf16*)q, ldq, nope, rot_dim,
-               rot_dims, freqs, positions, out, out_dim, out_off, n_head);
+               rot_dims, freqs, positions, out, out_dim, out_off, n_head, halves);
   else
     return NIB_ERR_BAD_ARGUMENT;
   NIB_LAUNCH_CHECK();
@@ -333,18 +338,18 @@ extern "C" int nib_rope_heads(int dtype, const void* q, int ldq, int nope, int r
 extern "C" int nib_latent_attention(int dtype, const float* q, const void* cache, void* out, int ldo,
                                     const int* block_table, int max_blocks, const int* rows, const int* row_entry,
                                     const int* positions, int n_rows, int n_head, int kv_rank, int D,
-                                    int page_size, int n_pages, float scale, int window, int* status, int n_splits,
-                                    float* partials, cudaStream_t stream) {
+                                    int page_size, int n_pages, float scale, int window, const float* gate, int ldg,
+                                    int* status, int n_splits, float* partials, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (kv_rank <= 0 || D < kv_rank || n_head <= 0) return NIB_ERR_BAD_ARGUMENT;
   if (n_splits < 1 || n_splits > 65535 || (n_splits > 1 && partials == nullptr)) return NIB_ERR_BAD_ARGUMENT;
   if (dtype == DT_F32)
     return pick_latent_attention<float>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-                                        n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, status,
+                                        n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status,
                                         n_splits, partials, stream);
   if (dtype == DT_BF16)
     return pick_latent_attention<bf16>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-                                       n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, status,
+                                       n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status,
                                        n_splits, partials, stream);
   return NIB_ERR_BAD_ARGUMENT;
 }

@@ -378,3 +378,128 @@ extern "C" int nib_rope_halves(float* rows, int ld, int q_off, int k_off, int n_
              positions, k_mul, decay, coef);
   NIB_LAUNCH_CHECK();
 }
+
+// ---------------------------------------------------------------------------------------------------------------
+// Heads with several maps (differential attention): a query head has `maps` queries of `dim` values and a key head as
+// many keys, each normed and turned by itself; the cache holds a head's keys side by side in one row of hd values.  A
+// query of map m is written as a head of its own with zeros everywhere but at its map's place in that row, so that
+// the attention kernels, which know one key a head, make the score of map m from the whole row.
+namespace nib {
+
+// A warp owns one (head, map) of q or k, or one value head: sum of squares, weight, rotation in the halves layout (a
+// value meets its partner through the warp's piece of shared memory), cast, padding, and the cache write.
+template <typename T>
+__global__ void __launch_bounds__(256)
+norm_rope_maps_append_kernel(const float* proj, int ld, int q_off, int k_off, int v_off, int n_head, int n_kv_head,
+                             int maps, int dim, int vdim, int hd, const float* __restrict__ wq,
+                             const float* __restrict__ wk, float eps, int rot_dims, const double* __restrict__ freqs,
+                             float amp, const int* __restrict__ positions, const int* __restrict__ row_entry, T* q_out,
+                             int ldq, T* cache, const int* __restrict__ block_table, int max_blocks, int page_size,
+                             int n_pages, int* status) {
+  pdl_trigger();
+  __shared__ float buf_sh[8][256];
+  const int t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float* buf = buf_sh[warp];
+  const int u = blockIdx.x * (blockDim.x >> 5) + warp;
+  const int nq = n_head * maps, nk = n_kv_head * maps;
+  if (u >= nq + nk + n_kv_head) return;
+  const int pos = positions[t], entry = row_entry[t];
+  const bool is_q = u < nq, is_k = !is_q && u < nq + nk;
+  const int i = is_q ? u : (is_k ? u - nq : u - nq - nk);          // index of the (head, map), or of the value head
+  const int m = is_q || is_k ? i % maps : 0;
+  T* dst = nullptr;
+  if (is_q) {
+    dst = q_out + (size_t)t * ldq + (size_t)i * hd;
+  } else if (entry >= 0 && cache != nullptr) {
+    const int page = block_table[(size_t)entry * max_blocks + pos / page_size];
+    if (page < 0 || page >= n_pages) {
+      if (lane == 0) *status = NIB_STATUS_BAD_PAGE;
+    } else {
+      dst = cache + kv_offset(page, is_k ? 0 : 1, is_k ? i / maps : i, pos % page_size, n_kv_head, page_size, hd);
+    }
+  }
+  // the rotation's angles do not wait for the projection
+  const int half = rot_dims / 2;
+  float cs[4], sn[4];
+  if (is_q || is_k) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int j = lane + 32 * k;
+      if (j < half) {
+        double sd, cd;
+        sincos((double)pos * freqs[j], &sd, &cd);
+        cs[k] = (float)cd * amp;
+        sn[k] = (float)sd * amp;
+      }
+    }
+  }
+  pdl_wait();
+  if (dst == nullptr) return;
+  if (!is_q && !is_k) {
+    const float* src = proj + (size_t)t * ld + v_off + (size_t)i * vdim;
+    for (int c = lane; c < hd; c += 32) dst[c] = from_float<T>(c < vdim ? src[c] : 0.0f);
+    return;
+  }
+  const float* src = proj + (size_t)t * ld + (is_q ? q_off : k_off) + (size_t)i * dim;
+  const float* w = is_q ? wq : wk;
+  float x[8], ss = 0.0f;
+#pragma unroll
+  for (int k = 0; k < 8; ++k) {
+    const int c = lane + 32 * k;
+    x[k] = c < dim ? src[c] : 0.0f;
+    ss += x[k] * x[k];
+  }
+  const float r = w != nullptr ? 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps) : 1.0f;
+#pragma unroll
+  for (int k = 0; k < 8; ++k) {
+    const int c = lane + 32 * k;
+    if (c < dim) buf[c] = w != nullptr ? x[k] * r * w[c] : x[k];
+  }
+  __syncwarp();
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int j = lane + 32 * k;
+    if (j < half) {
+      const float a = buf[j], b = buf[j + half];
+      buf[j] = a * cs[k] - b * sn[k];
+      buf[j + half] = b * cs[k] + a * sn[k];
+    }
+  }
+  __syncwarp();
+  // a query owns its whole head of hd values; a key its map's place, the last map's also what lies behind it
+  const int c_begin = is_q ? 0 : m * dim, c_end = is_q || m == maps - 1 ? hd : (m + 1) * dim;
+  for (int c = c_begin + lane; c < c_end; c += 32) {
+    const int d = c - m * dim;
+    dst[c] = from_float<T>(d >= 0 && d < dim ? buf[d] : 0.0f);
+  }
+}
+
+}  // namespace nib
+
+// maps * dim <= hd, vdim <= hd, dim <= 256, rot_dims even and at most dim; cache may be null (queries only).
+extern "C" int nib_norm_rope_maps_append(int dtype, const float* proj, int ld, int q_off, int k_off, int v_off, int n_head,
+                                         int n_kv_head, int maps, int dim, int vdim, int hd, const float* wq,
+                                         const float* wk, float eps, int rot_dims, const double* freqs, float amp,
+                                         const int* positions, const int* row_entry, void* q_out, int ldq, void* cache,
+                                         const int* block_table, int max_blocks, int page_size, int n_pages, int T,
+                                         int* status, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (maps <= 0 || dim <= 0 || vdim <= 0 || maps * dim > hd || vdim > hd || rot_dims < 0 || rot_dims > dim || (rot_dims & 1))
+    return NIB_ERR_BAD_ARGUMENT;
+  if (rot_dims > 0 && freqs == nullptr) return NIB_ERR_BAD_ARGUMENT;
+  if (dim > 256 || T > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
+  const int total = (n_head + n_kv_head) * maps + n_kv_head;
+  const int warps = total < 8 ? total : 8;
+  const dim3 grid((total + warps - 1) / warps, T), block(32 * warps);
+  if (dtype == DT_F32)
+    launch_pdl(norm_rope_maps_append_kernel<float>, grid, block, 0, stream, proj, ld, q_off, k_off, v_off, n_head,
+               n_kv_head, maps, dim, vdim, hd, wq, wk, eps, rot_dims, freqs, amp, positions, row_entry, (float*)q_out, ldq,
+               (float*)cache, block_table, max_blocks, page_size, n_pages, status);
+  else if (dtype == DT_BF16)
+    launch_pdl(norm_rope_maps_append_kernel<bf16>, grid, block, 0, stream, proj, ld, q_off, k_off, v_off, n_head,
+               n_kv_head, maps, dim, vdim, hd, wq, wk, eps, rot_dims, freqs, amp, positions, row_entry, (bf16*)q_out, ldq,
+               (bf16*)cache, block_table, max_blocks, page_size, n_pages, status);
+  else
+    return NIB_ERR_BAD_ARGUMENT;
+  NIB_LAUNCH_CHECK();
+}

@@ -58,14 +58,14 @@ _SIGNATURES = {
     "nib_attention_prefill_tc_supported": [_c_int, _c_int],
     "nib_attention_prefill_tc": [_c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr,
                                  _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float, _c_int,
-                                 _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
+                                 _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr],
     "nib_attention_simt": [_c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
                            _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float, _c_int,
-                           _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
+                           _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr],
     "nib_attention_decode": [_c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
                              _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float,
-                             _c_int, _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr,
-                             _c_ptr],
+                             _c_int, _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
+                             _c_ptr, _c_ptr],
     "nib_attention_decode_mma_supported": [_c_int, _c_int],
     "nib_attention_decode_mma_clusters": [_c_int, _c_int],
     "nib_attention_decode_mma": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
@@ -74,7 +74,7 @@ _SIGNATURES = {
     "nib_attention_prefill_supported": [_c_int],
     "nib_attention_prefill": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
                               _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float, _c_int,
-                              _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
+                              _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr],
     "nib_convert": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, ctypes.c_longlong, ctypes.c_longlong, _c_int, _c_ptr],
     "nib_argmax": [_c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "nib_sample": [_c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int,
@@ -86,11 +86,12 @@ _SIGNATURES = {
     "nib_unary": [_c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "nib_latent_prep": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_float,
                         _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
-                        _c_ptr, _c_ptr],
+                        _c_int, _c_ptr, _c_ptr],
     "nib_rope_heads": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
-                       _c_int, _c_int, _c_ptr],
+                       _c_int, _c_int, _c_int, _c_ptr],
     "nib_latent_attention": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int,
-                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr],
+                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr,
+                             _c_ptr],
     "nib_linear_heads": [_c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                          _c_int, _c_int, _c_ptr],
     "nib_delta_rule": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
@@ -141,6 +142,16 @@ _SIGNATURES = {
     "nib_selective_scan": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
                            _c_ptr, _c_ptr, ctypes.c_longlong, ctypes.c_longlong, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
                            _c_ptr, _c_int, _c_ptr],
+    "nib_group_norm": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_ptr],
+    "nib_embed_group_norm": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float,
+                             _c_ptr],
+    "nib_norm_rope_maps_append": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                                  _c_int, _c_ptr, _c_ptr, _c_float, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_ptr, _c_int,
+                                  _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
+    "nib_diff_combine": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int,
+                         _c_int, _c_ptr],
+    "nib_min_gru": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr,
+                    _c_int, _c_int, _c_ptr, _c_int, _c_ptr],
 }
 
 
@@ -649,21 +660,22 @@ class AttnExtras:
     sigmoid(gate[t, h]); ``out_scale``: and times this constant; ``span`` > 0: position i sees key j only if
     i // span == j // span (spans count from position 0 of the sequence); ``head_scale`` (float32 [n_head]): the
     scale times head_scale[h]; ``sinks`` (float32 [n_head]): with a sink, its term of the denominator is
-    exp(sinks[h]) instead of exp(0)."""
+    exp(sinks[h]) instead of exp(0); ``out32``: the output is float32 whatever the dtype of queries and cache."""
 
-    __slots__ = ("softcap", "keep_first", "slopes", "gate", "out_scale", "span", "head_scale", "sinks")
+    __slots__ = ("softcap", "keep_first", "slopes", "gate", "out_scale", "span", "head_scale", "sinks", "out32")
 
     def __init__(self, softcap: float = 0.0, keep_first: int = 0, slopes: Optional[torch.Tensor] = None,
                  gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, span: int = 0,
-                 head_scale: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
+                 head_scale: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, out32: bool = False):
         self.softcap, self.keep_first, self.slopes = float(softcap), int(keep_first), slopes
         self.gate, self.out_scale = gate, float(out_scale)
-        self.span, self.head_scale, self.sinks = int(span), head_scale, sinks
+        self.span, self.head_scale, self.sinks, self.out32 = int(span), head_scale, sinks, bool(out32)
 
     @property
     def plain(self) -> bool:
         return not (self.softcap > 0.0 or self.keep_first > 0 or self.slopes is not None or self.gate is not None
-                    or self.out_scale != 1.0 or self.span > 0 or self.head_scale is not None or self.sinks is not None)
+                    or self.out_scale != 1.0 or self.span > 0 or self.head_scale is not None or self.sinks is not None
+                    or self.out32)
 
     def args(self) -> tuple:
         g = self.gate
@@ -675,10 +687,15 @@ class AttnExtras:
         if self.span < 0:
             raise KernelError("attention: span must not be negative")
         return (self.softcap, self.keep_first, _ptr(self.slopes), _ptr(g), g.stride(0) if g is not None else 0,
-                self.out_scale, self.span, _ptr(self.head_scale), _ptr(self.sinks))
+                self.out_scale, self.span, _ptr(self.head_scale), _ptr(self.sinks), int(self.out32))
 
 
 _NO_EXTRAS = AttnExtras()
+
+
+def _attn_out_ok(out: torch.Tensor, dtype: torch.dtype, extras: Optional[AttnExtras]) -> bool:
+    """The output is in the dtype of queries and cache, or 32-bit floats where that was asked for."""
+    return out.dtype == (torch.float32 if extras is not None and extras.out32 else dtype)
 
 
 def attention_simt(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
@@ -688,7 +705,7 @@ def attention_simt(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bloc
     """Causal attention of T rows of q ([*, n_head * head_dim], any row stride) over one cache layer, with
     the general kernel (any head size up to 256, any page size).  ``rows`` lists the rows to process."""
     n_pages, _, n_kv_head, page_size, head_dim = cache.shape
-    if q.dtype != cache.dtype or out.dtype != cache.dtype or q.stride(1) != 1 or out.stride(1) != 1:
+    if q.dtype != cache.dtype or not _attn_out_ok(out, q.dtype, extras) or q.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("attention: q, out and cache must share a dtype, rows contiguous")
     _check(library().nib_attention_simt(_dt(q), _ptr(q), q.stride(0), _ptr(cache), _ptr(out), out.stride(0),
                                         _ptr(block_table), block_table.shape[1], _ptr(rows), _ptr(row_entry),
@@ -772,9 +789,14 @@ def decode_split(n_rows: int, n_head: int, max_keys: int, resident: int = DECODE
 
 
 def _note_attention(n_q: int, keys_seen: float, kv_rows: float, n_head: int, n_kv_head: int, head_dim: int,
-                    itemsize: int) -> None:
+                    itemsize: int, sizes=None, out_bytes: int = 0) -> None:
     """[queries, keys seen by them in all, width]: per key and head the score (2 hd), the softmax (~5)
     and the weighted sum (2 hd); the queries and outputs, and ``kv_rows`` key and value rows read once."""
+    if sizes is not None:     # (key, value, cached key row) sizes of their own: padding is not work
+        key, value, row = sizes
+        _note("attn", "attn", (n_q, int(keys_seen), n_head * value), keys_seen * n_head * (2.0 * (key + value) + 5.0),
+              n_q * n_head * (itemsize * key + (out_bytes or itemsize) * value) + itemsize * kv_rows * n_kv_head * (row + value))
+        return
     width = n_head * head_dim
     _note("attn", "attn", (n_q, int(keys_seen), width), keys_seen * (4.0 * width + 5.0 * n_head),
           itemsize * (2.0 * n_q * width + 2.0 * kv_rows * n_kv_head * head_dim))
@@ -798,7 +820,7 @@ def attention_decode(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
     96 or 128 runs on the warp-level MMA kernel, everything else (and float32, in true 32-bit
     arithmetic) on the streaming kernel."""
     n_pages, _, n_kv_head, page_size, head_dim = cache.shape
-    if q.dtype != cache.dtype or out.dtype != cache.dtype or q.stride(1) != 1 or out.stride(1) != 1:
+    if q.dtype != cache.dtype or not _attn_out_ok(out, q.dtype, extras) or q.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("attention: q, out and cache must share a dtype, rows contiguous")
     plain = extras is None or extras.plain     # (the MMA kernel takes no options on the scores or the output)
     mma = USE_DECODE_MMA and plain and q.dtype == torch.bfloat16 and _can("nib_attention_decode_mma_supported", head_dim, page_size) \
@@ -847,7 +869,7 @@ def attention_prefill_tc(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor
     """tcgen05 attention for prompt portions (bfloat16, head size 64): ``tiles`` holds (entry, first
     row within the entry) pairs of 128 rows each; ``q`` holds the step's ``n_rows`` rows."""
     n_pages, _, n_kv_head, page_size, head_dim = cache.shape
-    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or not _attn_out_ok(out, q.dtype, extras):
         raise KernelError("attention_prefill_tc: bfloat16 only")
     if not cache.is_contiguous() or q.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("attention_prefill_tc: contiguous cache layer and rows")
@@ -866,7 +888,7 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, b
     """Tiled tensor-core attention for prompt portions: ``tiles`` holds (entry, first row within the
     entry) pairs of 64 rows each."""
     n_pages, _, n_kv_head, page_size, head_dim = cache.shape
-    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or not _attn_out_ok(out, q.dtype, extras):
         raise KernelError("attention_prefill: bfloat16 only")
     _check(library().nib_attention_prefill(_ptr(q), q.stride(0), _ptr(cache), _ptr(out), out.stride(0),
                                            _ptr(block_table), block_table.shape[1], _ptr(tiles), n_tiles,
@@ -877,14 +899,15 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, b
 
 def attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, ctx,
               n_head: int, scale: float, window: int, plan, sink: bool = False,
-              extras: Optional[AttnExtras] = None) -> None:
+              extras: Optional[AttnExtras] = None, sizes=None) -> None:
     """Causal attention of the step's rows over one cache layer.  ``extras``: options on the scores and the output
     (``AttnExtras``); the kernels that take them are the general one, the two of prompt portions and the streaming split-KV one.  ``sink``: the softmax's denominator has
     one more term, exp(0) (a key of score 0 that has no value; every kernel adds it where it divides).
     ``ctx`` is the step's StepContext, ``plan`` says which rows are single decoded tokens and how the
     prompt portions are cut into tiles (``parts.attention.AttentionPlan``).  Single decoded tokens go to the split-KV kernel;
     prompt portions go to the tiled tensor-core kernels in bfloat16 (head sizes 16..128 in steps of
-    16) and to the general kernel otherwise."""
+    16) and to the general kernel otherwise.  ``sizes`` (for the trace's counts only): the sizes of a head's key and
+    value and of a cached key row, where they are smaller than the cache's head size."""
     n_pages, _, n_kv_head, page_size, head_dim = cache.shape
     fast_pages = page_size % 16 == 0 and head_dim % 8 == 0 and head_dim <= 128
     plain = extras is None or extras.plain
@@ -892,7 +915,7 @@ def attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_tab
     if not fast_pages:
         if traced:
             _note_attention(ctx.n_rows, plan.decode_keys + plan.prefill_keys, plan.decode_keys + plan.prefill_kv_rows,
-                            n_head, n_kv_head, head_dim, q.element_size())
+                            n_head, n_kv_head, head_dim, q.element_size(), sizes, out.element_size())
         attention_simt(q, cache, out, block_table, ctx.row_entry, ctx.positions, ctx.n_rows, n_head, scale,
                        window, ctx.status, sink=sink, extras=extras)
         return
@@ -902,13 +925,13 @@ def attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_tab
             keys = min(keys, extras.span)
         if traced:
             _note_attention(plan.n_decode, plan.decode_keys, plan.decode_keys, n_head, n_kv_head, head_dim,
-                            q.element_size())
+                            q.element_size(), sizes, out.element_size())
         attention_decode(q, cache, out, block_table, ctx.row_entry, ctx.positions, plan.n_decode, n_head, scale,
                          window, ctx.status, keys, ctx.workspace, plan.decode_rows, sink=sink, extras=extras)
     if plan.n_prefill_rows:
         if traced:
             _note_attention(plan.n_prefill_rows, plan.prefill_keys, plan.prefill_kv_rows, n_head, n_kv_head, head_dim,
-                            q.element_size())
+                            q.element_size(), sizes, out.element_size())
         if q.dtype == torch.bfloat16 and scale > 0 and _can("nib_attention_prefill_tc_supported", head_dim, page_size) \
                 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0 \
                 and out.data_ptr() % 16 == 0:
@@ -1052,11 +1075,13 @@ def unary(src: torch.Tensor, out: torch.Tensor, n_rows: int, kind: int, prm: Opt
 def latent_prep(proj: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, rot_dims: int, freqs: torch.Tensor,
                 wq: torch.Tensor, wkv: Optional[torch.Tensor], eps: float, cq: torch.Tensor,
                 cache: Optional[torch.Tensor], block_table: Optional[torch.Tensor], row_entry: torch.Tensor,
-                positions: torch.Tensor, T: int, status: torch.Tensor) -> None:
-    """From the down-projections' output ``proj`` (float32 [T, q_rank (+ kv_rank + rot_dim)]): the normed query
+                positions: torch.Tensor, T: int, status: torch.Tensor, halves: bool = False) -> None:
+    """From the down-projections' output ``proj`` (float32 [T, >= q_rank (+ kv_rank + rot_dim)]): the normed query
     latent into ``cq``, and (with ``cache``, one layer [pages, 1, 1, page_size, kv_rank + rot_dim]) the normed
-    key/value latent and the rotated shared key part into the rows' cache slots."""
-    _f32(proj, "latent_prep: proj")
+    key/value latent and the rotated shared key part into the rows' cache slots.  ``halves``: the rotation pairs value
+    i with value i + rot_dims / 2 instead of (2i, 2i + 1)."""
+    if proj.dtype != torch.float32 or proj.stride(1) != 1:
+        raise KernelError("latent_prep: proj must be float32 with contiguous rows")
     if freqs.dtype != torch.float64 or cq.stride(1) != 1:
         raise KernelError("latent_prep: freqs must be float64, cq rows contiguous")
     has_kv = cache is not None
@@ -1073,14 +1098,14 @@ def latent_prep(proj: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, rot
     _check(library().nib_latent_prep(_dt(cq), _ptr(proj), proj.stride(0), q_rank, kv_rank, rot_dim, rot_dims,
                                      _ptr(freqs), _ptr(wq), _ptr(wkv), float(eps), _ptr(cq), cq.stride(0),
                                      _ptr(cache), _ptr(block_table), block_table.shape[1] if has_kv else 0,
-                                     _ptr(row_entry), _ptr(positions), T, page_size, n_pages, int(has_kv),
+                                     _ptr(row_entry), _ptr(positions), T, page_size, n_pages, int(has_kv), int(halves),
                                      _ptr(status), _stream()), "latent_prep")
 
 
 def rope_heads(q: torch.Tensor, nope: int, rot_dim: int, rot_dims: int, freqs: torch.Tensor,
-               positions: torch.Tensor, out: torch.Tensor, out_off: int, n_head: int, T: int) -> None:
+               positions: torch.Tensor, out: torch.Tensor, out_off: int, n_head: int, T: int, halves: bool = False) -> None:
     """Rotates the last ``rot_dim`` values of every head of q ([T, n_head * (nope + rot_dim)]) by the rows'
-    positions (interleaved pairs over the first ``rot_dims``) into out[t, h, out_off:], float32 [T, n_head, D]."""
+    positions (interleaved pairs over the first ``rot_dims``, or halves) into out[t, h, out_off:], float32 [T, n_head, D]."""
     _f32(out, "rope_heads: out")
     if q.stride(1) != 1 or freqs.dtype != torch.float64:
         raise KernelError("rope_heads: q rows contiguous, freqs float64")
@@ -1088,7 +1113,7 @@ def rope_heads(q: torch.Tensor, nope: int, rot_dim: int, rot_dims: int, freqs: t
         _note("other", "rope", (T, n_head * rot_dim, 0), 6.0 * T * n_head * rot_dim,
               T * n_head * rot_dim * (q.element_size() + 4))
     _check(library().nib_rope_heads(_dt(q), _ptr(q), q.stride(0), nope, rot_dim, rot_dims, _ptr(freqs),
-                                    _ptr(positions), _ptr(out), out.shape[2], out_off, n_head, T, _stream()),
+                                    _ptr(positions), _ptr(out), out.shape[2], out_off, n_head, T, int(halves), _stream()),
            "rope_heads")
 
 
@@ -1111,10 +1136,14 @@ def latent_attention_reserve(workspace, n_head: int, kv_rank: int) -> None:
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, ctx,
-                     n_head: int, kv_rank: int, scale: float, window: int, n_splits: Optional[int] = None) -> None:
+                     n_head: int, kv_rank: int, scale: float, window: int, n_splits: Optional[int] = None,
+                     gate: Optional[torch.Tensor] = None) -> None:
     """Causal softmax attention of the step's rows over one latent cache layer: q float32 [T, n_head, D] (the
     absorbed query, then the rotated part), out [T, n_head * kv_rank] the weighted sums of latents.  A step of
-    few rows (decoded tokens) cuts every row's keys into ``n_splits`` pieces, merged by a second kernel."""
+    few rows (decoded tokens) cuts every row's keys into ``n_splits`` pieces, merged by a second kernel.  ``gate``
+    (float32 [rows, >= n_head], any row stride): head h's output of row t times sigmoid(gate[t, h])."""
+    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1):
+        raise KernelError("latent_attention: the gate must be float32 with contiguous rows")
     n_pages, _, _, page_size, D = cache.shape
     if n_splits is None:
         n_splits = latent_splits(ctx.n_rows, n_head)
@@ -1134,7 +1163,8 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
     _check(library().nib_latent_attention(_dt(cache), _ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
                                           block_table.shape[1], None, _ptr(ctx.row_entry), _ptr(ctx.positions),
                                           ctx.n_rows, n_head, kv_rank, D, page_size, n_pages, float(scale),
-                                          int(window), _ptr(ctx.status), int(n_splits), _ptr(partials), _stream()),
+                                          int(window), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                          _ptr(ctx.status), int(n_splits), _ptr(partials), _stream()),
            "latent_attention", 2 if n_splits > 1 else 1)
 
 
@@ -1738,3 +1768,119 @@ def selective_scan(dtp: torch.Tensor, x: torch.Tensor, bc: torch.Tensor, b_off: 
                                         state.stride(0), int(s_off), _ptr(ctx.entry_start), _ptr(ctx.entry_slot),
                                         ctx.n_entries, int(inner), int(n), _ptr(out), out.stride(0), _stream()),
            "selective_scan")
+
+
+# ----------------------------------------------------------------------------- norms in groups
+def group_norm(x: torch.Tensor, weight: Optional[torch.Tensor], groups: int, eps: float, out: Optional[torch.Tensor],
+               n_rows: int, rows: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None) -> None:
+    """out[r] = norm(x[rows[r]]) (rows None: x[r]): the row cut into ``groups`` equal parts, each over its own root mean
+    square (``eps`` inside the root), the whole times ``weight``; x is the 32-bit stream.  ``add`` (float32 [C]) is added
+    to the rows first, and x receives the sum; with ``out`` None that is all that happens."""
+    C = x.shape[1]
+    _f32(x, "group_norm: x")
+    if out is not None:
+        _f32(weight, "group_norm: weight")
+        if weight.numel() != C or out.shape[1] != C or out.shape[0] < n_rows or not out.is_contiguous():
+            raise KernelError("group_norm: weight [C], out contiguous [n_rows, C]")
+    if rows is not None:
+        _i32(rows, "rows")
+    if add is not None:
+        _f32(add, "group_norm: add")
+        if add.numel() != C or rows is not None:
+            raise KernelError("group_norm: add is one vector [C], for all rows in order")
+    if groups <= 0 or C % groups:
+        raise KernelError("group_norm: the parts must divide the width")
+    if tracing():
+        _note("ln", "ln", (n_rows, C, groups), 4.0 * n_rows * C,
+              n_rows * C * (4 + (out.element_size() if out is not None else 0) + (4 if add is not None else 0)) + 4 * C)
+    _check(library().nib_group_norm(_dt(out) if out is not None else 0, _ptr(x), _ptr(rows), _ptr(add), _ptr(weight),
+                                    _ptr(out), n_rows, C, int(groups), float(eps), _stream()), "group_norm")
+
+
+def embed_group_norm(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, weight: torch.Tensor, groups: int,
+                     eps: float, feedback: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+    """out[t] = norm(table[tokens[t]] * scale) as 32-bit floats, the norm in groups; tokens as in ``embed``."""
+    T, C = tokens.shape[0], table.shape[1]
+    _i32(tokens, "tokens"); _f32(weight, "embed_group_norm: weight")
+    if out.dtype != torch.float32 or out.shape[0] < T or out.shape[1] != C or not out.is_contiguous() \
+            or not table.is_contiguous() or weight.numel() != C or groups <= 0 or C % groups:
+        raise KernelError("embed_group_norm: out contiguous float32 [T, C], weight [C], parts that divide C")
+    if feedback is not None:
+        _i32(feedback, "feedback")
+    if tracing():
+        _note("embed", "embed", (T, C, groups), 5.0 * T * C, T * C * (table.element_size() + 4))
+    _check(library().nib_embed_group_norm(_dt(table), _ptr(tokens), _ptr(feedback), _ptr(table), float(scale), _ptr(weight),
+                                          _ptr(out), T, C, int(groups), float(eps), _stream()), "embed_group_norm")
+
+
+# ----------------------------------------------------------------------------- differential attention
+def norm_rope_maps_append(proj: torch.Tensor, offsets, n_head: int, n_kv_head: int, maps: int, dim: int, vdim: int,
+                          wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float, rot_dims: int,
+                          freqs: Optional[torch.Tensor], amp: float, ctx, q_out: torch.Tensor,
+                          cache: Optional[torch.Tensor], block_table: Optional[torch.Tensor]) -> None:
+    """From the 32-bit projection ``proj`` (q [n_head][maps][dim], k [n_kv_head][maps][dim], v [n_kv_head][vdim] at the
+    three column ``offsets``): an RMS norm of every (head, map) of q and k with a weight of ``dim`` values that all share
+    (None: no norm), rotary positions in the halves layout (cosine and sine times ``amp``), the cast; keys to plane 0 of
+    the rows' cache slots, the maps of a head side by side in a row of the cache's head size, values to plane 1; the query
+    of map m to head h * maps + m of ``q_out`` [rows, n_head * maps * head size] at its map's place in that row, zeros
+    elsewhere.  ``cache`` None: queries only."""
+    if proj.dtype != torch.float32 or proj.stride(1) != 1:
+        raise KernelError("norm_rope_maps_append: proj must be float32 with contiguous rows")
+    hd = q_out.shape[1] // (n_head * maps)
+    if cache is not None:
+        n_pages, two, g, page_size, chd = cache.shape
+        if two != 2 or g != n_kv_head or chd != hd or not cache.is_contiguous() or cache.dtype != q_out.dtype:
+            raise KernelError("norm_rope_maps_append: cache must be contiguous [pages, 2, kv heads, page, head size] of "
+                              "q_out's dtype")
+        _i32(block_table, "block_table")
+    else:
+        n_pages, page_size = 0, 1
+    for w in (wq, wk):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != dim):
+            raise KernelError("norm_rope_maps_append: a norm weight must be float32 [dim]")
+    if freqs is not None and freqs.dtype != torch.float64:
+        raise KernelError("norm_rope_maps_append: freqs must be float64")
+    if tracing():
+        n_in = (n_head + n_kv_head) * maps * dim + n_kv_head * vdim
+        n_out = (n_head * maps + 2 * n_kv_head) * hd
+        _note("kv_write", "norm_kv_write", (ctx.n_rows, n_out, 0), 8.0 * ctx.n_rows * n_in,
+              ctx.n_rows * (4.0 * n_in + n_out * q_out.element_size()))
+    _check(library().nib_norm_rope_maps_append(
+        _dt(q_out), _ptr(proj), proj.stride(0), offsets[0], offsets[1], offsets[2], n_head, n_kv_head, maps, dim, vdim, hd,
+        _ptr(wq), _ptr(wk), float(eps), rot_dims, _ptr(freqs), float(amp), _ptr(ctx.positions), _ptr(ctx.row_entry),
+        _ptr(q_out), q_out.stride(0), _ptr(cache), _ptr(block_table),
+        block_table.shape[1] if block_table is not None else 0, page_size, n_pages, ctx.n_rows, _ptr(ctx.status),
+        _stream()), "norm_rope_maps_append")
+
+
+def diff_combine(a: torch.Tensor, n_head: int, vdim: int, lam: float, eps: float, mul: float, out: torch.Tensor,
+                 n_rows: int) -> None:
+    """out[t, h * vdim + d] = mul * o_d / sqrt(mean(o^2) + eps), o = a[t, 2h] - lam * a[t, 2h + 1] over the first ``vdim``
+    values of the 32-bit heads ``a`` [rows, 2 * n_head * head size]."""
+    if a.dtype != torch.float32 or a.stride(1) != 1 or out.stride(1) != 1 or a.shape[1] % (2 * n_head) \
+            or out.shape[1] < n_head * vdim:
+        raise KernelError("diff_combine: a float32 [rows, 2 * heads * head size], out [rows, >= heads * vdim]")
+    if tracing():
+        n = n_head * vdim
+        _note("other", "diff_combine", (n_rows, n, 0), 6.0 * n_rows * n, n_rows * n * (8.0 + out.element_size()))
+    _check(library().nib_diff_combine(_dt(out), _ptr(a), a.stride(0), n_head, a.shape[1] // (2 * n_head), vdim, float(lam),
+                                      float(eps), float(mul), _ptr(out), out.stride(0), n_rows, _stream()), "diff_combine")
+
+
+# ----------------------------------------------------------------------------- the minimal gated recurrent unit
+def min_gru(proj: torch.Tensor, offsets, width: int, state: torch.Tensor, ctx, out: torch.Tensor) -> None:
+    """S <- S + z (c - S), out = S silu(g) over the step's rows, entry by entry in row order (csrc/min_gru.cu): z =
+    sigmoid(z logit), c = u + 1/2 where u >= 0 and sigmoid(u) where u < 0; the logits of z, u and g lie at the three
+    column ``offsets`` of the 32-bit ``proj``; ``state`` float32 [slots, >= width] is read and written at the entries'
+    slots; out[:, :width] in out's dtype."""
+    if proj.dtype != torch.float32 or proj.stride(1) != 1 or out.stride(1) != 1 or out.shape[1] < width:
+        raise KernelError("min_gru: proj float32, rows contiguous, out [rows, >= width]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < width:
+        raise KernelError("min_gru: state must be float32 [slots, >= width]")
+    if tracing():
+        T = ctx.n_rows
+        _note("scan", "min_gru", (T, width, 0), 20.0 * T * width,
+              T * width * (12.0 + out.element_size()) + 8.0 * ctx.n_entries * width)
+    _check(library().nib_min_gru(_dt(out), _ptr(proj), proj.stride(0), int(offsets[0]), int(offsets[1]), int(offsets[2]),
+                                 int(width), _ptr(state), state.stride(0), _ptr(ctx.entry_start), _ptr(ctx.entry_slot),
+                                 ctx.n_entries, ctx.n_rows, _ptr(out), out.stride(0), _stream()), "min_gru")

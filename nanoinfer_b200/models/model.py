@@ -14,6 +14,7 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
+from ..kernels import ops
 from ..parts import base as P
 from ..parts.block import BLOCKS, Block
 from .spec import ModelSpec, PartSpec
@@ -59,6 +60,8 @@ class Model:
             self.layers.append(cls(spec.width, built, **getattr(ls, "args", {})))
         self.final_norm = self._build(P.NORMS, spec.final_norm, "final_norm")
         self.head = self._build(P.HEADS, spec.head, "head")
+        self.stream_vectors = self._build(P.STREAM_VECTORS, spec.stream_vectors, "stream_vectors") \
+            if spec.stream_vectors else None
         self.schedule = list(spec.schedule)
         self._check_schedule()
         self.dtype: Optional[torch.dtype] = None
@@ -81,6 +84,9 @@ class Model:
         for i, e in enumerate(self.schedule):
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"schedule[{i}] names layer {e.layer}, but there are {len(self.layers)} layers")
+            if e.add_vector is not None and (self.stream_vectors is None
+                                             or not 0 <= e.add_vector < self.stream_vectors.count):
+                raise ValueError(f"schedule[{i}].add_vector {e.add_vector} names no stream vector")
             if e.cache_of is not None:
                 if not 0 <= e.cache_of < i or self.schedule[e.cache_of].cache_of is not None:
                     raise ValueError(f"schedule[{i}].cache_of must name an earlier entry that owns a cache")
@@ -116,6 +122,8 @@ class Model:
             pos = getattr(blk.mixer, "position", None)
             if pos is not None:
                 out.append(pos)
+        if self.stream_vectors is not None:
+            out.append(self.stream_vectors)
         out += [self.final_norm, self.head]
         return out
 
@@ -123,6 +131,8 @@ class Model:
         self.dtype, self.device = dtype, device
         for part in self.all_parts():
             part.prepare(dtype, device)
+        for blk in self.layers:
+            blk.prepare(dtype, device)
 
     # ------------------------------------------------------------------ what the cache manager must provide
     def kv_needs(self) -> List[Tuple[int, P.KVCacheSpec]]:
@@ -196,7 +206,15 @@ class Model:
         for i, e in enumerate(self.schedule):
             owner = i if e.cache_of is None else e.cache_of
             ctx.layer = i
-            ctx.next_block = self.layers[self.schedule[i + 1].layer] if i + 1 < len(self.schedule) else None
+            # (an arrangement may take the next one's first step ahead, unless a vector is added to the stream in between)
+            nxt = self.schedule[i + 1] if i + 1 < len(self.schedule) else None
+            ctx.next_block = self.layers[nxt.layer] if nxt is not None and nxt.add_vector is None else None
+            if e.add_vector is not None:
+                vector = self.stream_vectors.vector(e.add_vector)
+                if self.layers[e.layer].adds_vector:
+                    ctx.stream_vector = vector
+                else:
+                    ops.group_norm(x, None, 1, 0.0, None, ctx.n_rows, add=vector)
             self.layers[e.layer].forward(x, ctx, caches.get(owner), states.get(i), e.cache_of is None, self.dtype)
         ctx.layer, ctx.next_block = -1, None
         if n_logits <= 0:

@@ -52,6 +52,8 @@ class ScheduleEntry:
     layer: int                                  # index into ModelSpec.layers
     #: index of an EARLIER schedule entry whose keys and values this run reads; None: its own
     cache_of: Optional[int] = None
+    #: row of the model's stream vectors that is added to the residual stream ahead of this run; None: nothing
+    add_vector: Optional[int] = None
 
 
 @dataclass
@@ -70,3 +72,5 @@ class ModelSpec:
     #: regular expressions of tensors a checkpoint may hold that the model does not use
     ignorable: List[str] = field(default_factory=list)
     eos_token_id: Optional[int] = None
+    #: vectors that schedule entries add to the residual stream ahead of their run (``ScheduleEntry.add_vector``)
+    stream_vectors: Optional[PartSpec] = None

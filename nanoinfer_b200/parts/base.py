@@ -135,6 +135,9 @@ class StepPlan:
 
 
 class Norm(Part):
+    #: True: ``forward`` takes ``add``, a 32-bit vector that is added to the stream first, in the norm's own kernel
+    takes_vector = False
+
     def forward(self, x: torch.Tensor, out: torch.Tensor, n_rows: int,
                 rows: Optional[torch.Tensor] = None) -> None:
         """out[:n_rows] = norm(x[rows] or x[:n_rows]); x is the 32-bit residual stream."""
@@ -197,6 +200,85 @@ class Mixer(Part):
 
     def forward(self, xn: torch.Tensor, x: torch.Tensor, ctx: "StepContext", cache: Optional["KVCacheView"],
                 state: Optional[torch.Tensor], writes_cache: bool = True) -> None:
+        raise NotImplementedError
+
+
+class TwoProducts:
+    """A mixer or feed-forward that is ONE product of its input, something in between, and ONE product that adds into
+    the stream.  Where two such sublayers read the same input, an arrangement may make their first products one and
+    their second products one (``parallel_norm`` in block.py).
+
+    After ``prepare`` the part has ``w_in`` [n_in, width] (``b_in`` float32 [n_in] or None) and ``w_out`` [width, n_inner];
+    ``inner`` is what lies between: it reads the first product's result ``proj`` (float32 [rows, n_in], any row stride)
+    and leaves the second's input in ``out`` ([rows, n_inner], the engine's dtype, any row stride)."""
+
+    w_in: torch.Tensor
+    b_in: Optional[torch.Tensor] = None
+    w_out: torch.Tensor
+    n_in = n_inner = 0
+
+    def rebase(self, w_in: torch.Tensor, b_in: Optional[torch.Tensor], w_out: torch.Tensor) -> None:
+        """The same values in other memory (rows of a joint first matrix, columns of a joint second one): the
+        parameters that were views of the part's own matrices become views of these."""
+        old, start = self.w_in.untyped_storage().data_ptr(), self.w_in.storage_offset()
+        for key, t in self.params.items():
+            if t is self.w_out:
+                self.params[key] = w_out
+            elif t.untyped_storage().data_ptr() == old:
+                self.params[key] = w_in.as_strided(t.shape, t.stride(), w_in.storage_offset() + t.storage_offset() - start)
+            elif b_in is not None and t.untyped_storage().data_ptr() == self.b_in.untyped_storage().data_ptr():
+                self.params[key] = b_in.as_strided(t.shape, t.stride(), b_in.storage_offset() + t.storage_offset()
+                                                   - self.b_in.storage_offset())
+        self.w_in, self.w_out = w_in, w_out
+        if self.b_in is not None:
+            self.b_in = b_in
+
+    def stack_input(self, sections, width: int) -> None:
+        """``w_in`` (and ``b_in`` where a section has a bias) from (parameter name, first row) sections; parameters
+        ``<name>_weight`` and ``<name>_bias`` become views of them."""
+        p = self.params
+        first = p[sections[0][0] + "_weight"]
+        w = torch.zeros(self.n_in, width, dtype=first.dtype, device=first.device)
+        has_bias = any(name + "_bias" in p for name, _ in sections)
+        b = torch.zeros(self.n_in, dtype=torch.float32, device=first.device) if has_bias else None
+        for name, at in sections:
+            n = p[name + "_weight"].shape[0]
+            w[at:at + n] = p[name + "_weight"]
+            p[name + "_weight"] = w[at:at + n]
+            if name + "_bias" in p:
+                b[at:at + n] = p[name + "_bias"]
+                p[name + "_bias"] = b[at:at + n]
+        self.w_in, self.b_in = w, b
+
+    def inner(self, proj: torch.Tensor, out: torch.Tensor, ctx: "StepContext", cache: Optional["KVCacheView"] = None,
+              state: Optional[torch.Tensor] = None, writes_cache: bool = True) -> None:
+        raise NotImplementedError
+
+    def reserve_products(self, workspace: "Workspace", limits: "StepLimits") -> None:
+        workspace.reserve("two_products.proj", limits.max_rows * self.n_in, torch.float32)
+        workspace.reserve("two_products.inner", limits.max_rows * self.n_inner, limits.dtype)
+
+    def run_alone(self, xn, x: torch.Tensor, ctx: "StepContext", cache: Optional["KVCacheView"] = None,
+                  state: Optional[torch.Tensor] = None, writes_cache: bool = True, names=("in", "out")) -> None:
+        from ..kernels import ops
+
+        if isinstance(xn, ops.NormInput):
+            xn = xn.materialise(ctx.n_rows)
+        T, ws = ctx.n_rows, ctx.workspace
+        proj = ws.get("two_products.proj", (ctx.max_rows, self.n_in), torch.float32)
+        out = ws.get("two_products.inner", (ctx.max_rows, self.n_inner), self.dtype)
+        ops.trace_scope(ctx.layer, names[0])
+        ops.linear(xn, self.w_in, self.b_in, proj, T)
+        self.inner(proj, out, ctx, cache, state, writes_cache)
+        ops.trace_scope(ctx.layer, names[1])
+        ops.linear(out, self.w_out, None, x, T, residual=True)
+
+
+class StreamVectors(Part):
+    """Vectors that a schedule adds to the residual stream ahead of some of its runs (``ScheduleEntry.add_vector`` names
+    a row)."""
+
+    def vector(self, i: int) -> torch.Tensor:
         raise NotImplementedError
 
 
@@ -269,6 +351,7 @@ EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
 DEPTH_MIXES = Registry("depth mix")
 CONNECTORS = Registry("connector")
+STREAM_VECTORS = Registry("stream vectors")
 
 register_norm = NORMS.register
 register_position = POSITIONS.register
@@ -278,6 +361,7 @@ register_embedding = EMBEDDINGS.register
 register_head = HEADS.register
 register_depth_mix = DEPTH_MIXES.register
 register_connector = CONNECTORS.register
+register_stream_vectors = STREAM_VECTORS.register
 
 
 # ----------------------------------------------------------------------------- what a step shows to the parts
@@ -323,6 +407,9 @@ class StepContext:
     #: next one's first step in its own last kernel and say so in ``stream_entered``
     next_block: Optional[object] = None
     stream_entered: bool = False
+    #: float32 [width], to be added to the stream ahead of the run that starts next (None: nothing); an arrangement
+    #: that does this itself (``Block.adds_vector``) takes it away
+    stream_vector: Optional[torch.Tensor] = None
     #: int32 [slots]: the token last sampled for each slot, left on the device by the sampler; a
     #: negative entry -(s + 1) of ``tokens`` stands for ``token_feedback[s]``
     token_feedback: Optional[torch.Tensor] = None

@@ -12,7 +12,7 @@ import torch
 
 from ..kernels import ops
 from .base import (CONNECTORS, DEPTH_MIXES, FEED_FORWARDS, MIXERS, NORMS, KVCacheView, Mixer, Part, Registry, StepContext,
-                   StepLimits, Workspace)
+                   StepLimits, TwoProducts, Workspace)
 
 BLOCKS: Dict[str, Type["Block"]] = {}
 
@@ -30,6 +30,8 @@ class Block:
     slots: ClassVar[Dict[str, Registry]] = {}
     #: names of ``slots`` that a layer may leave out
     optional: ClassVar[tuple] = ()
+    #: True: ``forward`` adds ``ctx.stream_vector`` to the stream itself before anything else (and takes it away)
+    adds_vector: ClassVar[bool] = False
 
     def __init__(self, width: int, parts: Dict[str, Part]):
         missing, unknown = set(self.slots) - set(parts) - set(self.optional), set(parts) - set(self.slots)
@@ -48,6 +50,9 @@ class Block:
 
     def parts(self) -> Dict[str, Part]:
         return dict(self._parts)
+
+    def prepare(self, dtype: torch.dtype, device: torch.device) -> None:
+        """Called once after the parts' own ``prepare``."""
 
     def reserve(self, workspace: Workspace, limits: StepLimits) -> None:
         """Size the arrangement's own scratch (the parts size theirs themselves)."""
@@ -329,3 +334,84 @@ class HyperConnectionBlock(Block):
             self._back(self.connect_2, xn, y, copies, gate, ctx, T, last[0], last[1], total)
         if fuse:
             ctx.stream_entered = True
+
+
+@register_block("parallel_norm")
+class ParallelNormBlock(Block):
+    """One norm that both sublayers read, and one sum:
+        h = norm_1(x);   x <- x + (mixer(h) + feed_forward(h))
+    (a layer may have no feed-forward).  A vector that the schedule adds to the stream ahead of the layer
+    (``ctx.stream_vector``) is added by the norm's kernel.
+
+    The norm is taken once, ahead of both, so both sublayers add their products straight into the stream.  Where both are
+    ``TwoProducts`` parts the layer has two products in all: their first matrices lie under one another as one ([mixer's
+    rows | feed-forward's rows], 32-bit results), and their second matrices side by side as one, whose input is one row
+    [mixer's inner values | feed-forward's]; a step of few rows streams a layer's weights in two launches."""
+
+    slots = {"norm_1": NORMS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS}
+    optional = ("feed_forward",)
+    adds_vector = True
+
+    def __init__(self, width: int, parts: Dict[str, Part]):
+        super().__init__(width, parts)
+        self.feed_forward = parts.get("feed_forward")
+        #: whether the norm's kernel adds a vector to the stream as well
+        self.norm_adds = parts["norm_1"].takes_vector
+        self.joint = isinstance(self.mixer, TwoProducts) and isinstance(self.feed_forward, TwoProducts)
+        if self.joint:
+            m, f = self.mixer, self.feed_forward
+            up8 = lambda n: -(-n // 8) * 8
+            self.ff_row = up8(m.n_in)                     # first row (and column of the result) of the feed-forward
+            self.n_in = self.ff_row + up8(f.n_in)
+            # (no padding between or behind the inner values: a padded column would have to hold a number, not whatever
+            # another layer left there)
+            self.n_inner = m.n_inner + f.n_inner
+
+    def prepare(self, dtype, device) -> None:
+        if not self.joint:
+            return
+        m, f = self.mixer, self.feed_forward
+        w_in = torch.zeros(self.n_in, self.width, dtype=dtype, device=device)
+        w_in[:m.n_in], w_in[self.ff_row:self.ff_row + f.n_in] = m.w_in, f.w_in
+        b_in = None
+        if m.b_in is not None or f.b_in is not None:
+            b_in = torch.zeros(self.n_in, dtype=torch.float32, device=device)
+            for part, at in ((m, 0), (f, self.ff_row)):
+                if part.b_in is not None:
+                    b_in[at:at + part.n_in] = part.b_in
+        w_out = torch.cat([m.w_out, f.w_out], 1).contiguous()
+        for part, at, k in ((m, 0, 0), (f, self.ff_row, m.n_inner)):
+            part.rebase(w_in[at:at + part.n_in], None if b_in is None else b_in[at:at + part.n_in],
+                        w_out[:, k:k + part.n_inner])
+        self.w_in, self.b_in, self.w_out = w_in, b_in, w_out
+
+    def reserve(self, workspace, limits) -> None:
+        workspace.reserve("block.normed", limits.max_rows * self.width, limits.dtype)
+        if self.joint:
+            workspace.reserve("two_products.proj", limits.max_rows * self.n_in, torch.float32)
+            workspace.reserve("two_products.inner", limits.max_rows * self.n_inner, limits.dtype)
+
+    def forward(self, x, ctx, cache, state, writes_cache, dtype) -> None:
+        T, ws = ctx.n_rows, ctx.workspace
+        xn = ws.get("block.normed", (ctx.max_rows, self.width), dtype)
+        add, ctx.stream_vector = ctx.stream_vector, None
+        if self.norm_adds:
+            self.norm_1.forward(x, xn, T, add=add)
+        else:
+            if add is not None:
+                ops.group_norm(x, None, 1, 0.0, None, T, add=add)
+            self.norm_1.forward(x, xn, T)
+        m, f = self.mixer, self.feed_forward
+        if not self.joint:
+            m.forward(xn, x, ctx, cache, state, writes_cache)
+            if f is not None:
+                f.forward(xn, x, ctx)
+            return
+        proj = ws.get("two_products.proj", (ctx.max_rows, self.n_in), torch.float32)
+        mid = ws.get("two_products.inner", (ctx.max_rows, self.n_inner), dtype)
+        ops.trace_scope(ctx.layer, "layer_in")
+        ops.linear(xn, self.w_in, self.b_in, proj, T)
+        m.inner(proj[:, :m.n_in], mid[:, :m.n_inner], ctx, cache, state, writes_cache)
+        f.inner(proj[:, self.ff_row:self.ff_row + f.n_in], mid[:, m.n_inner:], ctx)
+        ops.trace_scope(ctx.layer, "layer_out")
+        ops.linear(mid, self.w_out, None, x, T, residual=True)

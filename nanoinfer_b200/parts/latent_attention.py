@@ -11,7 +11,10 @@ carried into the latent space, every head attends over the same cached rows, and
 the weighted sum of latents (csrc/latent_attention.cu, csrc/linear_heads.cu).  A layer built with
 ``own_kv=False`` has no W_dkv and reads the cache of the layer the schedule names, with its own W_uk,
 W_uv, queries and window.  Rotation: interleaved pairs (2i, 2i+1) of the first ``rot_dims`` values of the
-rotated part, angle = position * rot_base^(-2i / rot_dims).
+rotated part or, with ``rot_layout`` "halves", value i with value i + rot_dims / 2; angle = position *
+rot_base^(-2i / rot_dims).  ``head_gate``: head h's output is multiplied by sigmoid(W_g h)_h, one number per row
+and head; its logits are rows of the down-projections' product (32-bit), and the gate is applied to the head's
+weighted sum of latents.
 """
 from __future__ import annotations
 
@@ -21,14 +24,14 @@ import torch
 
 from ..kernels import ops
 from .base import (INIT_ONE_PLUS_NORMAL, MATRIX, VECTOR, KVCacheSpec, KVCacheView, Mixer, ParamSpec, StepContext,
-                   StepLimits, Workspace, register_mixer)
+                   StepLimits, TwoProducts, Workspace, register_mixer)
 
 
 @register_mixer("latent_attention")
-class LatentAttention(Mixer):
+class LatentAttention(TwoProducts, Mixer):
     def __init__(self, width: int, n_head: int, nope_dim: int, rot_dim: int, v_dim: int, q_rank: int,
                  kv_rank: int, scale: float, eps: float, window: int = 0, rot_base: float = 10000.0,
-                 rot_dims: Optional[int] = None, own_kv: bool = True):
+                 rot_dims: Optional[int] = None, own_kv: bool = True, rot_layout: str = "pairs", head_gate: bool = False):
         rot_dims = rot_dim if rot_dims is None else rot_dims
         for name, v in (("width", width), ("n_head", n_head), ("v_dim", v_dim), ("q_rank", q_rank),
                         ("kv_rank", kv_rank)):
@@ -45,6 +48,14 @@ class LatentAttention(Mixer):
         self.window, self.rot_base, self.rot_dims, self.own_kv = int(window), float(rot_base), int(rot_dims), bool(own_kv)
         self.qk_dim = self.nope_dim + self.rot_dim
         self.latent_dim = self.kv_rank + self.rot_dim
+        if rot_layout not in ("pairs", "halves"):
+            raise ValueError(f"latent_attention: rot_layout {rot_layout!r} is not 'pairs' or 'halves'")
+        self.halves, self.head_gate = rot_layout == "halves", bool(head_gate)
+        #: columns of the down-projections' product: the query latent, the key/value latent and the rotated part (not
+        #: in a layer on another's cache), the gate's logits
+        self.gate_off = self.q_rank + (self.latent_dim if self.own_kv else 0)
+        self.n_in = self.gate_off + (self.n_head if self.head_gate else 0)
+        self.n_inner = self.n_head * self.v_dim
 
     def param_specs(self) -> List[ParamSpec]:
         H = self.n_head
@@ -57,6 +68,8 @@ class LatentAttention(Mixer):
         specs += [ParamSpec("k_up", (H * self.nope_dim, self.kv_rank), MATRIX),
                   ParamSpec("v_up", (H * self.v_dim, self.kv_rank), MATRIX),
                   ParamSpec("out_weight", (self.width, H * self.v_dim), MATRIX)]
+        if self.head_gate:
+            specs.append(ParamSpec("gate_weight", (H, self.width), MATRIX))
         return specs
 
     def kv_spec(self) -> Optional[KVCacheSpec]:
@@ -68,8 +81,14 @@ class LatentAttention(Mixer):
     def prepare(self, dtype, device) -> None:
         super().prepare(dtype, device)
         p, H = self.params, self.n_head
-        # the two down-projections read the same rows: one product
-        self.down = torch.cat([p["q_down"], p["kv_down"]], 0).contiguous() if self.own_kv else p["q_down"]
+        # the down-projections and the gate read the same rows: one product
+        keys = ["q_down"] + (["kv_down"] if self.own_kv else []) + (["gate_weight"] if self.head_gate else [])
+        self.w_in = torch.cat([p[k] for k in keys], 0).contiguous()
+        self.w_out, at = p["out_weight"], 0
+        for k in keys:
+            n = p[k].shape[0]
+            p[k] = self.w_in[at:at + n]
+            at += n
         # W_uk per head, transposed: the map from a head's unrotated query into the latent space
         self.k_up_t = p["k_up"].view(H, self.nope_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.v_up = p["v_up"].view(H, self.v_dim, self.kv_rank)
@@ -78,29 +97,30 @@ class LatentAttention(Mixer):
 
     def reserve(self, workspace: Workspace, limits: StepLimits) -> None:
         n, H = limits.max_rows, self.n_head
-        workspace.reserve("latent.proj", n * (self.q_rank + self.latent_dim), torch.float32)
+        self.reserve_products(workspace, limits)
         workspace.reserve("latent.cq", n * self.q_rank, self.dtype)
         workspace.reserve("latent.q", n * H * self.qk_dim, self.dtype)
         workspace.reserve("latent.q_full", n * H * self.latent_dim, torch.float32)
         workspace.reserve("latent.out", n * H * self.kv_rank, self.dtype)
-        workspace.reserve("latent.att", n * H * self.v_dim, self.dtype)
         ops.latent_attention_reserve(workspace, H, self.kv_rank)
 
     def forward(self, xn: torch.Tensor, x: torch.Tensor, ctx: StepContext, cache: Optional[KVCacheView],
                 state: Optional[torch.Tensor], writes_cache: bool = True) -> None:
+        self.run_alone(xn, x, ctx, cache, state, writes_cache, names=("latent_down", "attn_proj"))
+
+    def inner(self, proj: torch.Tensor, out: torch.Tensor, ctx: StepContext, cache: Optional[KVCacheView] = None,
+              state: Optional[torch.Tensor] = None, writes_cache: bool = True) -> None:
         if cache is None:
             raise ValueError("latent_attention needs a paged latent cache")
         if writes_cache != self.own_kv:
             raise ValueError("latent_attention: a layer without W_dkv must read another layer's cache, and only it")
         T, p, H, ws, n = ctx.n_rows, self.params, self.n_head, ctx.workspace, ctx.max_rows
         D = self.latent_dim
-        proj = ws.get("latent.proj", (n, self.down.shape[0]), torch.float32)
-        ops.trace_scope(ctx.layer, "latent_down")
-        ops.linear(xn, self.down, None, proj, T)
         cq = ws.get("latent.cq", (n, self.q_rank), self.dtype)
         ops.latent_prep(proj, self.q_rank, self.kv_rank, self.rot_dim, self.rot_dims, self.freqs, p["q_norm"],
                         p.get("kv_norm"), self.eps, cq, cache.layer if self.own_kv else None,
-                        cache.block_table if self.own_kv else None, ctx.row_entry, ctx.positions, T, ctx.status)
+                        cache.block_table if self.own_kv else None, ctx.row_entry, ctx.positions, T, ctx.status,
+                        halves=self.halves)
         q = ws.get("latent.q", (n, H * self.qk_dim), self.dtype)
         ops.trace_scope(ctx.layer, "q_up")
         ops.linear(cq, p["q_up"], None, q, T)
@@ -108,11 +128,10 @@ class LatentAttention(Mixer):
         if self.nope_dim:
             ops.trace_scope(ctx.layer, "q_absorb")
             ops.linear_heads(q, self.qk_dim, self.k_up_t, qf.view(n, H * D), D, T)
-        ops.rope_heads(q, self.nope_dim, self.rot_dim, self.rot_dims, self.freqs, ctx.positions, qf, self.kv_rank, H, T)
+        ops.rope_heads(q, self.nope_dim, self.rot_dim, self.rot_dims, self.freqs, ctx.positions, qf, self.kv_rank, H, T,
+                       halves=self.halves)
         lat = ws.get("latent.out", (n, H * self.kv_rank), self.dtype)
-        ops.latent_attention(qf, cache.layer, lat, cache.block_table, ctx, H, self.kv_rank, self.scale, self.window)
-        att = ws.get("latent.att", (n, H * self.v_dim), self.dtype)
+        ops.latent_attention(qf, cache.layer, lat, cache.block_table, ctx, H, self.kv_rank, self.scale, self.window,
+                             gate=proj[:, self.gate_off:self.gate_off + H] if self.head_gate else None)
         ops.trace_scope(ctx.layer, "v_up")
-        ops.linear_heads(lat, self.kv_rank, self.v_up, att, self.v_dim, T)
-        ops.trace_scope(ctx.layer, "attn_proj")
-        ops.linear(att, p["out_weight"], None, x, T, residual=True)
+        ops.linear_heads(lat, self.kv_rank, self.v_up, out, self.v_dim, T)

@@ -12,7 +12,7 @@ from typing import List
 import torch
 
 from ..kernels import ops
-from .base import MATRIX, TABLE, VECTOR, FeedForward, ParamSpec, StepContext, register_feed_forward
+from .base import MATRIX, TABLE, VECTOR, FeedForward, ParamSpec, StepContext, TwoProducts, register_feed_forward
 
 
 @register_feed_forward("dense_mlp")
@@ -52,7 +52,7 @@ class DenseMLP(FeedForward):
 
 
 @register_feed_forward("gated_mlp")
-class GatedMLP(FeedForward):
+class GatedMLP(TwoProducts, FeedForward):
     """The gated dense feed-forward: x += W_down (act(W_gate h) * (W_up h)), without biases; ``activation`` is
     "silu" (z * sigmoid(z)) or one of the dense feed-forward's.  Gate and value rows are interleaved into one
     matrix at load ([2F, C]: row 2f the gate's, row 2f + 1 the value's), so that one product makes both as 32-bit
@@ -63,36 +63,31 @@ class GatedMLP(FeedForward):
             raise ValueError(f"gated_mlp: activation {activation!r} is not one of 'silu', 'tanh', 'erf', 'relu2'")
         if width <= 0 or inner <= 0:
             raise ValueError("gated_mlp: sizes must be positive")
-        self.width, self.inner, self.activation = int(width), int(inner), activation
+        self.width, self.n_inner, self.activation = int(width), int(inner), activation
+        self.n_in = 2 * self.n_inner
 
     def param_specs(self) -> List[ParamSpec]:
-        return [ParamSpec("gate_weight", (self.inner, self.width), MATRIX),
-                ParamSpec("up_weight", (self.inner, self.width), MATRIX),
-                ParamSpec("down_weight", (self.width, self.inner), MATRIX)]
+        return [ParamSpec("gate_weight", (self.n_inner, self.width), MATRIX),
+                ParamSpec("up_weight", (self.n_inner, self.width), MATRIX),
+                ParamSpec("down_weight", (self.width, self.n_inner), MATRIX)]
 
     def prepare(self, dtype, device) -> None:
         super().prepare(dtype, device)
         p = self.params
-        w = torch.empty(self.inner, 2, self.width, dtype=p["gate_weight"].dtype, device=p["gate_weight"].device)
+        w = torch.empty(self.n_inner, 2, self.width, dtype=p["gate_weight"].dtype, device=p["gate_weight"].device)
         w[:, 0], w[:, 1] = p["gate_weight"], p["up_weight"]
         p["gate_weight"], p["up_weight"] = w[:, 0], w[:, 1]
-        self.w_in = w.view(2 * self.inner, self.width)
+        self.w_in, self.w_out = w.view(2 * self.n_inner, self.width), p["down_weight"]
 
     def reserve(self, workspace, limits) -> None:
-        workspace.reserve("gated_mlp.pre", limits.max_rows * 2 * self.inner, torch.float32)
-        workspace.reserve("mlp.fc", limits.max_rows * self.inner, self.dtype)
+        self.reserve_products(workspace, limits)
 
     def forward(self, xn: torch.Tensor, x: torch.Tensor, ctx: StepContext) -> None:
-        if isinstance(xn, ops.NormInput):
-            xn = xn.materialise(ctx.n_rows)
-        T, ws = ctx.n_rows, ctx.workspace
-        pre = ws.get("gated_mlp.pre", (ctx.max_rows, 2 * self.inner), torch.float32)
-        ops.trace_scope(ctx.layer, "fc")
-        ops.linear(xn, self.w_in, None, pre, T)
-        fc = ws.get("mlp.fc", (ctx.max_rows, self.inner), self.dtype)
-        ops.glu(pre, fc, T, self.inner, ops.ACT_CODES[self.activation])
-        ops.trace_scope(ctx.layer, "fc_proj")
-        ops.linear(fc, self.params["down_weight"], None, x, T, residual=True)
+        self.run_alone(xn, x, ctx, names=("fc", "fc_proj"))
+
+    def inner(self, proj: torch.Tensor, out: torch.Tensor, ctx: StepContext, cache=None, state=None,
+              writes_cache: bool = True) -> None:
+        ops.glu(proj, out, ctx.n_rows, self.n_inner, ops.ACT_CODES[self.activation])
 
 
 @register_feed_forward("token_gated_input")

@@ -79,3 +79,24 @@ class ScalarRMSNorm(RMSNorm):
         if w.numel() == 1:
             self.scalar = w.reshape(())
             self.params["weight"] = w.reshape(1).expand(self.width).contiguous()
+
+
+@register_norm("grouped_rmsnorm")
+class GroupedRMSNorm(Norm):
+    """An RMS norm in groups: the vector is cut into ``groups`` equal consecutive parts, each part is divided by its own
+    sqrt(mean(part^2) + eps), and the whole is multiplied by one weight of the vector's size; statistics in 32-bit.  One
+    group is the plain RMS norm.  ``add`` (a 32-bit vector) is added to the stream first, in the same kernel."""
+
+    takes_vector = True
+
+    def __init__(self, width: int, eps: float, groups: int = 1):
+        if groups <= 0 or width % groups:
+            raise ValueError(f"grouped_rmsnorm: {groups} groups do not divide a width of {width}")
+        self.width, self.eps, self.groups = int(width), float(eps), int(groups)
+
+    def param_specs(self) -> List[ParamSpec]:
+        return [ParamSpec("weight", (self.width,), VECTOR, INIT_ONE_PLUS_NORMAL)]
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, n_rows: int, rows: Optional[torch.Tensor] = None,
+                add: Optional[torch.Tensor] = None) -> None:
+        ops.group_norm(x, self.params["weight"], self.groups, self.eps, out, n_rows, rows, add)

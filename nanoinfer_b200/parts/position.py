@@ -3,6 +3,7 @@
 context (crates/core/src/stages/mod.rs:516-519)."""
 from __future__ import annotations
 
+import math
 from typing import List, Optional
 
 import torch
@@ -79,6 +80,48 @@ class SinusoidalPositions(PositionEncoding):
 class RotaryHalves(RotaryPairs):
     """Rotary positions in the halves layout: of every query and key head the first ``dims`` values turn, value i
     paired with value i + dims / 2, by the angle position * base^(-2i / dims); the other values pass.  The rotation is
-    done by the mixer's own kernel (``kernels.ops.wide_norm_rope_append``, ``kernels.ops.rope_halves``)."""
+    done by the mixer's own kernel (``kernels.ops.wide_norm_rope_append``, ``kernels.ops.rope_halves``,
+    ``kernels.ops.norm_rope_maps_append``).
+
+    ``scaling`` (YaRN: factor, original, fast, slow) stretches the wavelengths for sequences longer than the ``original``
+    length: with index(t) the index whose wave turns t times in that length, frequencies below lo =
+    max(floor(index(fast)), 0) stay, those above hi = min(ceil(index(slow)), dims - 1) are divided by ``factor``, in
+    between a ramp over the indices mixes the two; cosine and sine are multiplied by ``amplitude`` = 0.1 ln(factor) + 1
+    (mixers whose kernel takes no amplitude refuse a scaled encoding)."""
 
     layout = "halves"
+
+    def __init__(self, base: float, dims: int, scaling: Optional[dict] = None):
+        super().__init__(base, dims)
+        #: what cosine and sine are multiplied by
+        self.amplitude = 1.0
+        self.scaling = dict(scaling) if scaling else None
+        if self.scaling is not None:
+            missing = {"factor", "original", "fast", "slow"} - set(self.scaling)
+            if missing or not all(float(self.scaling[k]) > 0.0 for k in ("factor", "original", "fast", "slow")):
+                raise ValueError("rotary_halves: scaling needs positive factor, original, fast and slow")
+            self.amplitude = 0.1 * math.log(float(self.scaling["factor"])) + 1.0
+
+    def frequencies(self) -> List[float]:
+        """The ``dims`` / 2 frequencies in double precision."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        sc = self.scaling
+        if sc is None:
+            return f
+
+        def index(turns: float) -> float:
+            # base^(-2i/dims) * original = 2 pi turns, solved for i
+            return self.dims * math.log(float(sc["original"]) / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+
+        lo = max(math.floor(index(float(sc["fast"]))), 0)
+        hi = min(math.ceil(index(float(sc["slow"]))), self.dims - 1)
+        out = []
+        for i, fi in enumerate(f):
+            ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            out.append(fi / float(sc["factor"]) * ramp + fi * (1.0 - ramp))
+        return out
+
+    def prepare(self, dtype, device) -> None:
+        PositionEncoding.prepare(self, dtype, device)
+        if self.dims:
+            self.freqs = torch.tensor(self.frequencies(), dtype=torch.float64, device=device)

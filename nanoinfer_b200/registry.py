@@ -91,5 +91,10 @@ def _register_builtin() -> None:
 
     register_architecture("Nagilix", NagilixConfig, build_nagilix_spec)
 
+    from .config.dedunex import DedunexConfig
+    from .models.dedunex import build_dedunex_spec
+
+    register_architecture("Dedunex", DedunexConfig, build_dedunex_spec)
+
 
 _register_builtin()

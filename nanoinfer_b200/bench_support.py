@@ -503,6 +503,25 @@ def nagilix_like(width: int, n_layer: int, vocab: int, context: int, span: int =
                 logit_scale=1.0, layers=layers)
 
 
+def dedunex_like(width: int, n_layer: int, vocab: int, window: int = 512) -> dict:
+    """A Dedunex configuration whose layers have the sizes of a GPT-2 of ``width`` (a gated feed-forward of 8/3 x width
+    beside every mixer): by turns attention through a latent of 256 + 32 (heads of 64), differential attention (heads of
+    two maps of 64 and values of 128, a key/value head for about two query heads, capped scores, a window, half of a map
+    turned with scaled wavelengths), a minimal gated recurrent unit of the model's width, and differential attention
+    again; two norm groups; the stack runs once, with its vector."""
+    heads = width // 128
+    kv_heads = max(d for d in range(1, max(1, heads // 2) + 1) if heads % d == 0)
+    att = dict(heads=heads, kv_heads=kv_heads, dim=64, vdim=128, scale=0.125, softcap=50.0, diff=0.5, mask=dict(size=window),
+               rot=dict(dims=32, base=10000.0, scaling=dict(factor=4.0, original=1024, fast=32.0, slow=1.0)))
+    lat = dict(heads=width // 64, dim=64, rot_dim=32, vdim=64, q_rank=width // 2, kv_rank=256, scale=96 ** -0.5,
+               rot=dict(base=10000.0, dims=32))
+    dense = dict(kind="dense", ff=-(-(8 * width // 3) // 64) * 64)
+    kinds = (("latent_attention", lat), ("attention", att), ("mingru", dict(width=width)), ("attention", att))
+    layers = [dict(type=kinds[i % 4][0], mixer=json.loads(json.dumps(kinds[i % 4][1])), mlp=dict(dense)) for i in range(n_layer)]
+    return dict(architecture="Dedunex", vocab=vocab, width=width, norm=dict(eps=1e-6, groups=2),
+                loop=dict(start=0, stop=n_layer, times=1), layers=layers)
+
+
 def folder_of(raw: dict, seed: int, dtype: torch.dtype) -> str:
     """A folder with seeded random weights of the configuration ``raw`` (made once, in the temporary folder)."""
     from .config.base import architecture_name
@@ -558,7 +577,7 @@ def profile_forward(eng, prompt, batch: int, repeats: int = 3):
 
 def compare_designs(widths=(768, 1024, 1600), n_layer: int = 4, batch: int = 8, context: int = 1024,
                     steps: int = 64, warmup: int = 8, designs=("vadonex", "gpt2")) -> List[dict]:
-    """The ``designs`` (of "nagilix", "kemuzen", "mulavik", "vadonex", "gpt2") side by side at equal width, depth, vocabulary and
+    """The ``designs`` (of "dedunex", "nagilix", "kemuzen", "mulavik", "vadonex", "gpt2") side by side at equal width, depth, vocabulary and
     context (random weights, bfloat16): one prompt of ``context - steps - warmup`` tokens in one step, decode at
     ``batch``, and where the time of each goes op by op with every op's fraction of its roofline (measured
     peaks)."""
@@ -571,7 +590,8 @@ def compare_designs(widths=(768, 1024, 1600), n_layer: int = 4, batch: int = 8, 
         made = {"vadonex": lambda: vadonex_like(width, n_layer, 50257, context), "gpt2": lambda: gpt2,
                 "mulavik": lambda: mulavik_like(width, n_layer, 50257),
                 "kemuzen": lambda: kemuzen_like(width, n_layer, 50257),
-                "nagilix": lambda: nagilix_like(width, n_layer, 50257, context)}
+                "nagilix": lambda: nagilix_like(width, n_layer, 50257, context),
+                "dedunex": lambda: dedunex_like(width, n_layer, 50257)}
         for name in designs:
             raw = made[name]()
             d = folder_of(raw, 1234, torch.bfloat16)

@@ -1158,7 +1158,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
         keys = sum(min(p + 1, window) if window > 0 else p + 1
                    for e, p0 in enumerate(ctx.host_entry_pos0)
                    for p in range(p0, p0 + ctx.host_entry_start[e + 1] - ctx.host_entry_start[e]))
-        _note("attn", "attn", (ctx.n_rows, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
+        _note("attn", "latent_attn", (ctx.n_rows, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
               4.0 * ctx.n_rows * n_head * D + out.element_size() * (ctx.n_rows * n_head * kv_rank + keys * D))
     _check(library().nib_latent_attention(_dt(cache), _ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
                                           block_table.shape[1], None, _ptr(ctx.row_entry), _ptr(ctx.positions),

@@ -211,17 +211,37 @@ int nib_latent_prep(int dtype, const float* proj, int ld, int q_rank, int kv_ran
                     void* cache, const int* block_table, int max_blocks, const int* row_entry,
                     const int* positions, int T, int page_size, int n_pages, int has_kv, int halves, int* status,
                     cudaStream_t stream);
-int nib_rope_heads(int dtype, const void* q, int ldq, int nope, int rot_dim, int rot_dims, const double* freqs,
-                   const int* positions, float* out, int out_dim, int out_off, int n_head, int T, int halves,
+int nib_rope_heads(int dtype, int out_dtype, const void* q, int ldq, int nope, int rot_dim, int rot_dims,
+                   const double* freqs, const int* positions, void* out, int out_dim, int out_off, int n_head, int T, int halves,
                    cudaStream_t stream);
-int nib_latent_attention(int dtype, const float* q, const void* cache, void* out, int ldo, const int* block_table,
+int nib_latent_attention(int dtype, int q_dtype, const void* q, const void* cache, void* out, int ldo, const int* block_table,
                          int max_blocks, const int* rows, const int* row_entry, const int* positions, int n_rows,
                          int n_head, int kv_rank, int D, int page_size, int n_pages, float scale, int window,
                          const float* gate, int ldg, int* status, int n_splits, float* partials, cudaStream_t stream);
 
-// ---- a product per head (linear_heads.cu): out[t, h, :N] = a[t, h, :K] . w[h]^T, w [n_head, N, K]
+// The same attention in bfloat16 (queries too) on the tensor cores: prompt portions in tiles of 128 rows on tcgen05
+// (latent_prefill_tc.cu), single tokens on warp-level MMAs with sixteen heads a tile and a row's pieces of keys as one
+// cluster (latent_decode_mma.cu; n_splits 1, 2, 4, 8 or 16).
+int nib_latent_prefill_tc_supported(int kv_rank, int D, int page_size);
+int nib_latent_prefill_tc(const void* q, int T, const void* cache, void* out, int ldo, const int* block_table,
+                          int max_blocks, const int* tiles, int n_tiles, const int* entry_start, const int* entry_pos0,
+                          int n_head, int kv_rank, int D, int page_size, int n_pages, float scale, int window,
+                          const float* gate, int ldg, int* status, cudaStream_t stream);
+int nib_latent_decode_mma_supported(int kv_rank, int D);
+int nib_latent_decode_mma(const void* q, const void* cache, void* out, int ldo, const int* block_table, int max_blocks,
+                          const int* rows, const int* row_entry, const int* positions, int n_rows, int n_head, int kv_rank,
+                          int D, int page_size, int n_pages, float scale, int window, const float* gate, int ldg,
+                          int* status, int n_splits, cudaStream_t stream);
+
+// ---- a product per head (linear_heads.cu; in bfloat16 on warp-level MMAs: linear_heads_mma.cu): out[t, h, :N] = a[t, h, :K] . w[h]^T, w [n_head, N, K]
 int nib_linear_heads(int dtype, int out_dtype, const void* a, int lda, int a_head_stride, const void* w, void* out,
                      int ldo, int out_head_stride, int M, int n_head, int N, int K, cudaStream_t stream);
+
+int nib_linear_heads_mma_supported(const void* a, int lda, int a_head_stride, const void* w, int K);
+// rot_dim > 0: a's heads are [K | rot_dim], out's [N | rot_dim]; the rotated part turned by the row's position goes with it.
+int nib_linear_heads_mma(int out_dtype, const void* a, int lda, int a_head_stride, const void* w, void* out, int ldo,
+                         int out_head_stride, int M, int n_head, int N, int K, const int* positions, const double* freqs,
+                         int rot_dim, int rot_dims, int halves, cudaStream_t stream);
 
 // ---- the generalised delta rule (delta_rule.cu)
 int nib_delta_rule(int dtype, float* proj, int ld, int r_off, int k_off, int v_off, int g_off, int a_off,

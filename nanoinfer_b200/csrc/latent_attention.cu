@@ -11,7 +11,8 @@
 //   latent_prep      : from the down-projections' output [c_q raw | c raw | k_rot raw] of a row:
 //                      c_q = rmsnorm(.) * w_q  -> the up-projection's input;
 //                      c = rmsnorm(.) * w_kv and k_rot rotated -> the row's slot of the paged latent cache
-//   rope_heads       : rotates the rot part of every head's query and writes it behind the absorbed part
+//   rope_heads       : rotates the rot part of every head's query and writes it behind the absorbed part (where
+//                      linear_heads_mma.cu does not do it with the product)
 //   latent_attention : softmax attention of rows over the cache, causal, with an optional window
 //                      (position i sees j with 0 <= i - j < window)
 // Rotation: pairs (2i, 2i+1) of the first rot_dims values or, with `halves`, value i with value i + rot_dims / 2;
@@ -65,12 +66,12 @@ latent_prep_kernel(const float* proj, int ld, int q_rank, int kv_rank, int rot_d
   for (int c = rot_dims + threadIdx.x; c < rot_dim; c += blockDim.x) dst[kv_rank + c] = from_float<T>(kr[c]);
 }
 
-// q: [T, H * (nope + rot_dim)] as the up-projection leaves it; out: float [T, H, out_dim], the rot part of
-// head h goes to out[t, h, out_off ...].
-template <typename T>
+// q: [T, H * (nope + rot_dim)] as the up-projection leaves it; out: [T, H, out_dim], the rot part of head h goes to
+// out[t, h, out_off ...].
+template <typename T, typename TO>
 __global__ void __launch_bounds__(128)
 rope_heads_kernel(const T* q, int ldq, int nope, int rot_dim, int rot_dims, const double* __restrict__ freqs,
-                  const int* __restrict__ positions, float* out, int out_dim, int out_off, int n_head, int halves) {
+                  const int* __restrict__ positions, TO* out, int out_dim, int out_off, int n_head, int halves) {
   pdl_trigger();
   extern __shared__ float cs[];   // cos, sin per pair
   const int t = blockIdx.x, half = rot_dims / 2;
@@ -87,15 +88,15 @@ rope_heads_kernel(const T* q, int ldq, int nope, int rot_dim, int rot_dims, cons
   for (int w = threadIdx.x; w < n_head * per_head; w += blockDim.x) {
     const int h = w / per_head, i = w % per_head;
     const T* src = q + (size_t)t * ldq + (size_t)h * (nope + rot_dim) + nope;
-    float* dst = out + ((size_t)t * n_head + h) * out_dim + out_off;
+    TO* dst = out + ((size_t)t * n_head + h) * out_dim + out_off;
     if (i < half) {
       const int iu = halves ? i : 2 * i, iv = halves ? i + half : 2 * i + 1;
       const float u = to_float(src[iu]), v = to_float(src[iv]), c = cs[2 * i], s = cs[2 * i + 1];
-      dst[iu] = u * c - v * s;
-      dst[iv] = v * c + u * s;
+      dst[iu] = from_float<TO>(u * c - v * s);
+      dst[iv] = from_float<TO>(v * c + u * s);
     } else {
       const int d = rot_dims + (i - half);
-      dst[d] = to_float(src[d]);
+      dst[d] = from_float<TO>(to_float(src[d]));
     }
   }
 }
@@ -107,9 +108,9 @@ constexpr int LA_TILE = 32;     // keys a tile, one a lane
 // floats (row stride odd: a lane reads its own key's row without bank conflicts), lane j of a warp makes
 // the score of key j for the warp's head, the tile's maximum and sum come from warp reductions, and for
 // the weighted sum lane l owns the latent's elements l, l + 32, ...
-template <typename T, int NACC>
+template <typename T, typename TQ, int NACC>
 __global__ void __launch_bounds__(LA_WARPS * 32)
-latent_attention_kernel(const float* q, const T* cache, T* out, int ldo, const int* __restrict__ block_table,
+latent_attention_kernel(const TQ* q, const T* cache, T* out, int ldo, const int* __restrict__ block_table,
                         int max_blocks, const int* __restrict__ rows, const int* __restrict__ row_entry,
                         const int* __restrict__ positions, int n_head, int kv_rank, int D, int page_size,
                         int n_pages, float scale, int window, const float* gate, int ldg, int* status, int n_splits, float* partials) {
@@ -136,8 +137,8 @@ latent_attention_kernel(const float* q, const T* cache, T* out, int ldo, const i
   }
   pdl_wait();
   if (live) {
-    const float* src = q + ((size_t)t * n_head + h) * D;
-    for (int d = lane; d < D; d += 32) qs[warp * D + d] = src[d];
+    const TQ* src = q + ((size_t)t * n_head + h) * D;
+    for (int d = lane; d < D; d += 32) qs[warp * D + d] = to_float(src[d]);
   }
   float m = -INFINITY, l = 0.0f, acc[NACC];
 #pragma unroll
@@ -250,8 +251,8 @@ latent_merge_kernel(const float* partials, T* out, int ldo, const int* __restric
   }
 }
 
-template <typename T, int NACC>
-static int launch_latent_attention(const float* q, const T* cache, T* out, int ldo, const int* block_table,
+template <typename T, typename TQ, int NACC>
+static int launch_latent_attention(const TQ* q, const T* cache, T* out, int ldo, const int* block_table,
                                    int max_blocks, const int* rows, const int* row_entry, const int* positions,
                                    int n_rows, int n_head, int kv_rank, int D, int page_size, int n_pages,
                                    float scale, int window, const float* gate, int ldg, int* status, int n_splits,
@@ -259,8 +260,8 @@ static int launch_latent_attention(const float* q, const T* cache, T* out, int l
   const size_t smem = ((size_t)LA_TILE * (D | 1) + (size_t)LA_WARPS * D) * sizeof(float);
   if (smem > 200 * 1024) return NIB_ERR_UNSUPPORTED_SIZE;
   if (smem > 48 * 1024)
-    cudaFuncSetAttribute(latent_attention_kernel<T, NACC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  launch_pdl(latent_attention_kernel<T, NACC>, dim3(n_rows, (n_head + LA_WARPS - 1) / LA_WARPS, n_splits),
+    cudaFuncSetAttribute(latent_attention_kernel<T, TQ, NACC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  launch_pdl(latent_attention_kernel<T, TQ, NACC>, dim3(n_rows, (n_head + LA_WARPS - 1) / LA_WARPS, n_splits),
              dim3(LA_WARPS * 32), smem, stream, q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
              n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status, n_splits, partials);
   if (n_splits > 1)
@@ -269,14 +270,14 @@ static int launch_latent_attention(const float* q, const T* cache, T* out, int l
   NIB_LAUNCH_CHECK();
 }
 
-template <typename T>
-static int pick_latent_attention(const float* q, const void* cache, void* out, int ldo, const int* block_table,
+template <typename T, typename TQ>
+static int pick_latent_attention(const void* q, const void* cache, void* out, int ldo, const int* block_table,
                                  int max_blocks, const int* rows, const int* row_entry, const int* positions,
                                  int n_rows, int n_head, int kv_rank, int D, int page_size, int n_pages,
                                  float scale, int window, const float* gate, int ldg, int* status, int n_splits,
                                  float* partials, cudaStream_t stream) {
 #define NIB_LA(N)                                                                                              \
-  return launch_latent_attention<T, N>(q, (const T*)cache, (T*)out, ldo, block_table, max_blocks, rows,       \
+  return launch_latent_attention<T, TQ, N>((const TQ*)q, (const T*)cache, (T*)out, ldo, block_table, max_blocks, rows,       \
                                        row_entry, positions, n_rows, n_head, kv_rank, D, page_size, n_pages,  \
                                        scale, window, gate, ldg, status, n_splits, partials, stream)
   const int n = (kv_rank + 31) / 32;
@@ -314,28 +315,31 @@ extern "C" int nib_latent_prep(int dtype, const float* proj, int ld, int q_rank,
   NIB_LAUNCH_CHECK();
 }
 
-extern "C" int nib_rope_heads(int dtype, const void* q, int ldq, int nope, int rot_dim, int rot_dims,
-                              const double* freqs, const int* positions, float* out, int out_dim, int out_off,
+extern "C" int nib_rope_heads(int dtype, int out_dtype, const void* q, int ldq, int nope, int rot_dim, int rot_dims,
+                              const double* freqs, const int* positions, void* out, int out_dim, int out_off,
                               int n_head, int T, int halves, cudaStream_t stream) {
   if (T <= 0 || rot_dim <= 0) return 0;
   if (rot_dims > rot_dim || (rot_dims & 1)) return NIB_ERR_BAD_ARGUMENT;
   const size_t smem = (size_t)(rot_dims + 2) * sizeof(float);
-  if (dtype == DT_F32)
-    launch_pdl(rope_heads_kernel<float>, dim3(T), dim3(128), smem, stream, (const float*)q, ldq, nope, rot_dim,
-               rot_dims, freqs, positions, out, out_dim, out_off, n_head, halves);
-  else if (dtype == DT_BF16)
-    launch_pdl(rope_heads_kernel<bf16>, dim3(T), dim3(128), smem, stream, (const bf16*)q, ldq, nope, rot_dim,
-               rot_dims, freqs, positions, out, out_dim, out_off, n_head, halves);
+  if (dtype == DT_F32 && out_dtype == DT_F32)
+    launch_pdl(rope_heads_kernel<float, float>, dim3(T), dim3(128), smem, stream, (const float*)q, ldq, nope, rot_dim,
+               rot_dims, freqs, positions, (float*)out, out_dim, out_off, n_head, halves);
+  else if (dtype == DT_BF16 && out_dtype == DT_F32)
+    launch_pdl(rope_heads_kernel<bf16, float>, dim3(T), dim3(128), smem, stream, (const bf16*)q, ldq, nope, rot_dim,
+               rot_dims, freqs, positions, (float*)out, out_dim, out_off, n_head, halves);
+  else if (dtype == DT_BF16 && out_dtype == DT_BF16)
+    launch_pdl(rope_heads_kernel<bf16, bf16>, dim3(T), dim3(128), smem, stream, (const bf16*)q, ldq, nope, rot_dim,
+               rot_dims, freqs, positions, (bf16*)out, out_dim, out_off, n_head, halves);
   else
     return NIB_ERR_BAD_ARGUMENT;
   NIB_LAUNCH_CHECK();
 }
 
-// q: float [T, n_head, D] (absorbed part, then the rotated part), D = kv_rank + rot_dim; cache: one layer
+// q: [T, n_head, D] (absorbed part, then the rotated part) in 32-bit or in the cache's dtype, D = kv_rank + rot_dim; cache: one layer
 // [n_pages, page_size, D]; out: [T, n_head * kv_rank] in the cache's dtype.  rows: the step's rows to
 // process (nullptr: rows 0..n_rows-1).  n_splits > 1: every row's keys are cut into that many pieces, each a
 // block of its own, and merged through `partials` (n_rows * n_head * n_splits * (kv_rank + 2) floats).
-extern "C" int nib_latent_attention(int dtype, const float* q, const void* cache, void* out, int ldo,
+extern "C" int nib_latent_attention(int dtype, int q_dtype, const void* q, const void* cache, void* out, int ldo,
                                     const int* block_table, int max_blocks, const int* rows, const int* row_entry,
                                     const int* positions, int n_rows, int n_head, int kv_rank, int D,
                                     int page_size, int n_pages, float scale, int window, const float* gate, int ldg,
@@ -343,13 +347,17 @@ extern "C" int nib_latent_attention(int dtype, const float* q, const void* cache
   if (n_rows <= 0) return 0;
   if (kv_rank <= 0 || D < kv_rank || n_head <= 0) return NIB_ERR_BAD_ARGUMENT;
   if (n_splits < 1 || n_splits > 65535 || (n_splits > 1 && partials == nullptr)) return NIB_ERR_BAD_ARGUMENT;
-  if (dtype == DT_F32)
-    return pick_latent_attention<float>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
+  if (dtype == DT_F32 && q_dtype == DT_F32)
+    return pick_latent_attention<float, float>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
                                         n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status,
                                         n_splits, partials, stream);
-  if (dtype == DT_BF16)
-    return pick_latent_attention<bf16>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-                                       n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status,
-                                       n_splits, partials, stream);
+  if (dtype == DT_BF16 && q_dtype == DT_F32)
+    return pick_latent_attention<bf16, float>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
+                                              n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg,
+                                              status, n_splits, partials, stream);
+  if (dtype == DT_BF16 && q_dtype == DT_BF16)
+    return pick_latent_attention<bf16, bf16>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
+                                             n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg,
+                                             status, n_splits, partials, stream);
   return NIB_ERR_BAD_ARGUMENT;
 }

@@ -5,13 +5,14 @@
 // The three logits of a row (biases added) lie at three column offsets of the 32-bit projection; S (one float a channel,
 // zero at a sequence's start) comes from and goes to the request's state slot; all arithmetic is 32-bit.
 //
-// A linear recurrence can be cut in time.  A block owns 32 channels (a lane each) of one entry; its warps take
-// consecutive runs of ROWS rows of a chunk of NW * ROWS rows.  A warp first walks its run from S = 0, keeping the run's
-// gates and candidates in registers, which gives the run's own result b and the fraction f of an incoming state that it
-// forgets (f <- f + z (1 - f), kept as the fraction FORGOTTEN: of a slow channel's remaining fraction, a number next to
-// 1, a float would lose what is forgotten); the runs are then chained through shared memory, S_out = b + S_in - f S_in,
-// and every warp walks its run once more from its true incoming state, in registers, and writes its rows.  A step of
-// single tokens takes the form with one row a warp and no chain.
+// A linear recurrence can be cut in time.  Thirty-two channels of one entry (a lane each) belong to a cluster of up to eight
+// blocks of sixteen warps; a chunk of up to 1024 rows is cut into runs of at most eight rows, a warp each, block after block.
+// A warp first walks its run from S = 0, keeping the run's gates and candidates in registers, which gives the run's own
+// result b and the fraction f of an incoming state that it forgets (f <- f + z (1 - f), kept as the fraction FORGOTTEN: of a
+// slow channel's remaining fraction, a number next to 1, a float would lose what is forgotten).  Runs compose:
+// S_out = b + S_in - f S_in.  A block chains its warps' runs through shared memory, the cluster its blocks' through
+// distributed shared memory, and every warp then walks its run once more, in registers, from its true incoming state and
+// writes its rows.  A step of single tokens takes a form of its own with nothing to chain.
 #include "api.h"
 #include "common.cuh"
 
@@ -19,27 +20,31 @@ namespace nib {
 
 __device__ __forceinline__ float mg_sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
 
-constexpr int MG_WARPS = 16, MG_ROWS = 8;
+constexpr int MG_WARPS = 16, MG_ROWS = 8, MG_MAX_CLUSTER = 8;
 
 template <typename OutT>
 __global__ void __launch_bounds__(MG_WARPS * 32)
 min_gru_kernel(const float* proj, int ld, int z_off, int u_off, int g_off, int width, float* state,
                long long state_stride, const int* __restrict__ entry_start, const int* __restrict__ entry_slot, OutT* out,
-               int ldo) {
+               int ldo, int cluster) {
   pdl_trigger();
   __shared__ float run_b[MG_WARPS][32], run_f[MG_WARPS][32];
+  __shared__ float blk[2][2][32];                   // [chunk parity][b, f][channel] of the whole block's runs
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int e = blockIdx.y, c = blockIdx.x * 32 + lane;
+  const int rank = cluster > 1 ? blockIdx.x % cluster : 0;
+  const int e = blockIdx.y, c = blockIdx.x / cluster * 32 + lane;
   const bool live = c < width;
   const int r_begin = entry_start[e], r_end = entry_start[e + 1];
   pdl_wait();
   float* slot = state + (size_t)entry_slot[e] * state_stride;
-  float carry = live ? slot[c] : 0.0f;              // the state ahead of the chunk, the same in every warp
-  for (int r0 = r_begin; r0 < r_end; r0 += MG_WARPS * MG_ROWS) {
-    // consecutive rows to consecutive warps, and no warp without rows while another has two more
-    const int n = min(MG_WARPS * MG_ROWS, r_end - r0);
-    const int per = (n + MG_WARPS - 1) / MG_WARPS;
-    const int a = r0 + warp * per, rows = max(0, min(per, r0 + n - a));
+  float carry = live ? slot[c] : 0.0f;              // the state ahead of the chunk, the same in every warp of the cluster
+  const int n_runs = cluster * MG_WARPS;
+  int parity = 0;
+  for (int r0 = r_begin; r0 < r_end; r0 += n_runs * MG_ROWS, parity ^= 1) {
+    // consecutive rows to consecutive runs, and no run without rows while another has two more
+    const int n = min(n_runs * MG_ROWS, r_end - r0);
+    const int per = (n + n_runs - 1) / n_runs;
+    const int a = r0 + (rank * MG_WARPS + warp) * per, rows = max(0, min(per, r0 + n - a));
     float z[MG_ROWS], cand[MG_ROWS], g[MG_ROWS];
 #pragma unroll
     for (int i = 0; i < MG_ROWS; ++i) {
@@ -64,12 +69,36 @@ min_gru_kernel(const float* proj, int ld, int z_off, int u_off, int g_off, int w
     run_b[warp][lane] = b;
     run_f[warp][lane] = f;
     __syncthreads();
-    float S = carry;
+    // the block's runs chained: what lies ahead of this warp's run, and the whole block
+    float B = 0.0f, F = 0.0f, Bw = 0.0f, Fw = 0.0f;
 #pragma unroll
     for (int w = 0; w < MG_WARPS; ++w) {
-      if (w == warp) S = carry;
-      carry = run_b[w][lane] + fmaf(-run_f[w][lane], carry, carry);
+      if (w == warp) {
+        Bw = B;
+        Fw = F;
+      }
+      const float rf = run_f[w][lane];
+      B = run_b[w][lane] + fmaf(-rf, B, B);
+      F = fmaf(rf, 1.0f - F, F);
     }
+    float S = carry;                                // the state ahead of this block
+    if (cluster == 1) {
+      carry = B + fmaf(-F, carry, carry);
+    } else {
+      if (warp == 0) {
+        blk[parity][0][lane] = B;
+        blk[parity][1][lane] = F;
+      }
+      cluster_arrive();
+      cluster_wait();
+      for (int k = 0; k < cluster; ++k) {
+        if (k == rank) S = carry;
+        const float kb = __uint_as_float(cluster_load(cluster_addr(&blk[parity][0][lane], k)));
+        const float kf = __uint_as_float(cluster_load(cluster_addr(&blk[parity][1][lane], k)));
+        carry = kb + fmaf(-kf, carry, carry);
+      }
+    }
+    S = Bw + fmaf(-Fw, S, S);                       // ... and ahead of this warp's run
 #pragma unroll
     for (int i = 0; i < MG_ROWS; ++i) {
       if (i < rows && live) {
@@ -78,7 +107,12 @@ min_gru_kernel(const float* proj, int ld, int z_off, int u_off, int g_off, int w
       }
     }
   }
-  if (warp == 0 && live) slot[c] = carry;
+  if (cluster > 1) {                                // nobody leaves while its shared memory is read
+    __syncthreads();
+    cluster_arrive();
+    cluster_wait();
+  }
+  if (rank == 0 && warp == 0 && live) slot[c] = carry;
 }
 
 // Single tokens: entry e is row e; a thread a (row, channel).
@@ -108,8 +142,14 @@ static int launch_min_gru(const float* proj, int ld, int z_off, int u_off, int g
     launch_pdl(min_gru_token_kernel<OutT>, dim3((width + 127) / 128, n_entries), dim3(128), 0, stream, proj, ld, z_off, u_off,
                g_off, width, state, state_stride, entry_slot, out, ldo);
   else
-    launch_pdl(min_gru_kernel<OutT>, dim3((width + 31) / 32, n_entries), dim3(MG_WARPS * 32), 0, stream, proj, ld, z_off,
-               u_off, g_off, width, state, state_stride, entry_start, entry_slot, out, ldo);
+  {
+    // blocks of a cluster: as many as the step's rows can fill (a function of the step's shape alone)
+    int cluster = 1;
+    while (cluster < MG_MAX_CLUSTER && n_rows > cluster * MG_WARPS * MG_ROWS) cluster *= 2;
+    launch_pdl_cluster(min_gru_kernel<OutT>, dim3((width + 31) / 32 * cluster, n_entries), dim3(MG_WARPS * 32), 0, stream,
+                       cluster, proj, ld, z_off, u_off, g_off, width, state, state_stride, entry_start, entry_slot, out, ldo,
+                       cluster);
+  }
   NIB_LAUNCH_CHECK();
 }
 

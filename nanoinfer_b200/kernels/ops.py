@@ -87,9 +87,9 @@ _SIGNATURES = {
     "nib_latent_prep": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_float,
                         _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                         _c_int, _c_ptr, _c_ptr],
-    "nib_rope_heads": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
+    "nib_rope_heads": [_c_int, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
                        _c_int, _c_int, _c_int, _c_ptr],
-    "nib_latent_attention": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int,
+    "nib_latent_attention": [_c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int,
                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr,
                              _c_ptr],
     "nib_linear_heads": [_c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
@@ -142,6 +142,15 @@ _SIGNATURES = {
     "nib_selective_scan": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
                            _c_ptr, _c_ptr, ctypes.c_longlong, ctypes.c_longlong, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
                            _c_ptr, _c_int, _c_ptr],
+    "nib_latent_prefill_tc_supported": [_c_int, _c_int, _c_int],
+    "nib_latent_prefill_tc": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int,
+                              _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr],
+    "nib_latent_decode_mma_supported": [_c_int, _c_int],
+    "nib_latent_decode_mma": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
+                              _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr],
+    "nib_linear_heads_mma_supported": [_c_ptr, _c_int, _c_int, _c_ptr, _c_int],
+    "nib_linear_heads_mma": [_c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                             _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
     "nib_group_norm": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_ptr],
     "nib_embed_group_norm": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float,
                              _c_ptr],
@@ -200,7 +209,8 @@ class _Library:
         counted = name not in ("nib_linear_tc_supported", "nib_linear_tc_pair_supported", "nib_linear_skinny_supported",
                                "nib_attention_prefill_tc_supported", "nib_attention_prefill_supported",
                                "nib_attention_decode_mma_supported", "nib_attention_decode_mma_clusters",
-                               "nib_gated_scan_padded")
+                               "nib_gated_scan_padded", "nib_latent_prefill_tc_supported",
+                               "nib_latent_decode_mma_supported", "nib_linear_heads_mma_supported")
 
         def call(*args):
             global _pending_op
@@ -1105,14 +1115,14 @@ def latent_prep(proj: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, rot
 def rope_heads(q: torch.Tensor, nope: int, rot_dim: int, rot_dims: int, freqs: torch.Tensor,
                positions: torch.Tensor, out: torch.Tensor, out_off: int, n_head: int, T: int, halves: bool = False) -> None:
     """Rotates the last ``rot_dim`` values of every head of q ([T, n_head * (nope + rot_dim)]) by the rows'
-    positions (interleaved pairs over the first ``rot_dims``, or halves) into out[t, h, out_off:], float32 [T, n_head, D]."""
-    _f32(out, "rope_heads: out")
-    if q.stride(1) != 1 or freqs.dtype != torch.float64:
-        raise KernelError("rope_heads: q rows contiguous, freqs float64")
+    positions (interleaved pairs over the first ``rot_dims``, or halves) into out[t, h, out_off:], [T, n_head, D] in
+    float32 or q's dtype."""
+    if q.stride(1) != 1 or freqs.dtype != torch.float64 or not out.is_contiguous():
+        raise KernelError("rope_heads: q rows contiguous, freqs float64, out contiguous")
     if tracing():
         _note("other", "rope", (T, n_head * rot_dim, 0), 6.0 * T * n_head * rot_dim,
               T * n_head * rot_dim * (q.element_size() + 4))
-    _check(library().nib_rope_heads(_dt(q), _ptr(q), q.stride(0), nope, rot_dim, rot_dims, _ptr(freqs),
+    _check(library().nib_rope_heads(_dt(q), _dt(out), _ptr(q), q.stride(0), nope, rot_dim, rot_dims, _ptr(freqs),
                                     _ptr(positions), _ptr(out), out.shape[2], out_off, n_head, T, int(halves), _stream()),
            "rope_heads")
 
@@ -1135,48 +1145,126 @@ def latent_attention_reserve(workspace, n_head: int, kv_rank: int) -> None:
     workspace.reserve("latent.partials", LATENT_BLOCKS * LATENT_HEADS_PER_BLOCK * (kv_rank + 2), torch.float32)
 
 
+def latent_decode_splits(n_rows: int, n_head: int, max_keys: int) -> int:
+    """Into how many pieces (1, 2, 4, 8 or 16: the blocks of a cluster) the MMA kernel cuts each single token's keys:
+    about two blocks an SM, pieces of at least a tile of 64 keys."""
+    groups = -(-n_head // 16)
+    want = min(LATENT_MAX_SPLITS, LATENT_BLOCKS // max(1, n_rows * groups), -(-max_keys // 64))
+    splits = 1
+    while 2 * splits <= want:
+        splits *= 2
+    return splits
+
+
+def _latent_keys(plan, ctx, window: int, single: bool) -> int:
+    """Keys seen by the step's single tokens, or by its portions' rows (for the trace's counts)."""
+    keys = 0
+    for e, p0 in enumerate(ctx.host_entry_pos0):
+        n = ctx.host_entry_start[e + 1] - ctx.host_entry_start[e]
+        if (n == 1) == single:
+            keys += sum(min(p + 1, window) if window > 0 else p + 1 for p in range(p0, p0 + n))
+    return keys
+
+
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, ctx,
                      n_head: int, kv_rank: int, scale: float, window: int, n_splits: Optional[int] = None,
-                     gate: Optional[torch.Tensor] = None) -> None:
-    """Causal softmax attention of the step's rows over one latent cache layer: q float32 [T, n_head, D] (the
-    absorbed query, then the rotated part), out [T, n_head * kv_rank] the weighted sums of latents.  A step of
+                     gate: Optional[torch.Tensor] = None, plan=None) -> None:
+    """Causal softmax attention of the step's rows over one latent cache layer: q [T, n_head, D] (the absorbed query,
+    then the rotated part) in float32 or the cache's dtype, out [T, n_head * kv_rank] the weighted sums of latents.  A step of
     few rows (decoded tokens) cuts every row's keys into ``n_splits`` pieces, merged by a second kernel.  ``gate``
     (float32 [rows, >= n_head], any row stride): head h's output of row t times sigmoid(gate[t, h])."""
     if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1):
         raise KernelError("latent_attention: the gate must be float32 with contiguous rows")
     n_pages, _, _, page_size, D = cache.shape
+    if q.dtype not in (torch.float32, cache.dtype) or not q.is_contiguous():
+        raise KernelError("latent_attention: q must be contiguous, float32 or of the cache's dtype")
+    if out.dtype != cache.dtype or out.stride(1) != 1 or q.shape[2] != D:
+        raise KernelError("latent_attention: out in the cache's dtype, q [T, heads, D]")
+    gate_args = (_ptr(gate), gate.stride(0) if gate is not None else 0)
+    if plan is not None and q.dtype == torch.bfloat16 and scale > 0 and n_splits is None:
+        # on the tensor cores where the sizes allow; what they do not take goes to the general kernel by lists of rows
+        lib, e = library(), q.element_size()
+        ok = q.data_ptr() % 16 == 0 and cache.data_ptr() % 16 == 0
+        todo = []
+        if plan.n_decode:
+            if tracing():
+                keys = _latent_keys(plan, ctx, window, True)
+                _note("attn", "latent_attn", (plan.n_decode, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
+                      e * (plan.n_decode * n_head * (D + kv_rank) + keys * D))
+            if ok and _can("nib_latent_decode_mma_supported", kv_rank, D):
+                splits = latent_decode_splits(plan.n_decode, n_head, plan.max_decode_keys if window <= 0 else
+                                              min(plan.max_decode_keys, window))
+                _check(lib.nib_latent_decode_mma(_ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
+                                                 block_table.shape[1], _ptr(plan.decode_rows), _ptr(ctx.row_entry),
+                                                 _ptr(ctx.positions), plan.n_decode, n_head, kv_rank, D, page_size, n_pages,
+                                                 float(scale), int(window), *gate_args, _ptr(ctx.status), splits, _stream()),
+                       "latent_decode_mma")
+            else:
+                todo.append((plan.decode_rows, plan.n_decode))
+        if plan.n_prefill_rows:
+            if tracing():
+                keys = _latent_keys(plan, ctx, window, False)
+                _note("attn", "latent_attn", (plan.n_prefill_rows, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
+                      e * (plan.n_prefill_rows * n_head * (D + kv_rank) + plan.prefill_kv_rows * D))
+            if ok and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0 \
+                    and _can("nib_latent_prefill_tc_supported", kv_rank, D, page_size):
+                _check(lib.nib_latent_prefill_tc(_ptr(q), ctx.n_rows, _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
+                                                 block_table.shape[1], _ptr(plan.wide_tiles), plan.n_wide_tiles,
+                                                 _ptr(ctx.entry_start), _ptr(ctx.entry_pos0), n_head, kv_rank, D, page_size,
+                                                 n_pages, float(scale), int(window), *gate_args, _ptr(ctx.status), _stream()),
+                       "latent_prefill_tc")
+            else:
+                # (portions alone: all of the step's rows, those of no request among them, which the kernel leaves out)
+                todo.append((plan.prefill_rows, plan.n_prefill_rows if plan.n_decode else ctx.n_rows))
+        for rows, n in todo:
+            _check(lib.nib_latent_attention(_dt(cache), _dt(q), _ptr(q), _ptr(cache), _ptr(out), out.stride(0),
+                                            _ptr(block_table), block_table.shape[1], _ptr(rows), _ptr(ctx.row_entry),
+                                            _ptr(ctx.positions), n, n_head, kv_rank, D, page_size, n_pages, float(scale),
+                                            int(window), *gate_args, _ptr(ctx.status), 1, None, _stream()), "latent_attention")
+        return
     if n_splits is None:
         n_splits = latent_splits(ctx.n_rows, n_head)
     partials = None
     if n_splits > 1:
         need = ctx.n_rows * n_head * n_splits * (kv_rank + 2)
         partials = ctx.workspace.get("latent.partials", (need,), torch.float32)
-    _f32(q, "latent_attention: q")
-    if out.dtype != cache.dtype or out.stride(1) != 1 or q.shape[2] != D:
-        raise KernelError("latent_attention: out in the cache's dtype, q [T, heads, D]")
     if tracing():
         keys = sum(min(p + 1, window) if window > 0 else p + 1
                    for e, p0 in enumerate(ctx.host_entry_pos0)
                    for p in range(p0, p0 + ctx.host_entry_start[e + 1] - ctx.host_entry_start[e]))
         _note("attn", "latent_attn", (ctx.n_rows, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
-              4.0 * ctx.n_rows * n_head * D + out.element_size() * (ctx.n_rows * n_head * kv_rank + keys * D))
-    _check(library().nib_latent_attention(_dt(cache), _ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
+              q.element_size() * ctx.n_rows * n_head * D + out.element_size() * (ctx.n_rows * n_head * kv_rank + keys * D))
+    _check(library().nib_latent_attention(_dt(cache), _dt(q), _ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
                                           block_table.shape[1], None, _ptr(ctx.row_entry), _ptr(ctx.positions),
                                           ctx.n_rows, n_head, kv_rank, D, page_size, n_pages, float(scale),
-                                          int(window), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                                          _ptr(ctx.status), int(n_splits), _ptr(partials), _stream()),
+                                          int(window), *gate_args, _ptr(ctx.status), int(n_splits), _ptr(partials), _stream()),
            "latent_attention", 2 if n_splits > 1 else 1)
 
 
 def linear_heads(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
-                 M: int) -> None:
-    """out[t, h * out_head_stride + n] = sum_k a[t, h * a_head_stride + k] * w[h, n, k] for w [heads, N, K]."""
+                 M: int, rot=None) -> None:
+    """out[t, h * out_head_stride + n] = sum_k a[t, h * a_head_stride + k] * w[h, n, k] for w [heads, N, K].  bfloat16
+    runs on warp-level MMAs where the strides allow.  ``rot`` (positions, frequencies, rot_dim, rot_dims, halves): a's heads
+    hold ``rot_dim`` more values, which are turned by the rows' positions (as ``rope_heads`` does) and written behind the
+    head's N values in the same launch where that form applies."""
     H, N, K = w.shape
     if a.dtype != w.dtype or not w.is_contiguous() or a.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("linear_heads: a and w share a dtype, w contiguous [heads, N, K]")
     if tracing():
         _note("matmul", "matmul_heads", (M, K, H * N), 2.0 * M * H * N * K,
               w.numel() * w.element_size() + M * H * (K * a.element_size() + N * out.element_size()))
+    if a.dtype == torch.bfloat16 and out.dtype in (torch.bfloat16, torch.float32) and \
+            _can("nib_linear_heads_mma_supported", 16 + (_ptr(a) & 15), a.stride(0), a_head_stride, 16 + (_ptr(w) & 15), K):
+        positions, freqs, rot_dim, rot_dims, halves = rot if rot is not None else (None, None, 0, 0, False)
+        _check(library().nib_linear_heads_mma(_dt(out), _ptr(a), a.stride(0), a_head_stride, _ptr(w), _ptr(out), out.stride(0),
+                                              out_head_stride, M, H, N, K, _ptr(positions), _ptr(freqs), int(rot_dim),
+                                              int(rot_dims), int(halves), _stream()), "linear_heads_mma")
+        return
+    if rot is not None:
+        positions, freqs, rot_dim, rot_dims, halves = rot
+        if out.stride(0) != H * out_head_stride or a_head_stride != K + rot_dim:
+            raise KernelError("linear_heads: with a rotated part a's heads are [K | rot_dim] and out is contiguous")
+        rope_heads(a, K, rot_dim, rot_dims, freqs, positions, out.view(out.shape[0], H, out_head_stride), N, H, M, halves)
     _check(library().nib_linear_heads(_dt(a), _dt(out), _ptr(a), a.stride(0), a_head_stride, _ptr(w), _ptr(out),
                                       out.stride(0), out_head_stride, M, H, N, K, _stream()), "linear_heads")
 

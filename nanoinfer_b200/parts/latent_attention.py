@@ -23,6 +23,7 @@ from typing import List, Optional
 import torch
 
 from ..kernels import ops
+from .attention import AttentionPlan
 from .base import (INIT_ONE_PLUS_NORMAL, MATRIX, VECTOR, KVCacheSpec, KVCacheView, Mixer, ParamSpec, StepContext,
                    StepLimits, TwoProducts, Workspace, register_mixer)
 
@@ -75,6 +76,9 @@ class LatentAttention(TwoProducts, Mixer):
     def kv_spec(self) -> Optional[KVCacheSpec]:
         return KVCacheSpec(1, self.latent_dim, self.window, planes=1)
 
+    def step_planner(self):
+        return "causal_attention", AttentionPlan
+
     def flops_per_key(self) -> float:
         return 2.0 * self.n_head * (self.latent_dim + self.kv_rank)
 
@@ -100,7 +104,7 @@ class LatentAttention(TwoProducts, Mixer):
         self.reserve_products(workspace, limits)
         workspace.reserve("latent.cq", n * self.q_rank, self.dtype)
         workspace.reserve("latent.q", n * H * self.qk_dim, self.dtype)
-        workspace.reserve("latent.q_full", n * H * self.latent_dim, torch.float32)
+        workspace.reserve("latent.q_full", n * H * self.latent_dim, self.dtype)
         workspace.reserve("latent.out", n * H * self.kv_rank, self.dtype)
         ops.latent_attention_reserve(workspace, H, self.kv_rank)
 
@@ -124,14 +128,22 @@ class LatentAttention(TwoProducts, Mixer):
         q = ws.get("latent.q", (n, H * self.qk_dim), self.dtype)
         ops.trace_scope(ctx.layer, "q_up")
         ops.linear(cq, p["q_up"], None, q, T)
-        qf = ws.get("latent.q_full", (n, H, D), torch.float32)
+        # the queries over the latent, [absorbed | rotated] a head, in the engine's dtype
+        qf = ws.get("latent.q_full", (n, H, D), self.dtype)
         if self.nope_dim:
             ops.trace_scope(ctx.layer, "q_absorb")
-            ops.linear_heads(q, self.qk_dim, self.k_up_t, qf.view(n, H * D), D, T)
-        ops.rope_heads(q, self.nope_dim, self.rot_dim, self.rot_dims, self.freqs, ctx.positions, qf, self.kv_rank, H, T,
-                       halves=self.halves)
+            ops.linear_heads(q, self.qk_dim, self.k_up_t, qf.view(n, H * D), D, T,
+                             rot=(ctx.positions, self.freqs, self.rot_dim, self.rot_dims, self.halves) if self.rot_dim else None)
+        else:
+            qf[:T, :, :self.kv_rank].zero_()
+            ops.rope_heads(q, self.nope_dim, self.rot_dim, self.rot_dims, self.freqs, ctx.positions, qf, self.kv_rank, H, T,
+                           halves=self.halves)
+        plan = ctx.plans.get("causal_attention")
+        if plan is None:
+            plan = ctx.plans["causal_attention"] = AttentionPlan(ctx.host_entry_start, ctx.host_entry_pos0,
+                                                                 device=proj.device)
         lat = ws.get("latent.out", (n, H * self.kv_rank), self.dtype)
         ops.latent_attention(qf, cache.layer, lat, cache.block_table, ctx, H, self.kv_rank, self.scale, self.window,
-                             gate=proj[:, self.gate_off:self.gate_off + H] if self.head_gate else None)
+                             gate=proj[:, self.gate_off:self.gate_off + H] if self.head_gate else None, plan=plan)
         ops.trace_scope(ctx.layer, "v_up")
         ops.linear_heads(lat, self.kv_rank, self.v_up, out, self.v_dim, T)

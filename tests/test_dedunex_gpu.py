@@ -268,54 +268,144 @@ def test_one_matching_key_of_either_map_just_inside_and_just_outside_the_window(
                 assert other < (1.01 if window == 1 else 0.55 if window == 2 else 0.2)
 
 
-def _latent_reference(q, lat, kv_rank, scale, positions, gate):
+def _latent_reference(q, lat, kv_rank, scale, positions, gate, window=0):
     out = []
     for i, p in enumerate(positions):
-        keys = lat[:p + 1].double()
+        lo = max(0, p - window + 1) if window else 0
+        keys = lat[lo:p + 1].double()
         pr = torch.softmax(torch.einsum("hd,jd->hj", q[i].double(), keys) * scale, -1)
         o = pr @ keys[:, :kv_rank]
         out.append(o * torch.sigmoid(gate[i].double())[:, None] if gate is not None else o)
     return torch.stack(out)
 
 
-@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("gated", [False, True])
-@pytest.mark.parametrize("H,kv_rank,rot,page", [(3, 32, 8, 16), (9, 64, 16, 16), (1, 20, 6, 32), (12, 128, 32, 48), (4, 256, 32, 16), (2, 512, 64, 16)])
-def test_latent_attention_with_a_gate_per_head(H, kv_rank, rot, page, gated, dtype):
-    """Portions that start anywhere beside single tokens, and single tokens alone, over pages in a scrambled order."""
-    from nanoinfer_b200.kernels import ops
+def _latent_cache(lats, page, D, seed, dt, gone_behind=None):
+    """Pages in a scrambled order; what no request holds is large; ``gone_behind[e]``: entry e's pages wholly behind that
+    position were given back."""
+    nbs = [-(-len(lat) // page) for lat in lats]
+    ids = torch.randperm(sum(nbs) + 3, generator=torch.Generator().manual_seed(seed)).tolist()
+    table = torch.full((len(lats), max(nbs) + 1), -1, dtype=torch.int32)
+    cache = torch.full((sum(nbs) + 3, 1, 1, page, D), 5.0)
+    for e, lat in enumerate(lats):
+        for b in range(nbs[e]):
+            pg = ids.pop()
+            c = min(page, len(lat) - b * page)
+            cache[pg, 0, 0, :c] = lat[b * page:b * page + c]
+            if gone_behind is None or (b + 1) * page > gone_behind[e]:
+                table[e, b] = pg
+    return cache.to(dt).to(DEV), table.to(DEV)
 
-    dt, D, scale = DT[dtype], kv_rank + rot, 0.9 / math.sqrt(kv_rank)
-    for lengths, q_rows in (([200, 77, 301, 40, 16], [130, 1, 260, 3, 16]), ([300, 1, 77, 64], [1, 1, 1, 1])):
-        g = torch.Generator().manual_seed(H + kv_rank)
-        nbs = [-(-n // page) for n in lengths]
-        ids = torch.randperm(sum(nbs) + 3, generator=g).tolist()
-        table = torch.full((len(lengths), max(nbs) + 1), -1, dtype=torch.int32)
-        cache = torch.full((sum(nbs) + 3, 1, 1, page, D), 5.0)
-        lats = []
-        for e, n in enumerate(lengths):
-            lat = torch.randn(n, D, generator=g).to(dt).float()
-            for b in range(nbs[e]):
-                table[e, b] = pg = ids.pop()
-                c = min(page, n - b * page)
-                cache[pg, 0, 0, :c] = lat[b * page:b * page + c]
-            lats.append(lat)
+
+LATENT_CASES = [(3, 32, 8, 16), (9, 64, 16, 16), (1, 20, 6, 32), (12, 128, 32, 48), (4, 256, 32, 16), (2, 512, 64, 16), (17, 96, 24, 16),
+                (5, 256, 64, 32), (40, 16, 8, 16), (2, 8, 0, 16), (3, 200, 40, 16)]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("gated,window", [(False, 0), (True, 0), (True, 70), (False, 1)])
+@pytest.mark.parametrize("H,kv_rank,rot,page", LATENT_CASES)
+def test_latent_attention_every_kernel_with_gates_and_windows(H, kv_rank, rot, page, gated, window, dtype):
+    """Portions that start anywhere beside single tokens, and single tokens alone: in bfloat16 the tcgen05 kernel (portions)
+    and the warp-MMA one (single tokens, their keys in one to sixteen pieces) where the sizes allow, the general one
+    elsewhere; pages behind the window are gone."""
+    from nanoinfer_b200.kernels import ops
+    from nanoinfer_b200.parts.attention import AttentionPlan
+
+    dt, D, scale = DT[dtype], kv_rank + rot, 1.5 / math.sqrt(kv_rank)
+    for lengths, q_rows in (([200, 77, 301, 40, 16], [130, 1, 260, 3, 16]), ([300, 1, 77, 64], [1, 1, 1, 1]), ([700], [1]), ([129, 2, 128], [129, 2, 127])):
+        g = torch.Generator().manual_seed(H + kv_rank + len(lengths))
+        lats = [torch.randn(n, D, generator=g).to(dt).float() for n in lengths]
+        first = [max(0, n - r - window + 1) if window else 0 for n, r in zip(lengths, q_rows)]
+        cache, table = _latent_cache(lats, page, D, H + kv_rank, dt, first)
         positions = [p for n, r in zip(lengths, q_rows) for p in range(n - r, n)]
-        ctx = step_ctx(q_rows, positions, n_pad=3)
+        n_pad = 3 if len(lengths) == 5 else 0
+        ctx = step_ctx(q_rows, positions, n_pad=n_pad)
         T = len(positions)
-        q = torch.randn(T + 3, H, D, generator=g)
-        gate_rows = torch.randn(T + 3, H + 5, generator=g) * 2
-        out = torch.full((T + 3, H * kv_rank + 8), 7.0, device=DEV, dtype=dt)
-        gate = gate_rows.to(DEV)[:, 2:2 + H] if gated else None
-        ops.latent_attention(q.to(DEV), cache.to(dt).to(DEV), out[:, :H * kv_rank], table.to(DEV), ctx, H, kv_rank, scale, 0, gate=gate)
+        q = torch.randn(T + n_pad, H, D, generator=g).to(dt)
+        gate_rows = torch.randn(T + n_pad, H + 5, generator=g) * 2
+        out = torch.full((T + n_pad, H * kv_rank + 8), 7.0, device=DEV, dtype=dt)
+        plan = AttentionPlan(ctx.host_entry_start, ctx.host_entry_pos0, device=torch.device(DEV))
+        ops.latent_attention(q.to(DEV), cache, out[:, :H * kv_rank], table, ctx, H, kv_rank, scale, window,
+                             gate=gate_rows.to(DEV)[:, 2:2 + H] if gated else None, plan=plan)
         assert int(ctx.status.item()) == 0
         at, want = 0, []
         for e, (n, r) in enumerate(zip(lengths, q_rows)):
-            want.append(_latent_reference(q[at:at + r], lats[e], kv_rank, scale, range(n - r, n), gate_rows[at:at + r, 2:2 + H] if gated else None))
+            want.append(_latent_reference(q[at:at + r], lats[e], kv_rank, scale, range(n - r, n),
+                                          gate_rows[at:at + r, 2:2 + H] if gated else None, window))
             at += r
-        err = float((out[:T, :H * kv_rank].double().cpu() - torch.cat(want).reshape(T, -1)).abs().max())
-        assert err < (2e-5 if dtype == "float32" else 3e-2), (lengths, err)
-        assert float(out[:, H * kv_rank:].float().min()) == 7.0
+        err = (out[:T, :H * kv_rank].double().cpu() - torch.cat(want).reshape(T, -1)).abs()
+        assert float(err.max()) < (2e-5 if dtype == "float32" else 4e-2), (lengths, float(err.max()), int(err.max(1).values.argmax()))
+        assert float(out[:, H * kv_rank:].float().min()) == 7.0 and float(out[T:].float().min() if n_pad else 7.0) == 7.0
+
+
+@pytest.mark.parametrize("window", [0, 33, 64])
+@pytest.mark.parametrize("rows", [1, 2, 70, 140])
+@pytest.mark.parametrize("H,kv_rank,rot", [(3, 64, 16), (2, 256, 32)])
+def test_one_matching_latent_just_inside_and_just_outside(H, kv_rank, rot, rows, window):
+    """bfloat16: one cached row towers over all others for every query; it must carry exactly the rows that see it."""
+    from nanoinfer_b200.kernels import ops
+    from nanoinfer_b200.parts.attention import AttentionPlan
+
+    D, page, n = kv_rank + rot, 16, 150 + rows
+    for far in sorted({0, 15, 16, n - 1, n - 2, n - rows, n - rows - 1, n - 64, n - 65, max(0, n - window), max(0, n - window - 1),
+                       max(0, n - rows - window), max(0, n - rows - window + 1)}):
+        if far >= n:
+            continue
+        lat = torch.zeros(n, D)
+        lat[:, 1] = 1.0
+        lat[far] = 0.0
+        lat[far, 2], lat[far, D - 1] = 1.0, 40.0           # the value it carries, and the match (in the rotated part)
+        cache, table = _latent_cache([lat], page, D, far, torch.bfloat16)
+        ctx = step_ctx([rows], list(range(n - rows, n)))
+        q = torch.zeros(rows, H, D)
+        q[:, :, D - 1] = 1.0
+        out = torch.zeros(rows, H * kv_rank, device=DEV, dtype=torch.bfloat16)
+        plan = AttentionPlan(ctx.host_entry_start, ctx.host_entry_pos0, device=torch.device(DEV))
+        ops.latent_attention(q.to(torch.bfloat16).to(DEV), cache, out, table, ctx, H, kv_rank, 1.0, window, plan=plan)
+        got = out.float().view(rows, H, kv_rank)[:, :, 2].cpu()
+        for i in range(rows):
+            p = n - rows + i
+            visible = far <= p and (not window or p - far < window)
+            assert bool((got[i] > 0.9).all()) == visible and bool((got[i] < 0.1).all()) != visible, (far, p)
+
+
+@pytest.mark.parametrize("M", [1, 7, 16, 17, 70, 129])
+@pytest.mark.parametrize("H,N,K,rot,halves", [(3, 64, 64, 0, False), (5, 256, 64, 32, True), (2, 24, 8, 6, False), (4, 72, 200, 10, True), (1, 100, 40, 8, True)])
+def test_product_per_head_on_the_tensor_cores_with_a_rotated_part_behind_it(H, N, K, rot, halves, M):
+    from nanoinfer_b200.kernels import ops
+
+    torch.manual_seed(M + N)
+    dt, dims = torch.bfloat16, rot // 4 * 2
+    a_hs = -(-(K + rot) // 8) * 8 if not rot else K + rot
+    if rot and a_hs % 8:
+        rot = dims = 8
+        a_hs = K + rot
+    a = torch.randn(M, H * a_hs, device=DEV).to(dt)
+    w = (torch.randn(H, N, K, device=DEV) / math.sqrt(K)).to(dt)
+    pos = torch.randint(0, 5000, (M,), dtype=torch.int32, device=DEV)
+    fr = 300.0 ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / max(dims, 1))
+    o_hs = N + rot
+    for out_dt in (dt, torch.float32):
+        out = torch.full((M, H * o_hs + 5), 7.0, device=DEV, dtype=out_dt)
+        view = out[:, :H * o_hs] if not rot else torch.full((M, H * o_hs), 7.0, device=DEV, dtype=out_dt)
+        ops.linear_heads(a, a_hs, w, view, o_hs, M, rot=(pos, fr.to(DEV), rot, dims, halves) if rot else None)
+        x = a.double().cpu().view(M, H, a_hs)
+        want = torch.einsum("mhk,hnk->mhn", x[..., :K], w.double().cpu())
+        got = view.double().cpu().view(M, H, o_hs)
+        tol = 1e-5 if out_dt == torch.float32 else 1e-2
+        assert float(((got[..., :N] - want) / (want.abs() + 1)).abs().max()) < tol
+        if rot:
+            tail = x[..., K:K + rot]
+            if halves:
+                t = _turn_halves(tail, pos.cpu(), dims, fr, 1.0)
+            else:
+                t = tail.clone()
+                ang = pos.cpu().double()[:, None] * fr
+                c, sn = torch.cos(ang)[:, None], torch.sin(ang)[:, None]
+                u, v = tail[..., 0:dims:2], tail[..., 1:dims:2]
+                t[..., 0:dims:2], t[..., 1:dims:2] = u * c - v * sn, v * c + u * sn
+            assert float(((got[..., N:] - t) / (t.abs() + 1)).abs().max()) < tol
+        else:
+            assert float(out[:, H * o_hs:].float().min()) == 7.0
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])

@@ -219,19 +219,26 @@ int nib_latent_attention(int dtype, int q_dtype, const void* q, const void* cach
                          int n_head, int kv_rank, int D, int page_size, int n_pages, float scale, int window,
                          const float* gate, int ldg, int* status, int n_splits, float* partials, cudaStream_t stream);
 
-// The same attention in bfloat16 (queries too) on the tensor cores: prompt portions in tiles of 128 rows on tcgen05
-// (latent_prefill_tc.cu), single tokens on warp-level MMAs with sixteen heads a tile and a row's pieces of keys as one
-// cluster (latent_decode_mma.cu; n_splits 1, 2, 4, 8 or 16).
-int nib_latent_prefill_tc_supported(int kv_rank, int D, int page_size);
-int nib_latent_prefill_tc(const void* q, int T, const void* cache, void* out, int ldo, const int* block_table,
-                          int max_blocks, const int* tiles, int n_tiles, const int* entry_start, const int* entry_pos0,
-                          int n_head, int kv_rank, int D, int page_size, int n_pages, float scale, int window,
+// ---- attention in bfloat16 over cached rows of any of two shapes: keys and values in two planes [n_pages, 2, n_kv_head,
+// page_size, row_dim], or one plane whose rows are both (planes = 1, the latent cache).  Options: softcap, window, a sigmoid
+// gate per row and head.
+// Prompt portions in tiles of 128 rows on tcgen05 (attention_wide_tc.cu): with maps > 1 head h scores against the values
+// (h % maps) * map_dim .. + map_dim of the key row; head h's v_cols values go to column h * out_head of its rows.
+int nib_attention_wide_tc_supported(int row_dim, int planes, int maps, int map_dim, int v_cols, int page_size);
+int nib_attention_wide_tc(const void* q, int ldq, int T, const void* cache, int planes, void* out, int ldo, int out_head,
+                          int out32, const int* block_table, int max_blocks, const int* tiles, int n_tiles,
+                          const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head, int row_dim, int maps,
+                          int map_dim, int v_cols, int page_size, int n_pages, float scale, int window, float softcap,
                           const float* gate, int ldg, int* status, cudaStream_t stream);
-int nib_latent_decode_mma_supported(int kv_rank, int D);
-int nib_latent_decode_mma(const void* q, const void* cache, void* out, int ldo, const int* block_table, int max_blocks,
-                          const int* rows, const int* row_entry, const int* positions, int n_rows, int n_head, int kv_rank,
-                          int D, int page_size, int n_pages, float scale, int window, const float* gate, int ldg,
-                          int* status, int n_splits, cudaStream_t stream);
+// Single tokens on warp-level MMAs with the heads of a group as rows and a row's pieces of keys as one cluster
+// (attention_group_mma.cu; n_splits 1, 2, 4, 8 or 16).  diff: the heads come in pairs, and pair i's column i * out_head
+// receives mul * o / sqrt(mean(o^2) + eps), o = a_2i - lambda a_2i+1.
+int nib_attention_group_mma_supported(int row_dim, int planes, int k_cols, int v_cols, int diff);
+int nib_attention_group_mma(const void* q, int ldq, const void* cache, int planes, void* out, int ldo, int out_head,
+                            const int* block_table, int max_blocks, const int* rows, const int* row_entry,
+                            const int* positions, int n_rows, int n_head, int n_kv_head, int row_dim, int k_cols, int v_cols,
+                            int page_size, int n_pages, float scale, int window, float softcap, const float* gate, int ldg,
+                            int diff, float lambda, float eps, float mul, int* status, int n_splits, cudaStream_t stream);
 
 // ---- a product per head (linear_heads.cu; in bfloat16 on warp-level MMAs: linear_heads_mma.cu): out[t, h, :N] = a[t, h, :K] . w[h]^T, w [n_head, N, K]
 int nib_linear_heads(int dtype, int out_dtype, const void* a, int lda, int a_head_stride, const void* w, void* out,
@@ -355,8 +362,9 @@ int nib_norm_rope_maps_append(int dtype, const float* proj, int ld, int q_off, i
                               float eps, int rot_dims, const double* freqs, float amp, const int* positions,
                               const int* row_entry, void* q_out, int ldq, void* cache, const int* block_table,
                               int max_blocks, int page_size, int n_pages, int T, int* status, cudaStream_t stream);
-// out[t, h, :vdim] = mul * o / sqrt(mean(o^2) + eps) with o = a[t, 2h] - lambda * a[t, 2h + 1], a 32-bit heads of hd.
-int nib_diff_combine(int out_dtype, const float* a, int lda, int n_head, int hd, int vdim, float lambda, float eps,
+// out[t, h, :vdim] = mul * o / sqrt(mean(o^2) + eps) with o = a[t, 2h] - lambda * a[t, 2h + 1], a 32-bit heads of hd; rows: the T rows
+// to process (null: rows 0..T-1).
+int nib_diff_combine(int out_dtype, const float* a, int lda, const int* rows, int n_head, int hd, int vdim, float lambda, float eps,
                      float mul, void* out, int ldo, int T, cudaStream_t stream);
 
 // ---- the minimal gated recurrent unit (min_gru.cu): z, u and g logits at three column offsets of the 32-bit proj.

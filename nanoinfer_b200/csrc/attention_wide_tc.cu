@@ -1,20 +1,28 @@
-// Attention through a low-rank latent for prompt portions, on the fifth-generation tensor cores (bfloat16).
+// Attention for prompt portions on the fifth-generation tensor cores where a cached row is wider than one swizzle row of 64
+// values (bfloat16), in two shapes of the cache:
 //
-// A head's query has been carried into the latent space (latent_attention.cu says how), so that every head attends over
-// the same cached rows [c | k_rot] of D values, and the weighted sum is over their first kv_rank values: one tile of the
-// cache is both the keys and the values.  One block takes 128 consecutive query rows of one request and one head and
-// walks the keys in tiles of 64:
-//   warp 0      the producer: Q once; then a tile of the cache at a time, 16 rows x 64 values a TMA load (a lane each, with
-//               its own look-up in the block table), into a ring of stages of 128-byte-swizzled shared memory, a stage
-//               being D / 64 chunks of [64 keys][64 values];
-//   warp 1      the MMAs: S = Q K^T (128 x 64 x D) into one of two score buffers in tensor memory; O += P V (128 x kv_rank x
-//               64) with P from shared memory and V the same stage read as an MN-major operand (keys down the rows, chunks of
-//               64 values side by side), accumulated in tensor memory over all tiles.  A stage is free when its P V is done;
-//   warps 2..5  the softmax, a thread a row: scores times log2(e), running maximum raised only when a tile exceeds it by
-//               more than 2^8 (O is then scaled in tensor memory), P as bfloat16, the sum in 32-bit; at the end the
-//               division, the head's gate, and the store.
+//   keys and values in planes of their own, rows of row_dim values (up to 256).  A head may own a part of the key row only:
+//   with `maps` > 1 query head h scores against the values [m map_dim, (m + 1) map_dim) of its key/value head's row,
+//   m = h % maps (differential attention lays the keys of a head's maps side by side; the query is zero elsewhere, so the
+//   bounds need not fall on a boundary of anything), and v_cols of the value row count;
+//
+//   one plane whose row is key and value at once (a latent [c | k_rot] shared by all heads, latent_attention.cu; rows up to
+//   320, v_cols = kv_rank up to 256): a tile is loaded once and read as both.
+//
+// One block takes 128 consecutive query rows of one request and one head and walks the keys in tiles of 64:
+//   warp 0      the producer: Q once; then a tile at a time, 16 rows x 64 values a TMA load (a lane each, with its own look-up
+//               in the block table), into a ring of stages of 128-byte-swizzled shared memory: chunks of [64 keys][64 values],
+//               those of the key row that the head needs, then those of the value row;
+//   warp 1      the MMAs: S = Q K^T (128 x 64 x the head's part of the row) into one of two score buffers in tensor memory;
+//               O += P V (128 x v_cols x 64) with P from shared memory and V as it lies, keys down the rows, an MN-major
+//               operand of chunks side by side, accumulated in tensor memory over all tiles.  Whatever is ready goes next,
+//               P V first (it frees a stage);
+//   warps 2..5  the softmax, a thread a row: scores times log2(e) (capped first where asked for), running maximum raised only
+//               when a tile exceeds it by more than 2^8 (O is then scaled in tensor memory), P as bfloat16, the sum in
+//               32-bit; at the end the division, an optional sigmoid gate per row and head, and the store (bfloat16, or
+//               32-bit floats).
 // Keys outside [lowest visible, last row] are masked; their rows are read from the nearest unit of the request that is
-// there.  What a box reaches beyond D, or beyond the step's rows, reads as zeros.
+// there.  What a box reaches beyond the row, or beyond the step's rows, reads as zeros.
 //
 // Every wait on a barrier is bounded: a wait that runs out sets the block's abort flag and the device status word, every
 // role leaves its loop, tensor memory is freed, and the kernel returns.
@@ -25,7 +33,7 @@
 namespace nib {
 
 constexpr int LP_BM = 128, LP_BN = 64, LP_UNIT = 16, LP_THREADS = 192, LP_NBUF = 2, LP_MAX_STAGES = 4;
-constexpr int LP_MAX_CHUNKS = 5, LP_MAX_V_CHUNKS = 4;        // D <= 320, kv_rank <= 256
+constexpr int LP_MAX_SLOTS = 8, LP_MAX_V_CHUNKS = 4;          // chunks of a stage (four lanes each), values <= 256
 constexpr int LP_CHUNK_Q = LP_BM * 128, LP_CHUNK_K = LP_BN * 128, LP_P_BYTES = LP_BM * 128;
 constexpr uint32_t LP_O_COL = LP_NBUF * LP_BN, LP_TMEM_COLS = 512;
 constexpr float LP_RAISE = 8.0f;
@@ -36,14 +44,16 @@ struct LpParams {
   const int* tiles;            // pairs (entry, first row within the entry), 128 rows each
   const int* entry_start;
   const int* entry_pos0;
-  int page_size, n_pages;
-  int kv_rank, n_chunks, v_chunks, stages;
-  float scale;
+  int page_size, n_pages, n_head, n_kv_head, planes;
+  int row_dim, maps, map_dim;   // a head's keys: values (h % maps) * map_dim .. + map_dim of the row
+  int v_cols, v_chunks;         // values of the result, chunks of the value row
+  int k_slots, stages;          // chunks of keys a stage holds room for
+  float scale, softcap;
   int window;
   const float* gate;
   int ldg;
-  bf16* out;
-  int ldo;
+  void* out;
+  int ldo, out_head, out32;     // rows and heads of the result, in elements
   int* status;
 };
 
@@ -77,16 +87,34 @@ __device__ __forceinline__ void lp_tmem_st16(uint32_t taddr, const float* v) {
       : "memory");
 }
 
+__device__ __forceinline__ bool lp_test(uint64_t* bar, uint32_t parity) {   // has the phase completed?  (does not wait)
+  uint32_t ok;
+  asm volatile(
+      "{\n\t.reg .pred P1;\n\t"
+      "mbarrier.test_wait.parity.shared::cta.b64 P1, [%1], %2;\n\t"
+      "selp.b32 %0, 1, 0, P1;\n\t}"
+      : "=r"(ok)
+      : "r"(smem_u32(bar)), "r"(parity)
+      : "memory");
+  return ok != 0;
+}
+
 __global__ void __launch_bounds__(LP_THREADS, 1)
-latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
+attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                          const LpParams prm) {
   extern __shared__ uint8_t lp_smem_raw[];
   // tiles must start on a 1024-byte boundary for the 128-byte swizzle
   uint8_t* smem = reinterpret_cast<uint8_t*>(((uintptr_t)lp_smem_raw + 1023) & ~(uintptr_t)1023);
-  const int nk = prm.n_chunks, nv = prm.v_chunks, stages = prm.stages;
-  const int stage_bytes = nk * LP_CHUNK_K;
+  const bool shared_row = prm.planes == 1;              // one row is key and value
+  const int h = blockIdx.x, hk = h / (prm.n_head / prm.n_kv_head);
+  // the head's part of the key row: steps of 16 values, chunks of 64
+  const int k_from = (h % prm.maps) * prm.map_dim, ks_lo = k_from / 16, ks_hi = (k_from + prm.map_dim + 15) / 16;
+  const int c_lo = ks_lo / 4, nk = (ks_hi + 3) / 4 - c_lo;
+  const int nv = prm.v_chunks, stages = prm.stages;
+  const int n_slots = prm.k_slots + (shared_row ? 0 : nv);              // of a stage
+  const int stage_bytes = n_slots * LP_CHUNK_K, v_off = shared_row ? 0 : prm.k_slots * LP_CHUNK_K;
   uint8_t* q_s = smem;                                  // [chunks][128 rows][64]
-  uint8_t* k_s = q_s + nk * LP_CHUNK_Q;                 // [stages][chunks][64 keys][64]
+  uint8_t* k_s = q_s + prm.k_slots * LP_CHUNK_Q;        // [stages][key chunks, value chunks][64 keys][64]
   uint8_t* p_s = k_s + stages * stage_bytes;            // [2][128 rows][64 keys]
   __shared__ __align__(8) uint64_t q_full, k_full[LP_MAX_STAGES], k_empty[LP_MAX_STAGES], s_full[LP_NBUF], p_full[LP_NBUF],
       o_full[LP_NBUF];
@@ -97,7 +125,6 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // (heads are the fast index of the grid: blocks start in the order of the tile list, longest first)
   const int e = prm.tiles[2 * blockIdx.y], q_off = prm.tiles[2 * blockIdx.y + 1];
-  const int h = blockIdx.x;
   const int row0 = prm.entry_start[e] + q_off;                    // first row of the tile in the step
   const int n_rows = min(LP_BM, prm.entry_start[e + 1] - row0);
   const int pos_first = prm.entry_pos0[e] + q_off;                // position of the tile's first row
@@ -135,9 +162,12 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     // ---------------- producer
     if (lane == 0) mbar_expect_tx(&q_full, (uint32_t)(nk * LP_CHUNK_Q));
     __syncwarp();
-    if (lane < nk) tma_load_3d(q_s + lane * LP_CHUNK_Q, &map_q, &q_full, lane * 64, h, row0);
-    const int u = lane & 3, chunk = lane >> 2;             // unit of 16 keys, chunk of 64 values
-    const bool active = chunk < nk;
+    if (lane < nk) tma_load_3d(q_s + lane * LP_CHUNK_Q, &map_q, &q_full, (c_lo + lane) * 64, h, row0);
+    const int u = lane & 3, slot = lane >> 2;              // unit of 16 keys, place in the stage
+    const bool is_v = !shared_row && slot >= prm.k_slots;
+    const bool active = is_v ? slot < n_slots : slot < nk;
+    const int x = is_v ? (slot - prm.k_slots) * 64 : (c_lo + slot) * 64;
+    const uint32_t tile_bytes = (uint32_t)((nk + (shared_row ? 0 : nv)) * LP_CHUNK_K);
     auto unit_row = [&](int it) -> int {
       if (!active || it >= n_it) return 0;
       int j = min((tile_first + it) * LP_BN + u * LP_UNIT, pos_last) / LP_UNIT * LP_UNIT;
@@ -147,20 +177,20 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         *prm.status = NIB_STATUS_BAD_PAGE;
         return 0;                                          // (page 0: in the pool)
       }
-      return page * prm.page_size + j % prm.page_size;
+      return ((page * prm.planes + (is_v ? 1 : 0)) * prm.n_kv_head + hk) * prm.page_size + j % prm.page_size;
     };
     bool ok = true;
     int row_next = unit_row(0);
-    uint8_t* dst = k_s + chunk * LP_CHUNK_K + u * (LP_UNIT * 128);
+    uint8_t* dst = k_s + slot * LP_CHUNK_K + u * (LP_UNIT * 128);
     for (int it = 0; it < n_it; ++it) {
       const int st = it % stages, round = it / stages;
       const int row = row_next;
       row_next = unit_row(it + 1);    // the next tile's look-up travels while this tile's stage is waited for
       if (round > 0) ok = warp_mbar_wait(&k_empty[st], (round + 1) & 1, abort_flag, lane);
       if (!ok) break;
-      if (lane == 0) mbar_expect_tx(&k_full[st], (uint32_t)stage_bytes);
+      if (lane == 0) mbar_expect_tx(&k_full[st], tile_bytes);
       __syncwarp();
-      if (active) tma_load_2d(dst + st * stage_bytes, &map_kv, &k_full[st], chunk * 64, row);
+      if (active) tma_load_2d(dst + st * stage_bytes, &map_kv, &k_full[st], x, row);
     }
     __syncwarp();
   } else if (warp == 1) {
@@ -170,35 +200,46 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       const uint32_t idesc_o = umma_idesc(LP_BM, nv * 64) | (1u << 16);   // B (= V) is MN-major: keys down the rows
       const uint32_t o_tmem = tmem_base + LP_O_COL;
       const uint32_t qa = smem_u32(q_s);
-      auto issue_s = [&](int it) -> bool {
-        const int st = it % stages;
-        if (!mbar_wait(&k_full[st], (it / stages) & 1, abort_flag)) return false;
+      auto issue_s = [&](int it) {
         tc_fence_after();
-        const uint32_t kb = smem_u32(k_s + st * stage_bytes);
-        for (int c = 0; c < nk; ++c)
-#pragma unroll
-          for (int k = 0; k < 4; ++k)   // 16 of a chunk's 64 values per instruction: 32 bytes along the row
-            umma_bf16(tmem_base + (uint32_t)((it % LP_NBUF) * LP_BN), umma_desc(qa + c * LP_CHUNK_Q + k * 32),
-                      umma_desc(kb + c * LP_CHUNK_K + k * 32), idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+        const uint32_t kb = smem_u32(k_s + (it % stages) * stage_bytes);
+        for (int ks = ks_lo; ks < ks_hi; ++ks) {   // 16 values per instruction: 32 bytes along a chunk's row
+          const int c = ks / 4 - c_lo, k = ks & 3;
+          umma_bf16(tmem_base + (uint32_t)((it % LP_NBUF) * LP_BN), umma_desc(qa + c * LP_CHUNK_Q + k * 32),
+                    umma_desc(kb + c * LP_CHUNK_K + k * 32), idesc_s, ks > ks_lo ? 1u : 0u);
+        }
         umma_commit(&s_full[it % LP_NBUF]);
-        return true;
       };
       // (V's chunks lie LP_CHUNK_K bytes apart along the values: that is the descriptor's leading byte offset)
       const uint64_t lead = (uint64_t)(LP_CHUNK_K >> 4) << 16;
       auto v_desc = [&](uint32_t addr) { return (umma_desc(addr) & ~(0x3fffull << 16)) | lead; };
-      bool ok = mbar_wait(&q_full, 0, abort_flag);
-      for (int a = 0; ok && a < LP_NBUF && a < n_it; ++a) ok = issue_s(a);
-      for (int it = 0; ok && it < n_it; ++it) {
-        const int st = it % stages, b = it % LP_NBUF;
-        if (!mbar_wait(&p_full[b], (it / LP_NBUF) & 1, abort_flag)) break;
+      auto issue_pv = [&](int it) {
         tc_fence_after();
-        const uint32_t vb = smem_u32(k_s + st * stage_bytes), pa = smem_u32(p_s + b * LP_P_BYTES);
+        const int st = it % stages, b = it % LP_NBUF;
+        const uint32_t vb = smem_u32(k_s + st * stage_bytes + v_off), pa = smem_u32(p_s + b * LP_P_BYTES);
 #pragma unroll
         for (int k = 0; k < LP_BN / 16; ++k)   // 16 keys per instruction: P 32 bytes along its row, V 16 rows down
           umma_bf16(o_tmem, umma_desc(pa + k * 32), v_desc(vb + k * 2048), idesc_o, (it > 0 || k > 0) ? 1u : 0u);
         umma_commit(&o_full[b]);
         umma_commit(&k_empty[st]);
-        if (it + LP_NBUF < n_it) ok = issue_s(it + LP_NBUF);
+      };
+      bool ok = mbar_wait(&q_full, 0, abort_flag);
+      int s_next = 0, pv_next = 0;
+      long long t0 = clock64();
+      while (ok && pv_next < n_it) {
+        if (pv_next < s_next && lp_test(&p_full[pv_next % LP_NBUF], (pv_next / LP_NBUF) & 1)) {
+          issue_pv(pv_next++);
+          t0 = clock64();
+        } else if (s_next < n_it && s_next < pv_next + LP_NBUF && lp_test(&k_full[s_next % stages], (s_next / stages) & 1)) {
+          // (the score buffer is free: P of two tiles ago was made from it, or its P V would not have been issued)
+          issue_s(s_next++);
+          t0 = clock64();
+        } else if (*abort_flag) {
+          ok = false;
+        } else if (clock64() - t0 > TC_WAIT_CYCLES) {
+          *abort_flag = 1;
+          ok = false;
+        }
       }
     }
     __syncwarp();
@@ -210,7 +251,10 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int p = pos_first + r;
     const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
     const int wp0 = pos_first + quarter * 32, wp1 = wp0 + 31;   // positions of the warp's rows
-    const float scale2 = prm.scale * 1.4426950408889634f;
+    constexpr float LOG2E = 1.4426950408889634f;
+    const bool capped = prm.softcap > 0.0f;
+    const float scale2 = capped ? 1.0f : prm.scale * LOG2E;    // (capped scores are brought to their final form first)
+    const float cap2 = prm.softcap * LOG2E, cap_in = capped ? 2.0f * LOG2E * prm.scale / prm.softcap : 0.0f;
     float m = -INFINITY, l = 0.0f;
     bool ok = true;
     for (int it = 0; it < n_it; ++it) {
@@ -223,6 +267,11 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       float v[LP_BN];
 #pragma unroll
       for (int c = 0; c < LP_BN / 32; ++c) lp_tmem_ld32(lane_addr + (uint32_t)(b * LP_BN + c * 32), v + c * 32);
+      if (capped) {
+        // c tanh(x / c) by tanh(y) = 1 - 2 / (1 + e^2y) with the hardware's 2^x and division: relative error about 1e-6
+#pragma unroll
+        for (int i = 0; i < LP_BN; ++i) v[i] = cap2 - __fdividef(2.0f * cap2, 1.0f + lp_pow2(v[i] * cap_in));
+      }
       if (edge) {
 #pragma unroll
         for (int i = 0; i < LP_BN; ++i)
@@ -284,18 +333,28 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       tc_fence_after();
       float inv = l > 0.0f ? 1.0f / l : 0.0f;
       if (prm.gate != nullptr && r < n_rows) inv *= 1.0f / (1.0f + __expf(-prm.gate[(size_t)(row0 + r) * prm.ldg + h]));
-      bf16* dst = prm.out + (size_t)(row0 + r) * prm.ldo + (size_t)h * prm.kv_rank;
+      const size_t at = (size_t)(row0 + r) * prm.ldo + (size_t)h * prm.out_head;
+      bf16* dst = reinterpret_cast<bf16*>(prm.out) + at;
+      float* dst32 = reinterpret_cast<float*>(prm.out) + at;
 #pragma unroll 1
       for (int c = 0; c < nv * 4; ++c) {
         float t[16];
         tmem_ld16(lane_addr + LP_O_COL + (uint32_t)(c * 16), t);
         if (r < n_rows) {
 #pragma unroll
-          for (int g = 0; g < 2; ++g)
-            if (c * 16 + 8 * g < prm.kv_rank)       // (kv_rank is a multiple of 8)
-              *reinterpret_cast<uint4*>(dst + c * 16 + 8 * g) =
+          for (int g = 0; g < 2; ++g) {
+            const int d = c * 16 + 8 * g;
+            if (d >= prm.v_cols) continue;          // (v_cols is a multiple of 8)
+            if (prm.out32) {
+              *reinterpret_cast<float4*>(dst32 + d) = make_float4(t[8 * g] * inv, t[8 * g + 1] * inv, t[8 * g + 2] * inv, t[8 * g + 3] * inv);
+              *reinterpret_cast<float4*>(dst32 + d + 4) =
+                  make_float4(t[8 * g + 4] * inv, t[8 * g + 5] * inv, t[8 * g + 6] * inv, t[8 * g + 7] * inv);
+            } else {
+              *reinterpret_cast<uint4*>(dst + d) =
                   make_uint4(pack_bf16(t[8 * g] * inv, t[8 * g + 1] * inv), pack_bf16(t[8 * g + 2] * inv, t[8 * g + 3] * inv),
                              pack_bf16(t[8 * g + 4] * inv, t[8 * g + 5] * inv), pack_bf16(t[8 * g + 6] * inv, t[8 * g + 7] * inv));
+            }
+          }
         }
       }
     }
@@ -309,12 +368,12 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   }
 }
 
-// Q as [T rows][heads][D values], moved in boxes of 128 rows x 1 head x 64 values; what lies beyond D or T reads as zeros.
-static bool make_q_map(CUtensorMap* map, const void* base, int T, int n_head, int D) {
+// Q as [T rows][heads][row_dim values], moved in boxes of 128 rows x 1 head x 64 values; what lies beyond reads as zeros.
+static bool make_q_map(CUtensorMap* map, const void* base, int ldq, int T, int n_head, int row_dim) {
   EncodeTiledFn fn = encode_fn();
   if (!fn) return false;
-  cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)n_head, (cuuint64_t)T};
-  cuuint64_t strides[2] = {(cuuint64_t)D * 2, (cuuint64_t)n_head * D * 2};
+  cuuint64_t dims[3] = {(cuuint64_t)row_dim, (cuuint64_t)n_head, (cuuint64_t)T};
+  cuuint64_t strides[2] = {(cuuint64_t)row_dim * 2, (cuuint64_t)ldq * 2};
   cuuint32_t box[3] = {64, 1, LP_BM};
   cuuint32_t estr[3] = {1, 1, 1};
   return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
@@ -322,53 +381,75 @@ static bool make_q_map(CUtensorMap* map, const void* base, int T, int n_head, in
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-static size_t lp_smem(int n_chunks, int stages) {
-  return (size_t)n_chunks * LP_CHUNK_Q + (size_t)stages * n_chunks * LP_CHUNK_K + (size_t)LP_NBUF * LP_P_BYTES + 1024;
+// chunks of 64 values that the keys of any map of a row touch (whole steps of 16 values)
+static int lp_key_chunks(int maps, int map_dim) {
+  int most = 0;
+  for (int m = 0; m < maps; ++m) {
+    const int lo = m * map_dim / 16, hi = ((m + 1) * map_dim + 15) / 16;
+    const int n = (hi + 3) / 4 - lo / 4;
+    if (n > most) most = n;
+  }
+  return most;
 }
+static size_t lp_smem(int k_slots, int v_slots, int stages) {
+  return (size_t)k_slots * LP_CHUNK_Q + (size_t)stages * (k_slots + v_slots) * LP_CHUNK_K + (size_t)LP_NBUF * LP_P_BYTES + 1024;
+}
+constexpr size_t LP_MAX_SMEM = 225 * 1024;
 
 }  // namespace nib
 
 using namespace nib;
 
-// 1 if the kernel takes these sizes: D a multiple of 8 up to 320, kv_rank a multiple of 8 up to 256, pages of a multiple
-// of 16 positions.
-extern "C" int nib_latent_prefill_tc_supported(int kv_rank, int D, int page_size) {
-  return D % 8 == 0 && D <= 64 * LP_MAX_CHUNKS && kv_rank % 8 == 0 && kv_rank > 0 && kv_rank <= 64 * LP_MAX_V_CHUNKS &&
-         kv_rank <= D && page_size >= LP_UNIT && page_size % LP_UNIT == 0;
+// 1 if the kernel takes these sizes: rows of a multiple of 8 values, v_cols a multiple of 8 up to 256, pages of a multiple of
+// 16 positions, two stages within shared memory.
+extern "C" int nib_attention_wide_tc_supported(int row_dim, int planes, int maps, int map_dim, int v_cols, int page_size) {
+  if (row_dim <= 0 || row_dim % 8 || (planes != 1 && planes != 2) || maps <= 0 || map_dim <= 0 || maps * map_dim > row_dim) return 0;
+  if (v_cols <= 0 || v_cols % 8 || v_cols > row_dim || v_cols > 64 * LP_MAX_V_CHUNKS) return 0;
+  if (page_size < LP_UNIT || page_size % LP_UNIT) return 0;
+  const int nv = (v_cols + 63) / 64, nk = lp_key_chunks(maps, map_dim), vs = planes == 1 ? 0 : nv;
+  if (planes == 1 && (maps != 1 || map_dim != row_dim)) return 0;
+  return nk + vs <= LP_MAX_SLOTS && lp_smem(nk, vs, 2) <= LP_MAX_SMEM;
 }
 
-// tiles: n_tiles pairs (entry, first row within the entry), 128 rows each (the last of an entry may be shorter).  q [T,
-// n_head, D] contiguous bfloat16; cache: one layer [n_pages, page_size, D]; out rows of n_head * kv_rank values, 16-byte
-// aligned.
-extern "C" int nib_latent_prefill_tc(const void* q, int T, const void* cache, void* out, int ldo, const int* block_table,
-                                     int max_blocks, const int* tiles, int n_tiles, const int* entry_start,
-                                     const int* entry_pos0, int n_head, int kv_rank, int D, int page_size, int n_pages,
-                                     float scale, int window, const float* gate, int ldg, int* status,
+// tiles: n_tiles pairs (entry, first row within the entry), 128 rows each (the last of an entry may be shorter).  q [T rows,
+// ldq], heads of row_dim values one after the other; cache: one layer [n_pages, planes, n_kv_head, page_size, row_dim]; out:
+// head h's v_cols values at column h * out_head of its rows (ldo elements apart), bfloat16 or with out32 32-bit floats.
+extern "C" int nib_attention_wide_tc(const void* q, int ldq, int T, const void* cache, int planes, void* out, int ldo,
+                                     int out_head, int out32, const int* block_table, int max_blocks, const int* tiles,
+                                     int n_tiles, const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head,
+                                     int row_dim, int maps, int map_dim, int v_cols, int page_size, int n_pages, float scale,
+                                     int window, float softcap, const float* gate, int ldg, int* status,
                                      cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
-  if (!nib_latent_prefill_tc_supported(kv_rank, D, page_size)) return NIB_ERR_UNSUPPORTED_SIZE;
-  if (n_head <= 0 || T <= 0 || !(scale > 0.0f)) return NIB_ERR_BAD_ARGUMENT;
-  if (((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 15) || (ldo & 7)) return NIB_ERR_UNSUPPORTED_SIZE;
-  const long long kv_rows = (long long)n_pages * page_size;
+  if (!nib_attention_wide_tc_supported(row_dim, planes, maps, map_dim, v_cols, page_size)) return NIB_ERR_UNSUPPORTED_SIZE;
+  if (n_head <= 0 || n_kv_head <= 0 || n_head % n_kv_head || T <= 0 || !(scale > 0.0f) || softcap < 0.0f)
+    return NIB_ERR_BAD_ARGUMENT;
+  const int align = out32 ? 3 : 7;
+  if (((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 15) || (ldo & align) || (out_head & align) || (ldq & 7))
+    return NIB_ERR_UNSUPPORTED_SIZE;
+  const long long kv_rows = (long long)n_pages * planes * n_kv_head * page_size;
   if (n_tiles > 65535 || kv_rows > 0x7fffffffll) return NIB_ERR_UNSUPPORTED_SIZE;
   CUtensorMap map_q, map_kv;
-  if (!make_q_map(&map_q, q, T, n_head, D)) return NIB_ERR_DRIVER;
-  if (!make_map(&map_kv, cache, false, (int)kv_rows, D, D, LP_UNIT, 64, true)) return NIB_ERR_DRIVER;
+  if (!make_q_map(&map_q, q, ldq, T, n_head, row_dim)) return NIB_ERR_DRIVER;
+  if (!make_map(&map_kv, cache, false, (int)kv_rows, row_dim, row_dim, LP_UNIT, 64, true)) return NIB_ERR_DRIVER;
   LpParams prm;
   prm.block_table = block_table; prm.max_blocks = max_blocks; prm.tiles = tiles;
   prm.entry_start = entry_start; prm.entry_pos0 = entry_pos0; prm.page_size = page_size; prm.n_pages = n_pages;
-  prm.kv_rank = kv_rank; prm.n_chunks = (D + 63) / 64; prm.v_chunks = (kv_rank + 63) / 64;
+  prm.n_head = n_head; prm.n_kv_head = n_kv_head; prm.planes = planes;
+  prm.row_dim = row_dim; prm.maps = maps; prm.map_dim = map_dim;
+  prm.v_cols = v_cols; prm.v_chunks = (v_cols + 63) / 64; prm.k_slots = lp_key_chunks(maps, map_dim);
+  const int vs = planes == 1 ? 0 : prm.v_chunks;
   prm.stages = 2;
-  while (prm.stages < LP_MAX_STAGES && lp_smem(prm.n_chunks, prm.stages + 1) <= 220 * 1024) ++prm.stages;
-  prm.scale = scale; prm.window = window; prm.gate = gate; prm.ldg = ldg; prm.out = (bf16*)out; prm.ldo = ldo;
-  prm.status = status;
-  const size_t smem = lp_smem(prm.n_chunks, prm.stages);
+  while (prm.stages < LP_MAX_STAGES && lp_smem(prm.k_slots, vs, prm.stages + 1) <= LP_MAX_SMEM) ++prm.stages;
+  prm.scale = scale; prm.softcap = softcap; prm.window = window; prm.gate = gate; prm.ldg = ldg;
+  prm.out = out; prm.ldo = ldo; prm.out_head = out_head; prm.out32 = out32; prm.status = status;
   static bool attr_set = false;
   if (!attr_set) {
-    const cudaError_t err = cudaFuncSetAttribute(latent_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);
+    const cudaError_t err = cudaFuncSetAttribute(attention_wide_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LP_MAX_SMEM);
     if (err != cudaSuccess) return (int)err;
     attr_set = true;
   }
-  launch_pdl(latent_prefill_tc_kernel, dim3(n_head, n_tiles), dim3(LP_THREADS), smem, stream, map_q, map_kv, prm);
+  launch_pdl(attention_wide_tc_kernel, dim3(n_head, n_tiles), dim3(LP_THREADS), lp_smem(prm.k_slots, vs, prm.stages), stream,
+             map_q, map_kv, prm);
   NIB_LAUNCH_CHECK();
 }

@@ -64,6 +64,12 @@ group_norm_vec_kernel(Src src, const float* __restrict__ w, OutT* out, int n_row
   const int unit = blockIdx.x * 8 + (threadIdx.x >> 5);
   const int r = unit / groups, g = unit % groups;
   const int gs = C / groups, n4 = gs >> 2, c0 = g * gs;
+  float4 ww[NV];                                   // (the weights do not wait for the kernel ahead)
+  if (out != nullptr) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (lane + 32 * i < n4) ww[i] = gn_load4(w + c0 + 4 * (lane + 32 * i));
+  }
   pdl_wait();
   if (r >= n_rows) return;
   auto* p = src.row(r, C) + c0;
@@ -93,8 +99,7 @@ group_norm_vec_kernel(Src src, const float* __restrict__ w, OutT* out, int n_row
   for (int i = 0; i < NV; ++i) {
     const int k = lane + 32 * i;
     if (k < n4) {
-      const float4 ww = gn_load4(w + c0 + 4 * k);
-      gn_store4(o + 4 * k, v[i].x * rstd * ww.x, v[i].y * rstd * ww.y, v[i].z * rstd * ww.z, v[i].w * rstd * ww.w);
+      gn_store4(o + 4 * k, v[i].x * rstd * ww[i].x, v[i].y * rstd * ww[i].y, v[i].z * rstd * ww[i].z, v[i].w * rstd * ww[i].w);
     }
   }
 }

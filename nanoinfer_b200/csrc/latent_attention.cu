@@ -32,34 +32,55 @@ latent_prep_kernel(const float* proj, int ld, int q_rank, int kv_rank, int rot_d
                    const int* __restrict__ row_entry, const int* __restrict__ positions, int page_size,
                    int n_pages, int has_kv, int halves, int* status) {
   pdl_trigger();
-  __shared__ float scratch[32];
-  const int t = blockIdx.x;
+  extern __shared__ float lat_cs[];               // cosine and sine of the row's pairs
+  __shared__ float sums[2][32];
+  const int t = blockIdx.x, half = rot_dims / 2;
   const int entry = row_entry[t], pos = positions[t];
+  const bool kv_row = has_kv && entry >= 0;        // not in a layer that reads another's cache, nor for a row of no request
+  int page = -1;
+  if (kv_row) {
+    page = block_table[(size_t)entry * max_blocks + pos / page_size];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      double sn, c;
+      sincos((double)pos * freqs[i], &sn, &c);
+      lat_cs[2 * i] = (float)c;
+      lat_cs[2 * i + 1] = (float)sn;
+    }
+  }
   pdl_wait();
   const float* src = proj + (size_t)t * ld;
-  float s = 0.0f;
+  const float* kv = src + q_rank;
+  float s = 0.0f, s2 = 0.0f;
   for (int c = threadIdx.x; c < q_rank; c += blockDim.x) s += src[c] * src[c];
-  const float rq = 1.0f / sqrtf(block_sum(s, scratch) / (float)q_rank + eps);
+  if (kv_row)
+    for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) s2 += kv[c] * kv[c];
+  // both sums over the block with one meeting, in a fixed order
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  s = warp_sum(s);
+  s2 = warp_sum(s2);
+  if (lane == 0) {
+    sums[0][warp] = s;
+    sums[1][warp] = s2;
+  }
+  __syncthreads();
+  s = warp_sum(lane < n_warps ? sums[0][lane] : 0.0f);
+  s2 = warp_sum(lane < n_warps ? sums[1][lane] : 0.0f);
+  const float rq = 1.0f / sqrtf(s / (float)q_rank + eps);
   for (int c = threadIdx.x; c < q_rank; c += blockDim.x)
     cq[(size_t)t * ld_cq + c] = from_float<T>(src[c] * rq * wq[c]);
-  if (!has_kv || entry < 0) return;    // a layer that reads another's cache; a row of no request
-  const int page = block_table[(size_t)entry * max_blocks + pos / page_size];
+  if (!kv_row) return;
   if (page < 0 || page >= n_pages) {
     if (threadIdx.x == 0) *status = NIB_STATUS_BAD_PAGE;
     return;
   }
-  const float* kv = src + q_rank;
-  s = 0.0f;
-  for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) s += kv[c] * kv[c];
-  const float rk = 1.0f / sqrtf(block_sum(s, scratch) / (float)kv_rank + eps);
+  const float rk = 1.0f / sqrtf(s2 / (float)kv_rank + eps);
   T* dst = cache + ((size_t)page * page_size + pos % page_size) * (size_t)(kv_rank + rot_dim);
   for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) dst[c] = from_float<T>(kv[c] * rk * wkv[c]);
   const float* kr = kv + kv_rank;
-  for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
-    double sn, cs;
-    sincos((double)pos * freqs[i], &sn, &cs);
-    const int iu = halves ? i : 2 * i, iv = halves ? i + rot_dims / 2 : 2 * i + 1;
-    const float u = kr[iu], v = kr[iv], c = (float)cs, sf = (float)sn;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const float c = lat_cs[2 * i], sf = lat_cs[2 * i + 1];
+    const int iu = halves ? i : 2 * i, iv = halves ? i + half : 2 * i + 1;
+    const float u = kr[iu], v = kr[iv];
     dst[kv_rank + iu] = from_float<T>(u * c - v * sf);
     dst[kv_rank + iv] = from_float<T>(v * c + u * sf);
   }
@@ -302,12 +323,14 @@ extern "C" int nib_latent_prep(int dtype, const float* proj, int ld, int q_rank,
   if (T <= 0) return 0;
   if (q_rank <= 0 || (has_kv && (kv_rank <= 0 || rot_dim < 0 || rot_dims > rot_dim || (rot_dims & 1))))
     return NIB_ERR_BAD_ARGUMENT;
+  const size_t smem = (size_t)(rot_dims > 0 ? rot_dims : 1) * sizeof(float);
+  if (smem > 40 * 1024) return NIB_ERR_UNSUPPORTED_SIZE;
   if (dtype == DT_F32)
-    launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(128), 0, stream, proj, ld, q_rank, kv_rank, rot_dim, rot_dims,
+    launch_pdl(latent_prep_kernel<float>, dim3(T), dim3(128), smem, stream, proj, ld, q_rank, kv_rank, rot_dim, rot_dims,
                freqs, wq, wkv, eps, (float*)cq, ld_cq, (float*)cache, block_table, max_blocks, row_entry, positions,
                page_size, n_pages, has_kv, halves, status);
   else if (dtype == DT_BF16)
-    launch_pdl(latent_prep_kernel<bf16>, dim3(T), dim3(128), 0, stream, proj, ld, q_rank, kv_rank, rot_dim, rot_dims,
+    launch_pdl(latent_prep_kernel<bf16>, dim3(T), dim3(128), smem, stream, proj, ld, q_rank, kv_rank, rot_dim, rot_dims,
                freqs, wq, wkv, eps, (bf16*)cq, ld_cq, (bf16*)cache, block_table, max_blocks, row_entry, positions,
                page_size, n_pages, has_kv, halves, status);
   else

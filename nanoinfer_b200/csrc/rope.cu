@@ -387,7 +387,8 @@ extern "C" int nib_rope_halves(float* rows, int ld, int q_off, int k_off, int n_
 namespace nib {
 
 // A warp owns one (head, map) of q or k, or one value head: sum of squares, weight, rotation in the halves layout (a
-// value meets its partner through the warp's piece of shared memory), cast, padding, and the cache write.
+// value meets its partner through the warp's piece of shared memory), cast, padding, and the cache write.  The row's sines
+// and cosines are made once a block, ahead of the wait.
 template <typename T>
 __global__ void __launch_bounds__(256)
 norm_rope_maps_append_kernel(const float* proj, int ld, int q_off, int k_off, int v_off, int n_head, int n_kv_head,
@@ -398,8 +399,17 @@ norm_rope_maps_append_kernel(const float* proj, int ld, int q_off, int k_off, in
                              int n_pages, int* status) {
   pdl_trigger();
   __shared__ float buf_sh[8][256];
+  __shared__ float cs_sh[128], sn_sh[128];
   const int t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   float* buf = buf_sh[warp];
+  const int half = rot_dims / 2;
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    double sd, cd;
+    sincos((double)positions[t] * freqs[j], &sd, &cd);
+    cs_sh[j] = (float)cd * amp;
+    sn_sh[j] = (float)sd * amp;
+  }
+  __syncthreads();
   const int u = blockIdx.x * (blockDim.x >> 5) + warp;
   const int nq = n_head * maps, nk = n_kv_head * maps;
   if (u >= nq + nk + n_kv_head) return;
@@ -416,21 +426,6 @@ norm_rope_maps_append_kernel(const float* proj, int ld, int q_off, int k_off, in
       if (lane == 0) *status = NIB_STATUS_BAD_PAGE;
     } else {
       dst = cache + kv_offset(page, is_k ? 0 : 1, is_k ? i / maps : i, pos % page_size, n_kv_head, page_size, hd);
-    }
-  }
-  // the rotation's angles do not wait for the projection
-  const int half = rot_dims / 2;
-  float cs[4], sn[4];
-  if (is_q || is_k) {
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const int j = lane + 32 * k;
-      if (j < half) {
-        double sd, cd;
-        sincos((double)pos * freqs[j], &sd, &cd);
-        cs[k] = (float)cd * amp;
-        sn[k] = (float)sd * amp;
-      }
     }
   }
   pdl_wait();
@@ -461,8 +456,8 @@ norm_rope_maps_append_kernel(const float* proj, int ld, int q_off, int k_off, in
     const int j = lane + 32 * k;
     if (j < half) {
       const float a = buf[j], b = buf[j + half];
-      buf[j] = a * cs[k] - b * sn[k];
-      buf[j + half] = b * cs[k] + a * sn[k];
+      buf[j] = a * cs_sh[j] - b * sn_sh[j];
+      buf[j + half] = b * cs_sh[j] + a * sn_sh[j];
     }
   }
   __syncwarp();

@@ -142,12 +142,14 @@ _SIGNATURES = {
     "nib_selective_scan": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
                            _c_ptr, _c_ptr, ctypes.c_longlong, ctypes.c_longlong, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
                            _c_ptr, _c_int, _c_ptr],
-    "nib_latent_prefill_tc_supported": [_c_int, _c_int, _c_int],
-    "nib_latent_prefill_tc": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int,
-                              _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr],
-    "nib_latent_decode_mma_supported": [_c_int, _c_int],
-    "nib_latent_decode_mma": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
-                              _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr],
+    "nib_attention_wide_tc_supported": [_c_int, _c_int, _c_int, _c_int, _c_int, _c_int],
+    "nib_attention_wide_tc": [_c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
+                              _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
+                              _c_int, _c_float, _c_ptr, _c_int, _c_ptr, _c_ptr],
+    "nib_attention_group_mma_supported": [_c_int, _c_int, _c_int, _c_int, _c_int],
+    "nib_attention_group_mma": [_c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
+                                _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float,
+                                _c_ptr, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int, _c_ptr],
     "nib_linear_heads_mma_supported": [_c_ptr, _c_int, _c_int, _c_ptr, _c_int],
     "nib_linear_heads_mma": [_c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                              _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
@@ -157,7 +159,7 @@ _SIGNATURES = {
     "nib_norm_rope_maps_append": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                   _c_int, _c_ptr, _c_ptr, _c_float, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_ptr, _c_int,
                                   _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
-    "nib_diff_combine": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int,
+    "nib_diff_combine": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int,
                          _c_int, _c_ptr],
     "nib_min_gru": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr,
                     _c_int, _c_int, _c_ptr, _c_int, _c_ptr],
@@ -209,8 +211,8 @@ class _Library:
         counted = name not in ("nib_linear_tc_supported", "nib_linear_tc_pair_supported", "nib_linear_skinny_supported",
                                "nib_attention_prefill_tc_supported", "nib_attention_prefill_supported",
                                "nib_attention_decode_mma_supported", "nib_attention_decode_mma_clusters",
-                               "nib_gated_scan_padded", "nib_latent_prefill_tc_supported",
-                               "nib_latent_decode_mma_supported", "nib_linear_heads_mma_supported")
+                               "nib_gated_scan_padded", "nib_attention_wide_tc_supported",
+                               "nib_attention_group_mma_supported", "nib_linear_heads_mma_supported")
 
         def call(*args):
             global _pending_op
@@ -670,22 +672,32 @@ class AttnExtras:
     sigmoid(gate[t, h]); ``out_scale``: and times this constant; ``span`` > 0: position i sees key j only if
     i // span == j // span (spans count from position 0 of the sequence); ``head_scale`` (float32 [n_head]): the
     scale times head_scale[h]; ``sinks`` (float32 [n_head]): with a sink, its term of the denominator is
-    exp(sinks[h]) instead of exp(0); ``out32``: the output is float32 whatever the dtype of queries and cache."""
+    exp(sinks[h]) instead of exp(0); ``out32``: the output is float32 whatever the dtype of queries and cache;
+    ``layout`` (maps, map size, values): not an option but what is known of the rows: query head h is zero outside the values
+    (h % maps) * size .. + size of its key row, and only the first so many values of a result are read."""
 
-    __slots__ = ("softcap", "keep_first", "slopes", "gate", "out_scale", "span", "head_scale", "sinks", "out32")
+    __slots__ = ("softcap", "keep_first", "slopes", "gate", "out_scale", "span", "head_scale", "sinks", "out32", "layout")
 
     def __init__(self, softcap: float = 0.0, keep_first: int = 0, slopes: Optional[torch.Tensor] = None,
                  gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, span: int = 0,
-                 head_scale: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, out32: bool = False):
+                 head_scale: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, out32: bool = False,
+                 layout: Optional[tuple] = None):
         self.softcap, self.keep_first, self.slopes = float(softcap), int(keep_first), slopes
         self.gate, self.out_scale = gate, float(out_scale)
         self.span, self.head_scale, self.sinks, self.out32 = int(span), head_scale, sinks, bool(out32)
+        self.layout = layout
 
     @property
     def plain(self) -> bool:
         return not (self.softcap > 0.0 or self.keep_first > 0 or self.slopes is not None or self.gate is not None
                     or self.out_scale != 1.0 or self.span > 0 or self.head_scale is not None or self.sinks is not None
                     or self.out32)
+
+    @property
+    def wide(self) -> bool:
+        """Whether the tcgen05 kernel for wide rows takes the options: a cap, a 32-bit output, no others."""
+        return not (self.keep_first > 0 or self.slopes is not None or self.gate is not None or self.out_scale != 1.0
+                    or self.span > 0 or self.head_scale is not None or self.sinks is not None)
 
     def args(self) -> tuple:
         g = self.gate
@@ -907,47 +919,115 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, b
                                            *(extras or _NO_EXTRAS).args(), _ptr(status), _stream()), "attention_prefill")
 
 
+def attention_wide_tc(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, out_head: int, block_table: torch.Tensor, ctx,
+                      plan, n_head: int, scale: float, window: int, maps: int, map_dim: int, v_cols: int,
+                      softcap: float = 0.0, gate: Optional[torch.Tensor] = None) -> bool:
+    """tcgen05 attention for the step's prompt portions over cached rows of any shape (csrc/attention_wide_tc.cu): ``cache``
+    [pages, planes, kv heads, page, row size] in bfloat16, planes 1 where a row is key and value at once; ``q`` heads of a
+    row's size; head h's first ``v_cols`` values go to column h * ``out_head`` of ``out`` (bfloat16 or float32).  False if a
+    size or an alignment is not taken."""
+    n_pages, planes, n_kv_head, page_size, row_dim = cache.shape
+    ldq = q.stride(0)
+    per = 3 if out.dtype == torch.float32 else 7
+    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or not scale > 0.0 or ldq % 8 or q.data_ptr() % 16 \
+            or cache.data_ptr() % 16 or out.data_ptr() % 16 or out.stride(0) & per or out_head & per \
+            or not _can("nib_attention_wide_tc_supported", row_dim, planes, maps, map_dim, v_cols, page_size):
+        return False
+    _check(library().nib_attention_wide_tc(
+        _ptr(q), ldq, ctx.n_rows, _ptr(cache), planes, _ptr(out), out.stride(0), int(out_head), int(out.dtype == torch.float32),
+        _ptr(block_table), block_table.shape[1], _ptr(plan.wide_tiles), plan.n_wide_tiles, _ptr(ctx.entry_start),
+        _ptr(ctx.entry_pos0), n_head, n_kv_head, row_dim, maps, map_dim, v_cols, page_size, n_pages, float(scale), int(window),
+        float(softcap), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(ctx.status), _stream()), "attention_wide_tc")
+    return True
+
+
+#: blocks of the grouped decode attention that fill the device about twice, and the most pieces of a row (one cluster)
+GROUP_BLOCKS, GROUP_MAX_SPLITS, GROUP_HEADS = 296, 16, 16
+
+
+def group_splits(n_rows: int, n_head: int, n_kv_head: int, max_keys: int) -> int:
+    """Into how many pieces (1, 2, 4, 8 or 16: the blocks of a cluster) the grouped kernel cuts each single token's keys:
+    while that leaves about two blocks an SM and pieces of more than half a tile of 64 keys."""
+    groups = n_kv_head * -(-(n_head // n_kv_head) // GROUP_HEADS)
+    splits = 1
+    while 2 * splits <= GROUP_MAX_SPLITS and 2 * splits * n_rows * groups <= GROUP_BLOCKS and splits * 64 < max_keys:
+        splits *= 2
+    return splits
+
+
+def attention_group_mma(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, out_head: int, block_table: torch.Tensor, ctx,
+                        plan, n_head: int, scale: float, window: int, k_cols: int, v_cols: int, softcap: float = 0.0,
+                        gate: Optional[torch.Tensor] = None, diff: Optional[tuple] = None,
+                        n_splits: Optional[int] = None) -> bool:
+    """Attention of the step's single tokens with the heads that share cached rows as the rows of an MMA tile
+    (csrc/attention_group_mma.cu); ``cache`` and ``q`` as in ``attention_wide_tc``, ``out`` bfloat16.  ``diff`` (lambda, eps,
+    factor): the heads come in pairs, and what is written for pair i, at column i * ``out_head``, is the normed difference of
+    its two results.  False if a size or an alignment is not taken."""
+    n_pages, planes, n_kv_head, page_size, row_dim = cache.shape
+    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or q.stride(0) % 8 \
+            or q.data_ptr() % 16 or cache.data_ptr() % 16 \
+            or not _can("nib_attention_group_mma_supported", row_dim, planes, k_cols, v_cols, int(diff is not None)):
+        return False
+    if n_splits is None:
+        keys = plan.max_decode_keys if window <= 0 else min(plan.max_decode_keys, window)
+        n_splits = group_splits(plan.n_decode, n_head, n_kv_head, keys)
+    lam, eps, mul = diff if diff is not None else (0.0, 0.0, 1.0)
+    _check(library().nib_attention_group_mma(
+        _ptr(q), q.stride(0), _ptr(cache), planes, _ptr(out), out.stride(0), int(out_head), _ptr(block_table),
+        block_table.shape[1], _ptr(plan.decode_rows), _ptr(ctx.row_entry), _ptr(ctx.positions), plan.n_decode, n_head, n_kv_head,
+        row_dim, k_cols, v_cols, page_size, n_pages, float(scale), int(window), float(softcap), _ptr(gate),
+        gate.stride(0) if gate is not None else 0, int(diff is not None), float(lam), float(eps), float(mul), _ptr(ctx.status),
+        int(n_splits), _stream()), "attention_group_mma")
+    return True
+
+
 def attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, ctx,
               n_head: int, scale: float, window: int, plan, sink: bool = False,
-              extras: Optional[AttnExtras] = None, sizes=None) -> None:
+              extras: Optional[AttnExtras] = None, sizes=None, single: bool = True) -> None:
     """Causal attention of the step's rows over one cache layer.  ``extras``: options on the scores and the output
-    (``AttnExtras``); the kernels that take them are the general one, the two of prompt portions and the streaming split-KV one.  ``sink``: the softmax's denominator has
-    one more term, exp(0) (a key of score 0 that has no value; every kernel adds it where it divides).
-    ``ctx`` is the step's StepContext, ``plan`` says which rows are single decoded tokens and how the
-    prompt portions are cut into tiles (``parts.attention.AttentionPlan``).  Single decoded tokens go to the split-KV kernel;
-    prompt portions go to the tiled tensor-core kernels in bfloat16 (head sizes 16..128 in steps of
-    16) and to the general kernel otherwise.  ``sizes`` (for the trace's counts only): the sizes of a head's key and
-    value and of a cached key row, where they are smaller than the cache's head size."""
+    (``AttnExtras``); the kernels that take them are the general one, the ones of prompt portions and the streaming
+    split-KV one.  ``sink``: the softmax's denominator has one more term, exp(0) (a key of score 0 that has no value; every
+    kernel that takes it adds it where it divides).  ``ctx`` is the step's StepContext, ``plan`` says which rows are single
+    decoded tokens and how the prompt portions are cut into tiles (``parts.attention.AttentionPlan``).  Single decoded tokens
+    (left out with ``single`` False: the caller has seen to them) go to the split-KV kernel; prompt portions in bfloat16 go to
+    the tensor cores: tcgen05 at head size 64, and, with a cap and a 32-bit output at most, at any other up to 256; the
+    warp-MMA kernel at head sizes 16..128 in steps of 16 with any options; everything else to the general kernel.  ``sizes``
+    (for the trace's counts only): the sizes of a head's key and value and of a cached key row, where they are smaller than
+    the cache's head size."""
     n_pages, _, n_kv_head, page_size, head_dim = cache.shape
     fast_pages = page_size % 16 == 0 and head_dim % 8 == 0 and head_dim <= 128
-    plain = extras is None or extras.plain
     traced = tracing()   # (the counts leave a window out: they are those of attention over all keys)
-    if not fast_pages:
-        if traced:
-            _note_attention(ctx.n_rows, plan.decode_keys + plan.prefill_keys, plan.decode_keys + plan.prefill_kv_rows,
-                            n_head, n_kv_head, head_dim, q.element_size(), sizes, out.element_size())
-        attention_simt(q, cache, out, block_table, ctx.row_entry, ctx.positions, ctx.n_rows, n_head, scale,
-                       window, ctx.status, sink=sink, extras=extras)
-        return
-    if plan.n_decode:
+    n_decode, n_portion = plan.n_decode if single else 0, plan.n_prefill_rows
+    layout = extras.layout if extras is not None and extras.layout is not None else None
+    if n_decode:
         keys = plan.max_decode_keys if window <= 0 else min(plan.max_decode_keys, window)
         if extras is not None and extras.span > 0:
             keys = min(keys, extras.span)
         if traced:
-            _note_attention(plan.n_decode, plan.decode_keys, plan.decode_keys, n_head, n_kv_head, head_dim,
+            _note_attention(n_decode, plan.decode_keys, plan.decode_keys, n_head, n_kv_head, head_dim,
                             q.element_size(), sizes, out.element_size())
-        attention_decode(q, cache, out, block_table, ctx.row_entry, ctx.positions, plan.n_decode, n_head, scale,
-                         window, ctx.status, keys, ctx.workspace, plan.decode_rows, sink=sink, extras=extras)
-    if plan.n_prefill_rows:
+        if fast_pages:
+            attention_decode(q, cache, out, block_table, ctx.row_entry, ctx.positions, n_decode, n_head, scale,
+                             window, ctx.status, keys, ctx.workspace, plan.decode_rows, sink=sink, extras=extras)
+        else:
+            attention_simt(q, cache, out, block_table, ctx.row_entry, ctx.positions, n_decode, n_head, scale, window,
+                           ctx.status, plan.decode_rows, sink=sink, extras=extras)
+    if n_portion:
         if traced:
-            _note_attention(plan.n_prefill_rows, plan.prefill_keys, plan.prefill_kv_rows, n_head, n_kv_head, head_dim,
+            _note_attention(n_portion, plan.prefill_keys, plan.prefill_kv_rows, n_head, n_kv_head, head_dim,
                             q.element_size(), sizes, out.element_size())
-        if q.dtype == torch.bfloat16 and scale > 0 and _can("nib_attention_prefill_tc_supported", head_dim, page_size) \
+        maps, map_dim, v_cols = layout if layout is not None else (1, head_dim, head_dim)
+        if q.dtype == torch.bfloat16 and (layout is not None or head_dim > 64) and not sink and (extras is None or extras.wide) \
+                and attention_wide_tc(q, cache, out, head_dim, block_table, ctx, plan, n_head, scale, window, maps, map_dim,
+                                      v_cols, softcap=extras.softcap if extras is not None else 0.0):
+            pass
+        elif fast_pages and q.dtype == torch.bfloat16 and scale > 0 \
+                and _can("nib_attention_prefill_tc_supported", head_dim, page_size) \
                 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0 \
                 and out.data_ptr() % 16 == 0:
             attention_prefill_tc(q, cache, out, block_table, plan.wide_tiles, plan.n_wide_tiles, ctx.entry_start,
                                  ctx.entry_pos0, ctx.n_rows, n_head, scale, window, ctx.status, sink=sink, extras=extras)
-        elif q.dtype == torch.bfloat16 and scale > 0 and _can("nib_attention_prefill_supported", head_dim) \
+        elif fast_pages and q.dtype == torch.bfloat16 and scale > 0 and _can("nib_attention_prefill_supported", head_dim) \
                 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0:
             attention_prefill(q, cache, out, block_table, plan.tiles, plan.n_tiles, ctx.entry_start, ctx.entry_pos0,
                               n_head, scale, window, ctx.status, sink=sink, extras=extras)
@@ -955,8 +1035,32 @@ def attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_tab
             # (portions alone: all of the step's rows, those of no request among them, which the kernel leaves out;
             # the launch then depends on the step's shape only, as a graph needs it)
             attention_simt(q, cache, out, block_table, ctx.row_entry, ctx.positions,
-                           plan.n_prefill_rows if plan.n_decode else ctx.n_rows, n_head, scale, window, ctx.status,
+                           n_portion if plan.n_decode else ctx.n_rows, n_head, scale, window, ctx.status,
                            plan.prefill_rows, sink=sink, extras=extras)
+
+
+def differential_attention(q: torch.Tensor, cache: torch.Tensor, maps_out: torch.Tensor, out: torch.Tensor,
+                           block_table: torch.Tensor, ctx, n_head: int, dim: int, vdim: int, scale: float, window: int,
+                           softcap: float, lam: float, eps: float, mul: float, plan) -> None:
+    """Both maps of every head over one cache layer and their normed difference into ``out`` [rows, >= n_head * vdim]: q holds
+    2 * n_head heads of the cache's size (``norm_rope_maps_append``), ``maps_out`` (float32, the shape of q) is scratch for
+    the maps' results.  In bfloat16 single tokens have the difference made where their pieces of keys are merged; otherwise,
+    and for prompt portions, it is a kernel of its own behind the attention."""
+    row_dim = cache.shape[4]
+    sizes = (dim, vdim, 2 * dim)
+    v8 = -(-vdim // 8) * 8
+    done = False
+    if plan.n_decode and q.dtype == torch.bfloat16:
+        if tracing():
+            _note_attention(plan.n_decode, plan.decode_keys, plan.decode_keys, 2 * n_head, cache.shape[2], row_dim,
+                            q.element_size(), sizes, out.element_size())
+        done = attention_group_mma(q, cache, out, vdim, block_table, ctx, plan, 2 * n_head, scale, window, 2 * dim, vdim,
+                                   softcap=softcap, diff=(lam, eps, mul))
+    if plan.n_prefill_rows or not done:
+        attention(q, cache, maps_out, block_table, ctx, 2 * n_head, scale, window, plan,
+                  extras=AttnExtras(softcap=softcap, out32=True, layout=(2, dim, v8)), sizes=sizes, single=not done)
+        rows, n = (plan.prefill_rows, plan.n_prefill_rows) if done else (None, ctx.n_rows)
+        diff_combine(maps_out, n_head, vdim, lam, eps, mul, out, n, rows)
 
 
 _SRC_CODES = {torch.float32: 0, torch.bfloat16: 1, torch.float16: 2}
@@ -1145,18 +1249,7 @@ def latent_attention_reserve(workspace, n_head: int, kv_rank: int) -> None:
     workspace.reserve("latent.partials", LATENT_BLOCKS * LATENT_HEADS_PER_BLOCK * (kv_rank + 2), torch.float32)
 
 
-def latent_decode_splits(n_rows: int, n_head: int, max_keys: int) -> int:
-    """Into how many pieces (1, 2, 4, 8 or 16: the blocks of a cluster) the MMA kernel cuts each single token's keys:
-    about two blocks an SM, pieces of at least a tile of 64 keys."""
-    groups = -(-n_head // 16)
-    want = min(LATENT_MAX_SPLITS, LATENT_BLOCKS // max(1, n_rows * groups), -(-max_keys // 64))
-    splits = 1
-    while 2 * splits <= want:
-        splits *= 2
-    return splits
-
-
-def _latent_keys(plan, ctx, window: int, single: bool) -> int:
+def _latent_keys(ctx, window: int, single: bool) -> int:
     """Keys seen by the step's single tokens, or by its portions' rows (for the trace's counts)."""
     keys = 0
     for e, p0 in enumerate(ctx.host_entry_pos0):
@@ -1181,46 +1274,31 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
     if out.dtype != cache.dtype or out.stride(1) != 1 or q.shape[2] != D:
         raise KernelError("latent_attention: out in the cache's dtype, q [T, heads, D]")
     gate_args = (_ptr(gate), gate.stride(0) if gate is not None else 0)
-    if plan is not None and q.dtype == torch.bfloat16 and scale > 0 and n_splits is None:
+    if plan is not None and q.dtype == torch.bfloat16 and n_splits is None:
         # on the tensor cores where the sizes allow; what they do not take goes to the general kernel by lists of rows
-        lib, e = library(), q.element_size()
-        ok = q.data_ptr() % 16 == 0 and cache.data_ptr() % 16 == 0
-        todo = []
+        e, todo = q.element_size(), []
+        q2 = q.view(q.shape[0], n_head * D)
         if plan.n_decode:
             if tracing():
-                keys = _latent_keys(plan, ctx, window, True)
+                keys = _latent_keys(ctx, window, True)
                 _note("attn", "latent_attn", (plan.n_decode, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
                       e * (plan.n_decode * n_head * (D + kv_rank) + keys * D))
-            if ok and _can("nib_latent_decode_mma_supported", kv_rank, D):
-                splits = latent_decode_splits(plan.n_decode, n_head, plan.max_decode_keys if window <= 0 else
-                                              min(plan.max_decode_keys, window))
-                _check(lib.nib_latent_decode_mma(_ptr(q), _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
-                                                 block_table.shape[1], _ptr(plan.decode_rows), _ptr(ctx.row_entry),
-                                                 _ptr(ctx.positions), plan.n_decode, n_head, kv_rank, D, page_size, n_pages,
-                                                 float(scale), int(window), *gate_args, _ptr(ctx.status), splits, _stream()),
-                       "latent_decode_mma")
-            else:
+            if not attention_group_mma(q2, cache, out, kv_rank, block_table, ctx, plan, n_head, scale, window, D, kv_rank, gate=gate):
                 todo.append((plan.decode_rows, plan.n_decode))
         if plan.n_prefill_rows:
             if tracing():
-                keys = _latent_keys(plan, ctx, window, False)
+                keys = _latent_keys(ctx, window, False)
                 _note("attn", "latent_attn", (plan.n_prefill_rows, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
                       e * (plan.n_prefill_rows * n_head * (D + kv_rank) + plan.prefill_kv_rows * D))
-            if ok and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0 \
-                    and _can("nib_latent_prefill_tc_supported", kv_rank, D, page_size):
-                _check(lib.nib_latent_prefill_tc(_ptr(q), ctx.n_rows, _ptr(cache), _ptr(out), out.stride(0), _ptr(block_table),
-                                                 block_table.shape[1], _ptr(plan.wide_tiles), plan.n_wide_tiles,
-                                                 _ptr(ctx.entry_start), _ptr(ctx.entry_pos0), n_head, kv_rank, D, page_size,
-                                                 n_pages, float(scale), int(window), *gate_args, _ptr(ctx.status), _stream()),
-                       "latent_prefill_tc")
-            else:
+            if not attention_wide_tc(q2, cache, out, kv_rank, block_table, ctx, plan, n_head, scale, window, 1, D, kv_rank, gate=gate):
                 # (portions alone: all of the step's rows, those of no request among them, which the kernel leaves out)
                 todo.append((plan.prefill_rows, plan.n_prefill_rows if plan.n_decode else ctx.n_rows))
         for rows, n in todo:
-            _check(lib.nib_latent_attention(_dt(cache), _dt(q), _ptr(q), _ptr(cache), _ptr(out), out.stride(0),
-                                            _ptr(block_table), block_table.shape[1], _ptr(rows), _ptr(ctx.row_entry),
-                                            _ptr(ctx.positions), n, n_head, kv_rank, D, page_size, n_pages, float(scale),
-                                            int(window), *gate_args, _ptr(ctx.status), 1, None, _stream()), "latent_attention")
+            _check(library().nib_latent_attention(_dt(cache), _dt(q), _ptr(q), _ptr(cache), _ptr(out), out.stride(0),
+                                                  _ptr(block_table), block_table.shape[1], _ptr(rows), _ptr(ctx.row_entry),
+                                                  _ptr(ctx.positions), n, n_head, kv_rank, D, page_size, n_pages, float(scale),
+                                                  int(window), *gate_args, _ptr(ctx.status), 1, None, _stream()),
+                   "latent_attention")
         return
     if n_splits is None:
         n_splits = latent_splits(ctx.n_rows, n_head)
@@ -1942,16 +2020,18 @@ def norm_rope_maps_append(proj: torch.Tensor, offsets, n_head: int, n_kv_head: i
 
 
 def diff_combine(a: torch.Tensor, n_head: int, vdim: int, lam: float, eps: float, mul: float, out: torch.Tensor,
-                 n_rows: int) -> None:
+                 n_rows: int, rows: Optional[torch.Tensor] = None) -> None:
     """out[t, h * vdim + d] = mul * o_d / sqrt(mean(o^2) + eps), o = a[t, 2h] - lam * a[t, 2h + 1] over the first ``vdim``
-    values of the 32-bit heads ``a`` [rows, 2 * n_head * head size]."""
+    values of the 32-bit heads ``a`` [rows, 2 * n_head * head size].  ``rows`` lists the ``n_rows`` rows to process."""
+    if rows is not None:
+        _i32(rows, "rows")
     if a.dtype != torch.float32 or a.stride(1) != 1 or out.stride(1) != 1 or a.shape[1] % (2 * n_head) \
             or out.shape[1] < n_head * vdim:
         raise KernelError("diff_combine: a float32 [rows, 2 * heads * head size], out [rows, >= heads * vdim]")
     if tracing():
         n = n_head * vdim
         _note("other", "diff_combine", (n_rows, n, 0), 6.0 * n_rows * n, n_rows * n * (8.0 + out.element_size()))
-    _check(library().nib_diff_combine(_dt(out), _ptr(a), a.stride(0), n_head, a.shape[1] // (2 * n_head), vdim, float(lam),
+    _check(library().nib_diff_combine(_dt(out), _ptr(a), a.stride(0), _ptr(rows), n_head, a.shape[1] // (2 * n_head), vdim, float(lam),
                                       float(eps), float(mul), _ptr(out), out.stride(0), n_rows, _stream()), "diff_combine")
 
 

@@ -111,7 +111,5 @@ class DifferentialAttention(TwoProducts, Mixer):
         if plan is None:
             plan = ctx.plans["causal_attention"] = AttentionPlan(ctx.host_entry_start, ctx.host_entry_pos0,
                                                                  device=proj.device)
-        ops.attention(q, cache.layer, maps, cache.block_table, ctx, H * MAPS, self.scale, self.window, plan,
-                      extras=ops.AttnExtras(softcap=self.softcap, out32=True),
-                      sizes=(self.head_dim, self.v_dim, MAPS * self.head_dim))
-        ops.diff_combine(maps, H, self.v_dim, self.lam, self.eps, 1.0 - self.diff, out, ctx.n_rows)
+        ops.differential_attention(q, cache.layer, maps, out, cache.block_table, ctx, H, self.head_dim, self.v_dim, self.scale,
+                                   self.window, self.softcap, self.lam, self.eps, 1.0 - self.diff, plan)

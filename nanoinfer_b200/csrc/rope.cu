@@ -410,62 +410,66 @@ norm_rope_maps_append_kernel(const float* proj, int ld, int q_off, int k_off, in
     sn_sh[j] = (float)sd * amp;
   }
   __syncthreads();
-  const int u = blockIdx.x * (blockDim.x >> 5) + warp;
-  const int nq = n_head * maps, nk = n_kv_head * maps;
-  if (u >= nq + nk + n_kv_head) return;
+  const int nq = n_head * maps, nk = n_kv_head * maps, n_warps = blockDim.x >> 5;
   const int pos = positions[t], entry = row_entry[t];
-  const bool is_q = u < nq, is_k = !is_q && u < nq + nk;
-  const int i = is_q ? u : (is_k ? u - nq : u - nq - nk);          // index of the (head, map), or of the value head
-  const int m = is_q || is_k ? i % maps : 0;
-  T* dst = nullptr;
-  if (is_q) {
-    dst = q_out + (size_t)t * ldq + (size_t)i * hd;
-  } else if (entry >= 0 && cache != nullptr) {
-    const int page = block_table[(size_t)entry * max_blocks + pos / page_size];
+  int page = -1;
+  if (entry >= 0 && cache != nullptr) {
+    page = block_table[(size_t)entry * max_blocks + pos / page_size];
     if (page < 0 || page >= n_pages) {
-      if (lane == 0) *status = NIB_STATUS_BAD_PAGE;
-    } else {
-      dst = cache + kv_offset(page, is_k ? 0 : 1, is_k ? i / maps : i, pos % page_size, n_kv_head, page_size, hd);
+      if (threadIdx.x == 0) *status = NIB_STATUS_BAD_PAGE;
+      page = -1;
     }
   }
   pdl_wait();
-  if (dst == nullptr) return;
-  if (!is_q && !is_k) {
-    const float* src = proj + (size_t)t * ld + v_off + (size_t)i * vdim;
-    for (int c = lane; c < hd; c += 32) dst[c] = from_float<T>(c < vdim ? src[c] : 0.0f);
-    return;
-  }
-  const float* src = proj + (size_t)t * ld + (is_q ? q_off : k_off) + (size_t)i * dim;
-  const float* w = is_q ? wq : wk;
-  float x[8], ss = 0.0f;
-#pragma unroll
-  for (int k = 0; k < 8; ++k) {
-    const int c = lane + 32 * k;
-    x[k] = c < dim ? src[c] : 0.0f;
-    ss += x[k] * x[k];
-  }
-  const float r = w != nullptr ? 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps) : 1.0f;
-#pragma unroll
-  for (int k = 0; k < 8; ++k) {
-    const int c = lane + 32 * k;
-    if (c < dim) buf[c] = w != nullptr ? x[k] * r * w[c] : x[k];
-  }
-  __syncwarp();
-#pragma unroll
-  for (int k = 0; k < 4; ++k) {
-    const int j = lane + 32 * k;
-    if (j < half) {
-      const float a = buf[j], b = buf[j + half];
-      buf[j] = a * cs_sh[j] - b * sn_sh[j];
-      buf[j + half] = b * cs_sh[j] + a * sn_sh[j];
+  for (int u = blockIdx.x * n_warps + warp; u < nq + nk + n_kv_head; u += gridDim.x * n_warps) {
+    const bool is_q = u < nq, is_k = !is_q && u < nq + nk;
+    const int i = is_q ? u : (is_k ? u - nq : u - nq - nk);          // index of the (head, map), or of the value head
+    const int m = is_q || is_k ? i % maps : 0;
+    T* dst = nullptr;
+    if (is_q) {
+      dst = q_out + (size_t)t * ldq + (size_t)i * hd;
+    } else if (page >= 0) {
+      dst = cache + kv_offset(page, is_k ? 0 : 1, is_k ? i / maps : i, pos % page_size, n_kv_head, page_size, hd);
     }
-  }
-  __syncwarp();
-  // a query owns its whole head of hd values; a key its map's place, the last map's also what lies behind it
-  const int c_begin = is_q ? 0 : m * dim, c_end = is_q || m == maps - 1 ? hd : (m + 1) * dim;
-  for (int c = c_begin + lane; c < c_end; c += 32) {
-    const int d = c - m * dim;
-    dst[c] = from_float<T>(d >= 0 && d < dim ? buf[d] : 0.0f);
+    if (dst == nullptr) continue;
+    if (!is_q && !is_k) {
+      const float* src = proj + (size_t)t * ld + v_off + (size_t)i * vdim;
+      for (int c = lane; c < hd; c += 32) dst[c] = from_float<T>(c < vdim ? src[c] : 0.0f);
+      continue;
+    }
+    const float* src = proj + (size_t)t * ld + (is_q ? q_off : k_off) + (size_t)i * dim;
+    const float* w = is_q ? wq : wk;
+    float x[8], ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int c = lane + 32 * k;
+      x[k] = c < dim ? src[c] : 0.0f;
+      ss += x[k] * x[k];
+    }
+    const float r = w != nullptr ? 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps) : 1.0f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int c = lane + 32 * k;
+      if (c < dim) buf[c] = w != nullptr ? x[k] * r * w[c] : x[k];
+    }
+    __syncwarp();
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int j = lane + 32 * k;
+      if (j < half) {
+        const float a = buf[j], b = buf[j + half];
+        buf[j] = a * cs_sh[j] - b * sn_sh[j];
+        buf[j + half] = b * cs_sh[j] + a * sn_sh[j];
+      }
+    }
+    __syncwarp();
+    // a query owns its whole head of hd values; a key its map's place, the last map's also what lies behind it
+    const int c_begin = is_q ? 0 : m * dim, c_end = is_q || m == maps - 1 ? hd : (m + 1) * dim;
+    for (int c = c_begin + lane; c < c_end; c += 32) {
+      const int d = c - m * dim;
+      dst[c] = from_float<T>(d >= 0 && d < dim ? buf[d] : 0.0f);
+    }
+    __syncwarp();          // (the next head's values go where these were read)
   }
 }
 
@@ -485,7 +489,8 @@ extern "C" int nib_norm_rope_maps_append(int dtype, const float* proj, int ld, i
   if (dim > 256 || T > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
   const int total = (n_head + n_kv_head) * maps + n_kv_head;
   const int warps = total < 8 ? total : 8;
-  const dim3 grid((total + warps - 1) / warps, T), block(32 * warps);
+  // (steps of many rows: one block a row, which makes the row's angles once; few rows: a warp for every head)
+  const dim3 grid(T >= 128 ? 1 : (total + warps - 1) / warps, T), block(32 * warps);
   if (dtype == DT_F32)
     launch_pdl(norm_rope_maps_append_kernel<float>, grid, block, 0, stream, proj, ld, q_off, k_off, v_off, n_head,
                n_kv_head, maps, dim, vdim, hd, wq, wk, eps, rot_dims, freqs, amp, positions, row_entry, (float*)q_out, ldq,

@@ -256,16 +256,78 @@ def test_one_matching_key_of_either_map_just_inside_and_just_outside_the_window(
                 c = min(page, n - b * page)
                 cache[perm[b], 0, 0, :c], cache[perm[b], 1, 0, :c] = k[b * page:b * page + c], v[b * page:b * page + c]
             ctx = step_ctx([rows], list(range(n - rows, n)))
-            out = torch.zeros(rows, 2 * hd, device=DEV)
             plan = AttentionPlan(ctx.host_entry_start, ctx.host_entry_pos0, device=torch.device(DEV))
-            ops.attention(q.view(rows, -1).to(dt).to(DEV), cache.to(dt).to(DEV), out, torch.tensor([perm], dtype=torch.int32, device=DEV),
-                          ctx, 2, 1.0, window, plan, extras=ops.AttnExtras(softcap=25.0, out32=True))
-            for i in (0, rows - 1):
-                p = n - rows + i
-                visible = 0 <= p - far < window
-                found, other = float(out[i, m * hd + 2]) > 0.9, float(out[i, (1 - m) * hd + 2])
-                assert found == visible, f"map {m}, key {far}, row at {p}: visible {visible}, found {found}"
-                assert other < (1.01 if window == 1 else 0.55 if window == 2 else 0.2)
+            table = torch.tensor([perm], dtype=torch.int32, device=DEV)
+            qd, cd = q.view(rows, -1).to(dt).to(DEV), cache.to(dt).to(DEV)
+            for layout in (None, (2, dim, hd)):         # (with the layout known, bfloat16 portions take the kernel for wide rows)
+                out = torch.zeros(rows, 2 * hd, device=DEV)
+                ops.attention(qd, cd, out, table, ctx, 2, 1.0, window, plan, extras=ops.AttnExtras(softcap=25.0, out32=True, layout=layout))
+                for i in (0, rows - 1):
+                    p = n - rows + i
+                    visible = 0 <= p - far < window
+                    found, other = float(out[i, m * hd + 2]) > 0.9, float(out[i, (1 - m) * hd + 2])
+                    assert found == visible, f"map {m}, key {far}, row at {p}: visible {visible}, found {found}"
+                    assert other < (1.01 if window == 1 else 0.55 if window == 2 else 0.2)
+            if dtype == "bfloat16" and rows == 1:       # ... and single tokens the grouped kernel, in one piece and in four
+                for splits in (1, 4):
+                    got = torch.zeros(1, 2 * hd, device=DEV, dtype=dt)
+                    assert ops.attention_group_mma(qd, cd, got, hd, table, ctx, plan, 2, 1.0, window, 2 * dim, hd, softcap=25.0, n_splits=splits)
+                    assert (float(got[0, m * hd + 2]) > 0.9) == (0 <= n - 1 - far < window)
+
+
+DIFF_CASES = [(4, 2, 16, 40, 48), (3, 1, 64, 128, 128), (2, 2, 9, 21, 32), (12, 1, 24, 48, 48), (2, 1, 100, 200, 208), (3, 3, 32, 64, 64),
+              (1, 1, 128, 256, 256), (5, 5, 40, 8, 80)]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("window,cap", [(0, 0.0), (70, 6.0), (1, 30.0)])
+@pytest.mark.parametrize("H,G,dim,vdim,hd", DIFF_CASES)
+def test_both_maps_and_their_normed_difference(H, G, dim, vdim, hd, window, cap, dtype):
+    """Portions beside single tokens, and single tokens alone with their keys in 1 to 16 pieces: in bfloat16 the tcgen05 kernel
+    for wide rows and the grouped one; pages behind the window are gone."""
+    from nanoinfer_b200.kernels import ops
+    from nanoinfer_b200.parts.attention import AttentionPlan
+
+    dt, page, scale, lam, eps, mul = DT[dtype], 16, 1.3 / math.sqrt(dim), 0.7, 1e-4, 0.6
+    for lengths, q_rows in (([200, 77, 450, 130, 16, 3, 333], [130, 1, 1, 40, 16, 2, 290]), ([450, 77, 2, 64], [1] * 4), ([1000], [1])):
+        cache, table, ks, vs, _ = _paged(dt, 2 * H, G, hd, page, lengths, q_rows, seed=hd)
+        cache[:, 0, :, :, 2 * dim:], cache[:, 1, :, :, vdim:] = 0.0, 0.0
+        for e, (n, r) in enumerate(zip(lengths, q_rows)):
+            for b in range(n // page):
+                if window and (b + 1) * page <= n - r - window + 1:
+                    table[e, b] = -1
+        g = torch.Generator().manual_seed(dim)
+        T = sum(q_rows)
+        q = torch.randn(T, H, 2, dim, generator=g).to(dt).float()
+        laid = torch.zeros(T, H, 2, hd)
+        laid[:, :, 0, :dim], laid[:, :, 1, dim:2 * dim] = q[:, :, 0], q[:, :, 1]
+        ctx = step_ctx(q_rows, [p for n, r in zip(lengths, q_rows) for p in range(n - r, n)])
+        at, want = 0, []
+        for n, r, k, v in zip(lengths, q_rows, ks, vs):
+            a = [_windowed(q[at:at + r, :, m], k[..., m * dim:(m + 1) * dim], v[..., :vdim], scale, n - r, window, cap) for m in (0, 1)]
+            o = a[0] - lam * a[1]
+            want.append((o / torch.sqrt((o ** 2).mean(-1, keepdim=True) + eps) * mul).reshape(r, H * vdim))
+            at += r
+        want = torch.cat(want)
+        plan = AttentionPlan(ctx.host_entry_start, ctx.host_entry_pos0, device=torch.device(DEV))
+        qd, cd, td = laid.view(T, -1).to(dt).to(DEV), cache.to(dt).to(DEV), table.to(DEV)
+        maps = torch.full((T, 2 * H * hd), 7.0, device=DEV)
+        tol = 1e-4 if dtype == "float32" else 5e-2
+
+        def check(out, what):
+            assert int(ctx.status.item()) == 0
+            err = (out[:, :H * vdim].double().cpu() - want).abs()
+            assert float(err.max()) < tol, (lengths, what, float(err.max()))
+            assert float(out[:, H * vdim:].float().min()) == 7.0
+        out = torch.full((T, H * vdim + 6), 7.0, device=DEV, dtype=dt)
+        ops.differential_attention(qd, cd, maps, out, td, ctx, H, dim, vdim, scale, window, cap, lam, eps, mul, plan)
+        check(out, "as the step runs it")
+        if dtype == "bfloat16" and plan.n_prefill_rows == 0:
+            for splits in (1, 2, 4, 8, 16):
+                out.fill_(7.0)
+                assert ops.attention_group_mma(qd, cd, out, vdim, td, ctx, plan, 2 * H, scale, window, 2 * dim, vdim, softcap=cap,
+                                               diff=(lam, eps, mul), n_splits=splits)
+                check(out, f"{splits} pieces")
 
 
 def _latent_reference(q, lat, kv_rank, scale, positions, gate, window=0):

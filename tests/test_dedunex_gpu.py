@@ -359,7 +359,7 @@ def _latent_cache(lats, page, D, seed, dt, gone_behind=None):
 
 
 LATENT_CASES = [(3, 32, 8, 16), (9, 64, 16, 16), (1, 20, 6, 32), (12, 128, 32, 48), (4, 256, 32, 16), (2, 512, 64, 16), (17, 96, 24, 16),
-                (5, 256, 64, 32), (40, 16, 8, 16), (2, 8, 0, 16), (3, 200, 40, 16)]
+                (5, 256, 64, 32), (40, 16, 8, 16), (2, 8, 0, 16), (3, 200, 40, 16), (2, 256, 128, 16), (3, 336, 48, 16)]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])

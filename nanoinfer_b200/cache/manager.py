@@ -12,7 +12,9 @@ Beyond the reference:
     group has a page pool, a device tensor and block tables of its own, so a group that keeps a
     window of keys gives pages back as the window passes them while another keeps all keys; a
     window may keep a request's first positions readable behind it (``KVCacheSpec.keep_first``):
-    the pages that hold them stay with the request until it ends;
+    the pages that hold them stay with the request until it ends; and it may keep one POOLED row for every
+    whole block of positions (``KVCacheSpec.pool``), in pages of their own out of the same pool, listed
+    behind the positions' pages in the request's block table row;
   * a step's allocation is all-or-nothing (the reference leaves a partial allocation behind
     when the pool runs out, batch.rs:243-254);
   * every request owns one STATE SLOT: an index into per-slot tensors of fixed size (a mixer's
@@ -106,13 +108,15 @@ class RequestCache:
     slot: int
     n_tokens: int = 0
     blocks: List[List[int]] = field(default_factory=list)
+    #: per group, the pages of the request's pooled rows, in order (empty where the group keeps none)
+    pooled: List[List[int]] = field(default_factory=list)
     live: bool = True
     #: per group, the block table row as the device wants it (int32 [max_blocks], -1 = no page):
-    #: a mirror of ``blocks`` kept by the manager so that a step copies it in one piece
+    #: a mirror of ``blocks`` and, from column ``pool_column`` of the group on, of ``pooled``, kept by the manager so that a step copies it in one piece
     table_rows: List[np.ndarray] = field(default_factory=list)
 
     def pages_held(self) -> int:
-        return sum(1 for g in self.blocks for p in g if p >= 0)
+        return sum(1 for g in self.blocks for p in g if p >= 0) + sum(len(g) for g in self.pooled)
 
 
 class StateSlots:
@@ -173,7 +177,8 @@ class CacheManager:
                  max_positions: Optional[int] = None, pages_per_group: Optional[Sequence[int]] = None,
                  padding: bool = False):
         """``max_tokens``: how many tokens live requests may hold together, each request's count
-        rounded up to whole pages; every group's pool gets ``ceil(max_tokens / page_size)`` pages
+        rounded up to whole pages; every group's pool gets ``ceil(max_tokens / page_size)`` pages (and
+        what the pooled rows of so many tokens take, where the group keeps some)
         unless ``pages_per_group`` says otherwise.  ``device`` None: bookkeeping only.
         ``padding``: one page per group and one state slot more than the pools hand out
         (``pad_page``, ``pad_slot``): the step function points the rows there with which it pads a
@@ -189,7 +194,8 @@ class CacheManager:
             by_spec.setdefault(spec, []).append(idx)
         self.groups: List[CacheGroup] = []
         for gi, (spec, owners) in enumerate(by_spec.items()):
-            n_pages = int(pages_per_group[gi]) if pages_per_group is not None else n_default
+            n_pages = int(pages_per_group[gi]) if pages_per_group is not None else n_default + (
+                -(-n_default // spec.pool) + int(max_requests) if spec.pool > 0 else 0)
             group = CacheGroup(spec, owners, self.page_size, PagePool(n_pages))
             if device is not None:
                 group.tensor = torch.zeros(
@@ -208,7 +214,10 @@ class CacheManager:
         self._state_keys = [("state", idx) for idx, _ in state_needs]
         self._live: List[RequestCache] = []
         # the longest block table a request can have, per group
-        self.max_blocks = [self._max_blocks(g) for g in self.groups]
+        longest = [self._max_blocks(g) for g in self.groups]
+        #: where the pages of pooled rows begin in a group's block table rows (behind those of the positions)
+        self.pool_column = longest
+        self.max_blocks = [n + self._pool_columns(g, n) for g, n in zip(self.groups, longest)]
         #: goes up whenever a group's block tables had to be made longer (``_grow_tables``): whoever sized
         #: buffers by ``max_blocks`` compares it before a step
         self.table_generation = 0
@@ -217,16 +226,26 @@ class CacheManager:
         limit = self.max_positions if self.max_positions is not None else g.pool.n_pages * self.page_size
         return max(1, -(-limit // self.page_size))
 
+    def _pool_columns(self, g: CacheGroup, n_blocks: int) -> int:
+        """Pages that the pooled rows of ``n_blocks`` pages of positions can take."""
+        return max(1, self._pool_pages(g, n_blocks * self.page_size)) if g.spec.pool > 0 else 0
+
+    def _pool_pages(self, g: CacheGroup, n_tokens: int) -> int:
+        """Pages that hold the pooled rows of a request's first ``n_tokens`` positions (one row a whole block)."""
+        return -(-(n_tokens // g.spec.pool) // self.page_size) if g.spec.pool > 0 else 0
+
     def _grow_tables(self, gi: int, n_blocks: int) -> None:
         """A model without a position limit, a group that keeps a window of keys: a request may become longer
         than the whole pool holds (pages behind the window go back), so its block table, one entry per
         logical block from position 0 on, outgrows what the pool's size gave it.  The tables of the group
         are then made at least twice as long."""
-        new = max(2 * self.max_blocks[gi], n_blocks)
-        self.max_blocks[gi] = new
+        new = max(2 * self.pool_column[gi], n_blocks)
+        self.pool_column[gi] = new
+        self.max_blocks[gi] = new + self._pool_columns(self.groups[gi], new)
         for r in self._live:
-            row = np.full(new, -1, dtype=np.int32)
-            row[:len(r.table_rows[gi])] = r.table_rows[gi]
+            row = np.full(self.max_blocks[gi], -1, dtype=np.int32)
+            row[:len(r.blocks[gi])] = r.blocks[gi]
+            row[new:new + len(r.pooled[gi])] = r.pooled[gi]
             r.table_rows[gi] = row
         self.table_generation += 1
 
@@ -234,7 +253,7 @@ class CacheManager:
     def open_request(self) -> RequestCache:
         slot = self.slots.take()
         self.slots.reset(slot, self._state_keys)
-        req = RequestCache(slot=slot, blocks=[[] for _ in self.groups],
+        req = RequestCache(slot=slot, blocks=[[] for _ in self.groups], pooled=[[] for _ in self.groups],
                            table_rows=[np.full(mb, -1, dtype=np.int32) for mb in self.max_blocks])
         self._live.append(req)
         return req
@@ -242,11 +261,12 @@ class CacheManager:
     def close_request(self, req: RequestCache) -> None:
         """Give back everything the request holds."""
         self._require_live(req)
-        for g, blocks, row in zip(self.groups, req.blocks, req.table_rows):
-            for p in blocks:
+        for g, blocks, pooled, row in zip(self.groups, req.blocks, req.pooled, req.table_rows):
+            for p in [*blocks, *pooled]:
                 if p >= 0:
                     g.pool.give_back(p)
             blocks.clear()
+            pooled.clear()
             row.fill(-1)
         self.slots.give_back(req.slot)
         req.live = False
@@ -262,7 +282,10 @@ class CacheManager:
         """The first logical block that a query at position ``pos0`` (or later) still reads."""
         if g.spec.window <= 0:
             return 0
-        return max(0, pos0 - g.spec.window + 1) // self.page_size
+        first = max(0, pos0 - g.spec.window + 1)
+        if g.spec.pool > 0:      # (the keys of a block that is not whole yet are still to be pooled)
+            first = min(first, pos0 // g.spec.pool * g.spec.pool)
+        return first // self.page_size
 
     def _first_kept_blocks(self, g: CacheGroup) -> int:
         """How many logical blocks at the start of a request hold positions that stay readable behind the window."""
@@ -274,9 +297,26 @@ class CacheManager:
         out = []
         end = req.n_tokens + n_new
         n_blocks = -(-end // self.page_size)
-        for g, blocks in zip(self.groups, req.blocks):
-            out.append(max(0, n_blocks - len(blocks)))
+        for g, blocks, pooled in zip(self.groups, req.blocks, req.pooled):
+            out.append(max(0, n_blocks - len(blocks)) + max(0, self._pool_pages(g, end) - len(pooled)))
         return out
+
+    def pages_for(self, n_tokens: int) -> List[int]:
+        """Pages per group that ``n_tokens`` positions of one request take if none goes back behind a window."""
+        return [-(-n_tokens // self.page_size) + self._pool_pages(g, n_tokens) for g in self.groups]
+
+    def room(self, req: RequestCache, free: Sequence[int]) -> Optional[int]:
+        """How many tokens the request could append with so many free pages per group (None: any number)."""
+        most = None
+        for g, blocks, pooled, f in zip(self.groups, req.blocks, req.pooled, free):
+            k = f                # pages for positions; what is left must do for the pooled rows
+            while k > 0 and k + max(0, self._pool_pages(g, (len(blocks) + k) * self.page_size) - len(pooled)) > f:
+                k -= 1
+            n = (len(blocks) + k) * self.page_size - req.n_tokens
+            while n > 0 and self._pool_pages(g, req.n_tokens + n) - len(pooled) > f - k:
+                n -= 1
+            most = n if most is None else min(most, n)
+        return most
 
     def can_append(self, work: Sequence[Tuple[RequestCache, int]]) -> bool:
         need = [0] * len(self.groups)
@@ -298,13 +338,17 @@ class CacheManager:
         for req, n in work:
             n_blocks = -(-(req.n_tokens + n) // self.page_size)
             for gi, g in enumerate(self.groups):
-                if n_blocks > self.max_blocks[gi]:
+                if n_blocks > self.pool_column[gi]:
                     self._grow_tables(gi, n_blocks)
-            for g, blocks, row in zip(self.groups, req.blocks, req.table_rows):
+            for g, blocks, pooled, row, at in zip(self.groups, req.blocks, req.pooled, req.table_rows, self.pool_column):
                 while len(blocks) < n_blocks:
                     page = g.pool.take()
                     row[len(blocks)] = page
                     blocks.append(page)
+                while len(pooled) < self._pool_pages(g, req.n_tokens + n):
+                    page = g.pool.take()
+                    row[at + len(pooled)] = page
+                    pooled.append(page)
 
     def commit(self, req: RequestCache, n_new: int) -> None:
         """The step ran: the request is ``n_new`` tokens longer; pages a window has passed go back."""
@@ -333,7 +377,7 @@ class CacheManager:
         if self._state_keys and n_tokens != req.n_tokens:
             raise CacheError("truncate: a mixer keeps per-request state, which cannot be rolled back")
         keep = -(-n_tokens // self.page_size)
-        for g, blocks, row in zip(self.groups, req.blocks, req.table_rows):
+        for g, blocks, pooled, row, at in zip(self.groups, req.blocks, req.pooled, req.table_rows, self.pool_column):
             if g.spec.window > 0 and n_tokens < req.n_tokens:
                 first = self._first_needed_block(g, n_tokens)
                 kept = range(min(self._first_kept_blocks(g), keep, len(blocks)))
@@ -344,6 +388,9 @@ class CacheManager:
                 row[len(blocks)] = -1
                 if p >= 0:
                     g.pool.give_back(p)
+            while len(pooled) > self._pool_pages(g, n_tokens):
+                g.pool.give_back(pooled.pop())
+                row[at + len(pooled)] = -1
         req.n_tokens = n_tokens
 
     # ------------------------------------------------------------------ views and accounting
@@ -355,7 +402,9 @@ class CacheManager:
         views: Dict[int, KVCacheView] = {}
         for gi, g in enumerate(self.groups):
             for li, idx in enumerate(g.owners):
-                views[idx] = KVCacheView(g.tensor[li], block_tables[gi], self.page_size, g.spec.window)
+                at = self.pool_column[gi]
+                views[idx] = KVCacheView(g.tensor[li], block_tables[gi], self.page_size, g.spec.window,
+                                         block_tables[gi][:, at:] if g.spec.pool > 0 else None)
         return views
 
     @property
@@ -375,14 +424,17 @@ class CacheManager:
         """Invariants: every page is free or held by exactly one live request; slots likewise."""
         for gi, g in enumerate(self.groups):
             g.pool.check()
-            held = [p for r in self._live for p in r.blocks[gi] if p >= 0]
+            held = [p for r in self._live for p in [*r.blocks[gi], *r.pooled[gi]] if p >= 0]
             if len(set(held)) != len(held):
                 raise CacheError(f"group {gi}: a page is held twice")
             if len(held) != g.pool.n_used:
                 raise CacheError(f"group {gi}: {g.pool.n_used} pages are out but requests hold {len(held)}")
             for r in self._live:
-                row = r.table_rows[gi]
-                if list(row[:len(r.blocks[gi])]) != r.blocks[gi] or (row[len(r.blocks[gi]):] != -1).any():
+                row, at = r.table_rows[gi], self.pool_column[gi]
+                want = np.full(self.max_blocks[gi], -1, dtype=np.int32)
+                want[:len(r.blocks[gi])] = r.blocks[gi]
+                want[at:at + len(r.pooled[gi])] = r.pooled[gi]
+                if not np.array_equal(row, want):
                     raise CacheError(f"group {gi}: a block table row does not mirror the request's pages")
         self.slots.check()
         if len({r.slot for r in self._live}) != len(self._live):

@@ -25,6 +25,11 @@
 //   head_scale:   one number per query head that multiplies the scale (a temperature);
 //   sinks:        with `sink` set, one number per query head: the denominator's extra term is exp(sinks[h]) instead
 //                 of exp(0);
+//   gate_dim > 0: the gate has one number per element, gate[t * ldg + h * gate_dim + d], for the first gate_dim values of a
+//                 head's result (0: one number per head);
+//   pool > 0:     with a window, the blocks of `pool` positions that lie wholly behind it are seen as one key and one value
+//                 each, the rows b = 0, 1, ... of `pool_table` (pages of the same cache, one table row per entry, max_blocks
+//                 apart like block_table's): position i sees block b if (b + 1) pool - 1 <= i - window;
 //   out32:        `out` holds 32-bit floats whatever the dtype of queries and cache (what follows the attention
 //                 subtracts or norms its results before they are rounded).
 struct AttnExtras {
@@ -38,6 +43,9 @@ struct AttnExtras {
   const float* head_scale;
   const float* sinks;
   int out32;
+  int gate_dim;
+  int pool;
+  const int* pool_table;
 };
 
 #ifdef __cplusplus
@@ -114,7 +122,7 @@ int nib_attention_simt(int dtype, const void* q, int ldq, const void* cache, voi
                        const int* block_table, int max_blocks, const int* rows, const int* row_entry,
                        const int* positions, int T, int n_head, int n_kv_head, int head_dim,
                        int page_size, int n_pages, float scale, int window, int sink, float softcap,
-                       int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
+                       int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int gate_dim, int pool, const int* pool_table, int* status,
                        cudaStream_t stream);
 
 // tcgen05 attention for prompt portions (bfloat16, head size 64, page size a multiple of 16): tiles of
@@ -125,7 +133,7 @@ int nib_attention_prefill_tc(const void* q, int ldq, int T, const void* cache, v
                              const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                              const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head, int head_dim,
                              int page_size, int n_pages, float scale, int window, int sink, float softcap, int keep_first,
-                             const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
+                             const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int gate_dim, int pool, const int* pool_table, int* status,
                              cudaStream_t stream);
 
 // Split-KV attention for single decoded tokens (float32 or bfloat16, head sizes up to 128 in steps
@@ -135,7 +143,7 @@ int nib_attention_decode(int dtype, const void* q, int ldq, const void* cache, f
                          int ldo, const int* block_table, int max_blocks, const int* rows,
                          const int* row_entry, const int* positions, int n_rows, int n_head, int n_kv_head,
                          int head_dim, int page_size, int n_pages, float scale, int window, int sink, float softcap,
-                         int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int chunk,
+                         int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int gate_dim, int pool, const int* pool_table, int chunk,
                          int n_splits, int* counters, int* status, cudaStream_t stream);
 
 // Tiled tensor-core attention for prompt portions (bfloat16, head sizes 16..128 in steps of 16), with the options of
@@ -145,7 +153,7 @@ int nib_attention_prefill(const void* q, int ldq, const void* cache, void* out, 
                           const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                           const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head,
                           int head_dim, int page_size, int n_pages, float scale, int window, int sink, float softcap,
-                          int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
+                          int keep_first, const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int gate_dim, int pool, const int* pool_table, int* status,
                           cudaStream_t stream);
 
 // Loading: src holds [rows, cols] values as a checkpoint stores them (src_dtype 0: 32-bit floats, 1:
@@ -205,7 +213,8 @@ int nib_mlstm(int dtype, const float* proj, int ld, int q_off, int k_off, int v_
               float eps, float* gates, float* num, int ld_num, float* den, void* out, int ldo, cudaStream_t stream);
 
 // ---- attention through a shared low-rank latent (latent_attention.cu); halves: the layout of the rotation (0: pairs
-// (2i, 2i + 1), 1: i with i + rot_dims / 2); gate (may be null): head h's output times sigmoid(gate[t * ldg + h])
+// (2i, 2i + 1), 1: i with i + rot_dims / 2); gate (may be null): head h's output times sigmoid(gate[t * ldg + h]);
+// sinks (may be null): exp(sinks[h]) joins the softmax's denominator
 int nib_latent_prep(int dtype, const float* proj, int ld, int q_rank, int kv_rank, int rot_dim, int rot_dims,
                     const double* freqs, const float* wq, const float* wkv, float eps, void* cq, int ld_cq,
                     void* cache, const int* block_table, int max_blocks, const int* row_entry,
@@ -217,11 +226,12 @@ int nib_rope_heads(int dtype, int out_dtype, const void* q, int ldq, int nope, i
 int nib_latent_attention(int dtype, int q_dtype, const void* q, const void* cache, void* out, int ldo, const int* block_table,
                          int max_blocks, const int* rows, const int* row_entry, const int* positions, int n_rows,
                          int n_head, int kv_rank, int D, int page_size, int n_pages, float scale, int window,
-                         const float* gate, int ldg, int* status, int n_splits, float* partials, cudaStream_t stream);
+                         const float* gate, int ldg, const float* sinks, int* status, int n_splits, float* partials,
+                         cudaStream_t stream);
 
 // ---- attention in bfloat16 over cached rows of any of two shapes: keys and values in two planes [n_pages, 2, n_kv_head,
 // page_size, row_dim], or one plane whose rows are both (planes = 1, the latent cache).  Options: softcap, window, a sigmoid
-// gate per row and head.
+// gate per row and head or (gate_dim > 0) per element, learned sinks, pooled blocks behind the window (as in AttnExtras).
 // Prompt portions in tiles of 128 rows on tcgen05 (attention_wide_tc.cu): with maps > 1 head h scores against the values
 // (h % maps) * map_dim .. + map_dim of the key row; head h's v_cols values go to column h * out_head of its rows.
 int nib_attention_wide_tc_supported(int row_dim, int planes, int maps, int map_dim, int v_cols, int page_size);
@@ -229,7 +239,8 @@ int nib_attention_wide_tc(const void* q, int ldq, int T, const void* cache, int 
                           int out32, const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                           const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head, int row_dim, int maps,
                           int map_dim, int v_cols, int page_size, int n_pages, float scale, int window, float softcap,
-                          const float* gate, int ldg, int* status, cudaStream_t stream);
+                          const float* gate, int ldg, int gate_dim, const float* sinks, int pool, const int* pool_table,
+                          int* status, cudaStream_t stream);
 // Single tokens on warp-level MMAs with the heads of a group as rows and a row's pieces of keys as one cluster
 // (attention_group_mma.cu; n_splits 1, 2, 4, 8 or 16).  diff: the heads come in pairs, and pair i's column i * out_head
 // receives mul * o / sqrt(mean(o^2) + eps), o = a_2i - lambda a_2i+1.
@@ -238,17 +249,19 @@ int nib_attention_group_mma(const void* q, int ldq, const void* cache, int plane
                             const int* block_table, int max_blocks, const int* rows, const int* row_entry,
                             const int* positions, int n_rows, int n_head, int n_kv_head, int row_dim, int k_cols, int v_cols,
                             int page_size, int n_pages, float scale, int window, float softcap, const float* gate, int ldg,
-                            int diff, float lambda, float eps, float mul, int* status, int n_splits, cudaStream_t stream);
+                            int gate_dim, const float* sinks, int pool, const int* pool_table, int diff, float lambda, float eps, float mul, int* status, int n_splits, cudaStream_t stream);
 
-// ---- a product per head (linear_heads.cu; in bfloat16 on warp-level MMAs: linear_heads_mma.cu): out[t, h, :N] = a[t, h, :K] . w[h]^T, w [n_head, N, K]
+// ---- a product per head (linear_heads.cu; in bfloat16 on warp-level MMAs: linear_heads_mma.cu): out[t, h, :N] = a[t, h, :K] . w[h]^T, w [n_head, N, K];
+// gate (may be null): times sigmoid(gate[t * ldg + h * N + n])
 int nib_linear_heads(int dtype, int out_dtype, const void* a, int lda, int a_head_stride, const void* w, void* out,
-                     int ldo, int out_head_stride, int M, int n_head, int N, int K, cudaStream_t stream);
+                     int ldo, int out_head_stride, int M, int n_head, int N, int K, const float* gate, int ldg,
+                     cudaStream_t stream);
 
 int nib_linear_heads_mma_supported(const void* a, int lda, int a_head_stride, const void* w, int K);
 // rot_dim > 0: a's heads are [K | rot_dim], out's [N | rot_dim]; the rotated part turned by the row's position goes with it.
 int nib_linear_heads_mma(int out_dtype, const void* a, int lda, int a_head_stride, const void* w, void* out, int ldo,
                          int out_head_stride, int M, int n_head, int N, int K, const int* positions, const double* freqs,
-                         int rot_dim, int rot_dims, int halves, cudaStream_t stream);
+                         int rot_dim, int rot_dims, int halves, const float* gate, int ldg, cudaStream_t stream);
 
 // ---- the generalised delta rule (delta_rule.cu)
 int nib_delta_rule(int dtype, float* proj, int ld, int r_off, int k_off, int v_off, int g_off, int a_off,
@@ -261,7 +274,7 @@ int nib_delta_rule(int dtype, float* proj, int ld, int r_off, int k_off, int v_o
 // number per expert added to the score for the choice only.  The experts n_real .. n_expert - 1 have no matrices:
 // a row that chooses one gets its own input times the score added to x [T, C] here, and the id -1.
 int nib_moe_route(int dtype, const void* h, int ldh, const void* w_router, int T, int C, int n_expert, int top,
-                  int renorm, int score, const float* choice_bias, int n_real, float* x, int* ids, float* weights,
+                  int renorm, int score, const float* logit_bias, const float* choice_bias, int n_real, float* x, int* ids, float* weights,
                   cudaStream_t stream);
 // gated: w_up [experts, 2F, C], rows 2f and 2f + 1 the gate and the value of output f; inner = act(s g) * (s u) with
 // s = in_weights[t * top + k] (null: 1).
@@ -343,10 +356,22 @@ int nib_selective_scan(int out_dtype, const float* dtp, int ld_dt, const float* 
 
 // ---- norms in groups (group_norm.cu): every row is cut into `groups` equal consecutive parts, each divided by its own
 // root mean square (eps inside the root), and the whole multiplied by w.
-// out[r] = norm(x[rows[r]] (+ add)); with `add` (one vector of C floats) the sum is also written back to x (rows null
-// then).  out may be null: the sum only.
-int nib_group_norm(int out_dtype, float* x, const int* rows, const float* add, const float* w, void* out, int n_rows,
-                   int C, int groups, float eps, cudaStream_t stream);
+// out[r] = norm(x[rows[r]] (+ add)); with `add` (one vector of C floats) or `add_rows` (C floats a row, added ahead of
+// it) the sum is also written back to x (rows null then).  out may be null: the sum only.
+int nib_group_norm(int out_dtype, float* x, const int* rows, const float* add, const float* add_rows, const float* w, void* out,
+                   int n_rows, int C, int groups, float eps, cudaStream_t stream);
+
+// ---- short convolution, norm per head, cache write and pooled rows of an attention whose values are its keys
+// (conv_pool_append.cu)
+int nib_conv_pool_append(int dtype, const float* proj, int ld, int taps, const float* w, float* state,
+                         long long state_stride, const int* entry_start, const int* entry_slot, const int* positions,
+                         const int* row_entry, int n_head, int n_kv_head, int dim, int hd, int norm, float eps, void* q_out,
+                         int ldq, void* cache, const int* block_table, const int* pool_table, int max_blocks,
+                         int page_size, int n_pages, int pool, int shift_state, int T, int* status, cudaStream_t stream);
+// The state of a short convolution behind a step (the second half of nib_short_conv on its own).
+int nib_short_conv_state(const float* proj, int ld, int c_off, int Cn, int taps, float* state, long long state_stride,
+                         const int* entry_start, const int* entry_slot, int n_entries, cudaStream_t stream);
+
 // x[t] = norm(table[token_t] * scale) in 32-bit (tokens as in nib_embed).
 int nib_embed_group_norm(int dtype, const int* tokens, const int* feedback, const void* table, float scale,
                          const float* w, float* x, int T, int C, int groups, float eps, cudaStream_t stream);

@@ -10,8 +10,10 @@
 // (crates/core/src/kernels/reference.rs:109-142).
 //
 // Options (AttnExtras, api.h): a soft cap and a distance bias on the scores, the first keys kept behind a window
-// (the first split walks them ahead of its own share), a per-head sigmoid gate and a constant on the output.
+// or one pooled key and value a block of positions behind it (the first split walks them ahead of its own share), a
+// sigmoid gate per head or per element and a constant on the output.
 #include "api.h"
+#include "attention_extras.cuh"
 #include "common.cuh"
 
 namespace nib {
@@ -117,7 +119,9 @@ attention_decode_kernel(const T* q, int ldq, const T* cache, float* part_o,
   const int n_main = (first_batch + warp <= last_batch) ? (last_batch - first_batch - warp) / DEC_WARPS + 1 : 0;
   // keys 0 .. kept - 1 that the window has passed stay visible: the first split walks them, in batches of their
   // own, ahead of its share of the window
-  const int kept = split == 0 ? min(ex.keep_first, lo) : 0;
+  // (or, with pooled blocks, the one key and value of each block that lies wholly behind the window)
+  const int kept = split != 0 ? 0 : ex.pool > 0 ? pooled_blocks_seen(pos, window, ex.pool) : min(ex.keep_first, lo);
+  const int* kept_table = ex.pool > 0 ? ex.pool_table + (size_t)row_entry[t] * max_blocks : table;
   const int last_kept = kept > 0 ? (kept - 1) / BK : -1;
   const int n_kept = warp <= last_kept ? (last_kept - warp) / DEC_WARPS + 1 : 0;
   const int n_mine = n_kept + n_main;
@@ -135,7 +139,7 @@ attention_decode_kernel(const T* q, int ldq, const T* cache, float* part_o,
     const int j0 = in_kept ? (warp + i * DEC_WARPS) * BK : (first_batch + warp + (i - n_kept) * DEC_WARPS) * BK;
     const int j_lo = in_kept ? 0 : k_begin, j_hi = in_kept ? kept : k_end;
     cur_j0 = j0;
-    const int page = table[page_size == 16 ? (j0 >> 4) : j0 / page_size];
+    const int page = (in_kept ? kept_table : table)[page_size == 16 ? (j0 >> 4) : j0 / page_size];
     live = 0;
     if (page < 0 || page >= n_pages) {
       if (lane == 0) *status = NIB_STATUS_BAD_PAGE;
@@ -253,12 +257,12 @@ attention_decode_kernel(const T* q, int ldq, const T* cache, float* part_o,
   // a sink (one more term in the denominator: a key of score 0 without a value) counts once, where the row's
   // weights are divided
   const float L1 = (sink && n_splits == 1) ? L + pow2<T>(sink2 - M) : L;
-  const float mul1 = n_splits == 1 ? ex.out_scale * (ex.gate ? 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.ldg + h])) : 1.0f) : 1.0f;
+  const float mul1 = n_splits == 1 ? ex.out_scale * (ex.gate && ex.gate_dim == 0 ? 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.ldg + h])) : 1.0f) : 1.0f;
   for (int d = threadIdx.x; d < head_dim; d += blockDim.x) {
     float acc = 0.0f;
     for (int w = 0; w < ALL_GROUPS; ++w) acc += (gm[w] == -INFINITY) ? 0.0f : go[w * head_dim + d] * pow2<T>(gm[w] - M);
     if (n_splits == 1) {
-      const float y = acc / L1 * mul1;
+      const float y = acc / L1 * mul1 * element_gate(ex, t, h, d);
       if (ex.out32) reinterpret_cast<float*>(out)[(size_t)t * ldo + h * head_dim + d] = y;
       else out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(y);
     } else if (cluster_merge)
@@ -307,14 +311,14 @@ attention_decode_kernel(const T* q, int ldq, const T* cache, float* part_o,
     if (ls > 0.0f) Lx += ls * pow2<T>(part_ml[2 * (base + sp)] - Mx);
   }
   if (sink) Lx += pow2<T>(sink2 - Mx);
-  const float mulx = ex.out_scale * (ex.gate ? 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.ldg + h])) : 1.0f);
+  const float mulx = ex.out_scale * (ex.gate && ex.gate_dim == 0 ? 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.ldg + h])) : 1.0f);
   for (int d = threadIdx.x; d < head_dim; d += blockDim.x) {
     float acc = 0.0f;
     for (int sp = 0; sp < n_splits; ++sp) {
       const float ls = part_ml[2 * (base + sp) + 1];
       if (ls > 0.0f) acc += part_o[(base + sp) * head_dim + d] * pow2<T>(part_ml[2 * (base + sp)] - Mx);
     }
-    const float y = acc / Lx * mulx;
+    const float y = acc / Lx * mulx * element_gate(ex, t, h, d);
     if (ex.out32) reinterpret_cast<float*>(out)[(size_t)t * ldo + h * head_dim + d] = y;
     else out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(y);
   }
@@ -365,13 +369,14 @@ extern "C" int nib_attention_decode(int dtype, const void* q, int ldq, const voi
                                     const int* row_entry, const int* positions, int n_rows, int n_head,
                                     int n_kv_head, int head_dim, int page_size, int n_pages, float scale,
                                     int window, int sink, float softcap, int keep_first, const float* slopes,
-                                    const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int chunk, int n_splits,
+                                    const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int gate_dim, int pool, const int* pool_table, int chunk, int n_splits,
                                     int* counters, int* status, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32};
+  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32, gate_dim, pool, pool_table};
   if (head_dim <= 0 || head_dim > DEC_MAX_HD || (head_dim & 7)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (page_size % 16 != 0 || chunk <= 0 || chunk % 16 != 0 || n_splits <= 0) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_kv_head <= 0 || n_head % n_kv_head != 0) return NIB_ERR_BAD_ARGUMENT;
+  if (bad_pool(ex, window)) return NIB_ERR_BAD_ARGUMENT;
   if (n_rows > 65535 || n_head > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_splits > 1 && (scratch == nullptr || counters == nullptr)) return NIB_ERR_BAD_ARGUMENT;
   float* part_o = scratch;
@@ -444,5 +449,5 @@ extern "C" int nib_attention_decode_static(int dtype, const void* q, int ldq, co
   if (e != cudaSuccess) return (int)e;
   return nib_attention_decode(dtype, q, ldq, cache, scratch, out, ldo, block_table, max_blocks, rows, row_entry,
                               positions, n_rows, n_head, n_kv_head, head_dim, page_size, n_pages, scale, window,
-                              0, 0.0f, 0, nullptr, nullptr, 0, 1.0f, 0, nullptr, nullptr, 0, chunk, n_splits, counters, status, stream);
+                              0, 0.0f, 0, nullptr, nullptr, 0, 1.0f, 0, nullptr, nullptr, 0, 0, 0, nullptr, chunk, n_splits, counters, status, stream);
 }

@@ -12,10 +12,13 @@
 // them ahead of griddepcontrol.wait where it does not hold the row's own key.  The pieces of a row are the blocks of one
 // cluster: each leaves its (maximum, sum, unscaled result) in its own shared memory, and the warps of all of them share the
 // merge through distributed shared memory, in the order of the pieces.  What is written:
-//   a head's result, times sigmoid(gate[t, h]) where there is a gate; or (`diff`) for every pair of heads (2i, 2i + 1) the
+//   a head's result, times sigmoid(gate[t, h]), or of a gate per element, where there is one; or (`diff`) for every pair of heads (2i, 2i + 1) the
 //   difference a_2i - lambda a_2i+1 over its root mean square, times a constant (differential.cu says it for portions).
+// With pooled blocks behind the window (one key and value for `pool` positions, rows of another list of pages of the same
+// cache) a row's keys are one sequence, the blocks first; a learned sink joins the sum where the pieces merge.
 // Scores (capped where asked for), softmax, sums, difference and norm are 32-bit.
 #include "api.h"
+#include "attention_extras.cuh"
 #include "common.cuh"
 
 namespace nib {
@@ -65,7 +68,10 @@ struct GmParams {
   float scale, softcap;
   int window;
   const float* gate;
-  int ldg;
+  int ldg, gate_dim;            // gate_dim 0: one gate a head, else one for each of a head's first gate_dim values
+  const float* sinks;           // a logit per head that joins the denominator (null: none)
+  int pool;                     // > 0: blocks of so many positions behind the window are one key and value each,
+  const int* pool_table;        // rows of these pages
   int diff;
   float lambda, eps, mul;
   int* status;
@@ -99,15 +105,19 @@ attention_group_mma_kernel(const GmParams prm) {
   const int entry = prm.row_entry[t], pos = prm.positions[t];
   // (a row of no request takes part in the cluster's barriers with an empty piece)
   const int lo = prm.window > 0 ? max(0, pos - prm.window + 1) : 0;
-  const int per = ((pos - lo + n_splits) / n_splits + 15) / 16 * 16;
-  const int k_begin = lo + split * per, k_end = entry < 0 ? 0 : min(pos + 1, k_begin + per);
+  // the row's keys in one sequence: its pooled blocks, then the window's positions (key k >= nb is position k + shift)
+  const int nb = pooled_blocks_seen(pos, prm.window, prm.pool), shift = lo - nb, n_keys = pos + 1 - shift;
+  const int per = ((n_keys - 1 + n_splits) / n_splits + 15) / 16 * 16;
+  const int k_begin = split * per, k_end = entry < 0 ? 0 : min(n_keys, k_begin + per);
   const int n_it = k_end > k_begin ? (k_end - k_begin + GM_BN - 1) / GM_BN : 0;
   const int* table = prm.block_table + (size_t)max(entry, 0) * prm.max_blocks;
+  const int* pool_table = prm.pool_table + (size_t)max(entry, 0) * prm.max_blocks;
 
   // the cached row (counted in rows of row_dim values) of key j for this group; -1: not there
-  auto cached_row = [&](int j) -> int {
-    if (j >= k_end) return -1;
-    const int page = table[j / prm.page_size];
+  auto cached_row = [&](int k) -> int {
+    if (k >= k_end) return -1;
+    const int j = k < nb ? k : k + shift;
+    const int page = (k < nb ? pool_table : table)[j / prm.page_size];
     if (page < 0 || page >= prm.n_pages) {
       *prm.status = NIB_STATUS_BAD_PAGE;
       return -1;
@@ -138,7 +148,7 @@ attention_group_mma_kernel(const GmParams prm) {
     load_plane(ks + buf * GM_BN * LDK, LDK, Dk / 8, prm.row_dim, row_lo, row_hi, 0);
     if (!shared_row) load_plane(vs + buf * GM_BN * LDV, LDV, Dv / 8, prm.row_dim, row_lo, row_hi, prm.n_kv_head * prm.page_size);
   };
-  const bool early = n_it > 0 && min(k_end, k_begin + GM_BN) <= pos;  // the first tile does not hold the row's own key
+  const bool early = n_it > 0 && min(k_end, k_begin + GM_BN) < n_keys;  // the first tile does not hold the row's own key
   if (early) load_tile(0, 0);
   pdl_wait();
   if (n_it > 0) {
@@ -318,6 +328,7 @@ attention_group_mma_kernel(const GmParams prm) {
             }
           }
       }
+      if (prm.sinks != nullptr) L += gm_pow2(prm.sinks[h0 + hh] * LOG2E - M);
       const float inv = 1.0f / L;
       return make_float4(acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv);
     };
@@ -329,9 +340,15 @@ attention_group_mma_kernel(const GmParams prm) {
         const int hh = u / parts, d = (u % parts) * 128 + 4 * lane;
         if (d >= v_cols) continue;
         const float4 v = merged4(hh, d);
-        const float g = prm.gate ? 1.0f / (1.0f + __expf(-prm.gate[(size_t)t * prm.ldg + h0 + hh])) : 1.0f;
+        const float g = prm.gate && prm.gate_dim == 0 ? 1.0f / (1.0f + __expf(-prm.gate[(size_t)t * prm.ldg + h0 + hh])) : 1.0f;
         bf16* dst = row + (size_t)(h0 + hh) * prm.out_head + d;
-        const float w[4] = {v.x * g, v.y * g, v.z * g, v.w * g};
+        float w[4] = {v.x * g, v.y * g, v.z * g, v.w * g};
+        if (prm.gate_dim > 0) {
+          const float* gr = prm.gate + (size_t)t * prm.ldg + (size_t)(h0 + hh) * prm.gate_dim + d;
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+            if (d + c < prm.gate_dim) w[c] *= 1.0f / (1.0f + __expf(-gr[c]));
+        }
 #pragma unroll
         for (int c = 0; c < 4; ++c)
           if (d + c < v_cols) dst[c] = from_float<bf16>(w[c]);
@@ -413,13 +430,16 @@ extern "C" int nib_attention_group_mma(const void* q, int ldq, const void* cache
                                        const int* block_table, int max_blocks, const int* rows, const int* row_entry,
                                        const int* positions, int n_rows, int n_head, int n_kv_head, int row_dim, int k_cols,
                                        int v_cols, int page_size, int n_pages, float scale, int window, float softcap,
-                                       const float* gate, int ldg, int diff, float lambda, float eps, float mul, int* status,
+                                       const float* gate, int ldg, int gate_dim, const float* sinks, int pool, const int* pool_table,
+                                       int diff, float lambda, float eps, float mul, int* status,
                                        int n_splits, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (n_head <= 0 || n_kv_head <= 0 || n_head % n_kv_head || page_size <= 0 || softcap < 0.0f ||
       !(n_splits == 1 || n_splits == 2 || n_splits == 4 || n_splits == 8 || n_splits == 16))
     return NIB_ERR_BAD_ARGUMENT;
   if (diff && (n_head / n_kv_head) % 2) return NIB_ERR_BAD_ARGUMENT;
+  if (pool < 0 || gate_dim < 0 || (pool > 0 && (window <= 0 || pool_table == nullptr)) || (gate_dim > 0 && gate == nullptr))
+    return NIB_ERR_BAD_ARGUMENT;
   if (!nib_attention_group_mma_supported(row_dim, planes, k_cols, v_cols, diff) || n_rows > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || (ldq & 7)) return NIB_ERR_UNSUPPORTED_SIZE;
   if ((long long)n_pages * planes * n_kv_head * page_size > 0x7fffffffll) return NIB_ERR_UNSUPPORTED_SIZE;
@@ -429,6 +449,7 @@ extern "C" int nib_attention_group_mma(const void* q, int ldq, const void* cache
   prm.row_entry = row_entry; prm.positions = positions; prm.n_head = n_head; prm.n_kv_head = n_kv_head; prm.planes = planes;
   prm.row_dim = row_dim; prm.k_cols = k_cols; prm.v_cols = v_cols; prm.page_size = page_size; prm.n_pages = n_pages;
   prm.scale = scale; prm.softcap = softcap; prm.window = window; prm.gate = gate; prm.ldg = ldg; prm.diff = diff;
+  prm.gate_dim = gate_dim; prm.sinks = sinks; prm.pool = pool; prm.pool_table = pool > 0 ? pool_table : block_table;
   prm.lambda = lambda; prm.eps = eps; prm.mul = mul; prm.status = status; prm.n_splits = n_splits;
   if (v_cols <= 64) return launch_group_mma<1>(prm, n_rows, stream);
   if (v_cols <= 128) return launch_group_mma<2>(prm, n_rows, stream);

@@ -363,9 +363,10 @@ extern "C" int nib_attention_prefill(const void* q, int ldq, const void* cache, 
                                      const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head,
                                      int head_dim, int page_size, int n_pages, float scale, int window,
                                      int sink, float softcap, int keep_first, const float* slopes,
-                                     const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status, cudaStream_t stream) {
+                                     const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int gate_dim, int pool, const int* pool_table, int* status, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
-  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32};
+  if (gate_dim > 0 || pool > 0) return NIB_ERR_UNSUPPORTED_SIZE;   // (attention_wide_tc.cu takes those)
+  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32, gate_dim, pool, pool_table};
   const bool plain = !(softcap > 0.0f) && (keep_first <= 0 || window <= 0) && !slopes && !gate && out_scale == 1.0f &&
                      span <= 0 && !head_scale && !sinks && !out32;
   if (span < 0) return NIB_ERR_BAD_ARGUMENT;

@@ -11,9 +11,10 @@
 //
 // Options on the scores and the output (AttnExtras, api.h): a soft cap s <- cap tanh(s / cap); a distance
 // bias s <- s - slope_h (pos - j); with a window, the first `keep_first` keys stay visible behind it (at their
-// true positions); head h's output times sigmoid(gate[t, h]) and times one constant; keys of the position's own
-// span only; a scale and a sink's logit per head.
+// true positions), or one pooled key and value a block of positions does; head h's output times sigmoid(gate[t, h]) (or a
+// gate per element) and times one constant; keys of the position's own span only; a scale and a sink's logit per head.
 #include "api.h"
+#include "attention_extras.cuh"
 #include "common.cuh"
 
 namespace nib {
@@ -57,17 +58,19 @@ attention_simt_kernel(const T* q, int ldq, const T* cache,
   float m = -INFINITY, l = 0.0f;
   const float slope = ex.slopes ? ex.slopes[h] : 0.0f;
   // two runs of keys: those the window has passed but that are kept (0 .. keep_first - 1), then the window's
-  const int kept = min(ex.keep_first, lo);
+  // (or, with pooled blocks, one key and value a block that lies wholly behind the window)
+  const int kept = ex.pool > 0 ? pooled_blocks_seen(pos, window, ex.pool) : min(ex.keep_first, lo);
 
   for (int run = kept > 0 ? 0 : 1; run < 2; ++run) {
   const int j_begin = run == 0 ? 0 : lo, j_end = run == 0 ? kept : pos + 1;
+  const int* tab = run == 0 && ex.pool > 0 ? ex.pool_table + (size_t)row_entry[t] * max_blocks : table;
   for (int j0 = j_begin; j0 < j_end; j0 += 32) {
     const int j = j0 + lane;
     const bool valid = j < j_end;
     float s = -INFINITY;
     unsigned long long vo = 0;
     if (valid) {
-      const int page = table[j / page_size];
+      const int page = tab[j / page_size];
       if (page < 0 || page >= n_pages) {
         *status = NIB_STATUS_BAD_PAGE;
       } else {
@@ -107,13 +110,14 @@ attention_simt_kernel(const T* q, int ldq, const T* cache,
   // a sink: one more term in the denominator, a key of score 0 that has no value
   if (sink) l += expf((ex.sinks ? ex.sinks[h] : 0.0f) - m);
   float inv = ex.out_scale / l;
-  if (ex.gate) inv *= 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.ldg + h]));
+  if (ex.gate && ex.gate_dim == 0) inv *= 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.ldg + h]));
 #pragma unroll
   for (int i = 0; i < ATT_MAX_ND; ++i) {
     const int d = lane + 32 * i;
     if (d >= head_dim) continue;
-    if (ex.out32) reinterpret_cast<float*>(out)[(size_t)t * ldo + h * head_dim + d] = o[i] * inv;
-    else out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(o[i] * inv);
+    const float y = o[i] * inv * element_gate(ex, t, h, d);
+    if (ex.out32) reinterpret_cast<float*>(out)[(size_t)t * ldo + h * head_dim + d] = y;
+    else out[(size_t)t * ldo + h * head_dim + d] = from_float<T>(y);
   }
 }
 
@@ -126,12 +130,13 @@ extern "C" int nib_attention_simt(int dtype, const void* q, int ldq, const void*
                                   const int* row_entry, const int* positions, int T, int n_head,
                                   int n_kv_head, int head_dim, int page_size, int n_pages,
                                   float scale, int window, int sink, float softcap, int keep_first,
-                                  const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int* status,
+                                  const float* slopes, const float* gate, int ldg, float out_scale, int span, const float* head_scale, const float* sinks, int out32, int gate_dim, int pool, const int* pool_table, int* status,
                                   cudaStream_t stream) {
   if (T <= 0) return 0;
-  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32};
+  const AttnExtras ex = {softcap, keep_first, slopes, gate, ldg, out_scale, span, head_scale, sinks, out32, gate_dim, pool, pool_table};
   if (head_dim <= 0 || head_dim > 32 * ATT_MAX_ND || (head_dim & 1)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_kv_head <= 0 || n_head % n_kv_head != 0) return NIB_ERR_BAD_ARGUMENT;
+  if (bad_pool(ex, window)) return NIB_ERR_BAD_ARGUMENT;
   if (T > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
   dim3 grid((n_head + ATT_WARPS - 1) / ATT_WARPS, T);
   const size_t smem = (size_t)ATT_WARPS * (head_dim + 32 + 64) * sizeof(float);

@@ -19,14 +19,17 @@
 //               P V first (it frees a stage);
 //   warps 2..5  the softmax, a thread a row: scores times log2(e) (capped first where asked for), running maximum raised only
 //               when a tile exceeds it by more than 2^8 (O is then scaled in tensor memory), P as bfloat16, the sum in
-//               32-bit; at the end the division, an optional sigmoid gate per row and head, and the store (bfloat16, or
-//               32-bit floats).
+//               32-bit; at the end an optional learned sink, the division, an optional sigmoid gate per row and head or per
+//               element, and the store (bfloat16, or 32-bit floats).
+// Ahead of the window's tiles come those of pooled blocks where there are any: rows of another list of pages of the same
+// cache, one key and value for `pool` positions that lie wholly behind the window; every row knows how many it sees.
 // Keys outside [lowest visible, last row] are masked; their rows are read from the nearest unit of the request that is
 // there.  What a box reaches beyond the row, or beyond the step's rows, reads as zeros.
 //
 // Every wait on a barrier is bounded: a wait that runs out sets the block's abort flag and the device status word, every
 // role leaves its loop, tensor memory is freed, and the kernel returns.
 #include "api.h"
+#include "attention_extras.cuh"
 #include "common.cuh"
 #include "tcgen05.cuh"
 
@@ -51,7 +54,10 @@ struct LpParams {
   float scale, softcap;
   int window;
   const float* gate;
-  int ldg;
+  int ldg, gate_dim;            // gate_dim 0: one gate a head, else one for each of a head's first gate_dim values
+  const float* sinks;           // a logit per head that joins the denominator (null: none)
+  int pool;                     // > 0: blocks of so many positions behind the window are one key and value each,
+  const int* pool_table;        // rows of these pages
   void* out;
   int ldo, out_head, out32;     // rows and heads of the result, in elements
   int* status;
@@ -68,6 +74,7 @@ __device__ __forceinline__ float lp_pow2(float x) {   // the hardware's 2^x (rel
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float lp_sigmoid(float x) { return 1.0f / (1.0f + __expf(-x)); }
 __device__ __forceinline__ void lp_tmem_ld32(uint32_t taddr, float* v) {
   uint32_t r[32];
   tmem_ld16_issue(taddr, r);
@@ -132,7 +139,10 @@ attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int* table = prm.block_table + (size_t)e * prm.max_blocks;
   const int window = prm.window;
   const int key_lo = (window > 0 && pos_first - window + 1 > 0) ? pos_first - window + 1 : 0;
-  const int tile_first = key_lo / LP_BN, n_it = pos_last / LP_BN - tile_first + 1;
+  // the pooled blocks that the tile's rows see come first, in tiles of their own
+  const int nb_last = pooled_blocks_seen(pos_last, window, prm.pool), n_pool = (nb_last + LP_BN - 1) / LP_BN;
+  const int* pool_table = prm.pool_table + (size_t)e * prm.max_blocks;
+  const int tile_first = key_lo / LP_BN - n_pool, n_it = pos_last / LP_BN - tile_first + 1;
 
   if (threadIdx.x == 0) {
     abort_sh = 0;
@@ -170,9 +180,15 @@ attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const uint32_t tile_bytes = (uint32_t)((nk + (shared_row ? 0 : nv)) * LP_CHUNK_K);
     auto unit_row = [&](int it) -> int {
       if (!active || it >= n_it) return 0;
-      int j = min((tile_first + it) * LP_BN + u * LP_UNIT, pos_last) / LP_UNIT * LP_UNIT;
-      if (j + LP_UNIT - 1 < key_lo) j = key_lo / LP_UNIT * LP_UNIT;      // (behind the window: its page may be gone)
-      const int page = table[j / prm.page_size];
+      const bool in_pool = it < n_pool;
+      int j;
+      if (in_pool) {
+        j = min(it * LP_BN + u * LP_UNIT, nb_last - 1) / LP_UNIT * LP_UNIT;
+      } else {
+        j = min((tile_first + it) * LP_BN + u * LP_UNIT, pos_last) / LP_UNIT * LP_UNIT;
+        if (j + LP_UNIT - 1 < key_lo) j = key_lo / LP_UNIT * LP_UNIT;    // (behind the window: its page may be gone)
+      }
+      const int page = (in_pool ? pool_table : table)[j / prm.page_size];
       if (page < 0 || page >= prm.n_pages) {
         *prm.status = NIB_STATUS_BAD_PAGE;
         return 0;                                          // (page 0: in the pool)
@@ -251,6 +267,7 @@ attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int p = pos_first + r;
     const int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
     const int wp0 = pos_first + quarter * 32, wp1 = wp0 + 31;   // positions of the warp's rows
+    const int nb = pooled_blocks_seen(p, window, prm.pool), wnb0 = pooled_blocks_seen(wp0, window, prm.pool);
     constexpr float LOG2E = 1.4426950408889634f;
     const bool capped = prm.softcap > 0.0f;
     const float scale2 = capped ? 1.0f : prm.scale * LOG2E;    // (capped scores are brought to their final form first)
@@ -262,8 +279,11 @@ attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       ok = warp_mbar_wait(&s_full[b], (it / LP_NBUF) & 1, abort_flag, lane);
       if (!ok) break;
       tc_fence_after();
-      const int j0 = (tile_first + it) * LP_BN;
-      const bool edge = j0 + LP_BN - 1 > wp0 || (window > 0 && j0 < wp1 - window + 1);   // only these tiles need the mask
+      const bool in_pool = it < n_pool;
+      const int j0 = in_pool ? it * LP_BN : (tile_first + it) * LP_BN;
+      // a row sees the keys first .. last of the tile's kind; only tiles at an edge need the mask
+      const int first = in_pool ? 0 : lo, last = in_pool ? nb - 1 : p;
+      const bool edge = in_pool ? j0 + LP_BN > wnb0 : j0 + LP_BN - 1 > wp0 || (window > 0 && j0 < wp1 - window + 1);
       float v[LP_BN];
 #pragma unroll
       for (int c = 0; c < LP_BN / 32; ++c) lp_tmem_ld32(lane_addr + (uint32_t)(b * LP_BN + c * 32), v + c * 32);
@@ -275,7 +295,7 @@ attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       if (edge) {
 #pragma unroll
         for (int i = 0; i < LP_BN; ++i)
-          if (!(j0 + i <= p && j0 + i >= lo)) v[i] = -INFINITY;
+          if (!(j0 + i <= last && j0 + i >= first)) v[i] = -INFINITY;
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // four chains, not one of 64 links
 #pragma unroll
@@ -331,8 +351,9 @@ attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (ok) ok = warp_mbar_wait(&o_full[(n_it - 1) % LP_NBUF], ((n_it - 1) / LP_NBUF) & 1, abort_flag, lane);
     if (ok) {
       tc_fence_after();
+      if (prm.sinks != nullptr) l += lp_pow2(prm.sinks[h] * LOG2E - m);
       float inv = l > 0.0f ? 1.0f / l : 0.0f;
-      if (prm.gate != nullptr && r < n_rows) inv *= 1.0f / (1.0f + __expf(-prm.gate[(size_t)(row0 + r) * prm.ldg + h]));
+      if (prm.gate != nullptr && prm.gate_dim == 0 && r < n_rows) inv *= 1.0f / (1.0f + __expf(-prm.gate[(size_t)(row0 + r) * prm.ldg + h]));
       const size_t at = (size_t)(row0 + r) * prm.ldo + (size_t)h * prm.out_head;
       bf16* dst = reinterpret_cast<bf16*>(prm.out) + at;
       float* dst32 = reinterpret_cast<float*>(prm.out) + at;
@@ -341,6 +362,22 @@ attention_wide_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         float t[16];
         tmem_ld16(lane_addr + LP_O_COL + (uint32_t)(c * 16), t);
         if (r < n_rows) {
+          if (prm.gate_dim > 0) {
+            const float* gr = prm.gate + (size_t)(row0 + r) * prm.ldg + h * prm.gate_dim + c * 16;
+            const int left = prm.gate_dim - c * 16;
+            if (left >= 16 && ((uintptr_t)gr & 15) == 0) {
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const float4 g4 = reinterpret_cast<const float4*>(gr)[i];
+                t[4 * i] *= lp_sigmoid(g4.x); t[4 * i + 1] *= lp_sigmoid(g4.y);
+                t[4 * i + 2] *= lp_sigmoid(g4.z); t[4 * i + 3] *= lp_sigmoid(g4.w);
+              }
+            } else {
+#pragma unroll
+              for (int i = 0; i < 16; ++i)
+                if (i < left) t[i] *= lp_sigmoid(gr[i]);
+            }
+          }
 #pragma unroll
           for (int g = 0; g < 2; ++g) {
             const int d = c * 16 + 8 * g;
@@ -418,11 +455,13 @@ extern "C" int nib_attention_wide_tc(const void* q, int ldq, int T, const void* 
                                      int out_head, int out32, const int* block_table, int max_blocks, const int* tiles,
                                      int n_tiles, const int* entry_start, const int* entry_pos0, int n_head, int n_kv_head,
                                      int row_dim, int maps, int map_dim, int v_cols, int page_size, int n_pages, float scale,
-                                     int window, float softcap, const float* gate, int ldg, int* status,
-                                     cudaStream_t stream) {
+                                     int window, float softcap, const float* gate, int ldg, int gate_dim, const float* sinks,
+                                     int pool, const int* pool_table, int* status, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (!nib_attention_wide_tc_supported(row_dim, planes, maps, map_dim, v_cols, page_size)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_head <= 0 || n_kv_head <= 0 || n_head % n_kv_head || T <= 0 || !(scale > 0.0f) || softcap < 0.0f)
+    return NIB_ERR_BAD_ARGUMENT;
+  if (pool < 0 || gate_dim < 0 || (pool > 0 && (window <= 0 || pool_table == nullptr)) || (gate_dim > 0 && gate == nullptr))
     return NIB_ERR_BAD_ARGUMENT;
   const int align = out32 ? 3 : 7;
   if (((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 15) || (ldo & align) || (out_head & align) || (ldq & 7))
@@ -442,6 +481,7 @@ extern "C" int nib_attention_wide_tc(const void* q, int ldq, int T, const void* 
   prm.stages = 2;
   while (prm.stages < LP_MAX_STAGES && lp_smem(prm.k_slots, vs, prm.stages + 1) <= LP_MAX_SMEM) ++prm.stages;
   prm.scale = scale; prm.softcap = softcap; prm.window = window; prm.gate = gate; prm.ldg = ldg;
+  prm.gate_dim = gate_dim; prm.sinks = sinks; prm.pool = pool; prm.pool_table = pool > 0 ? pool_table : block_table;
   prm.out = out; prm.ldo = ldo; prm.out_head = out_head; prm.out32 = out32; prm.status = status;
   static bool attr_set = false;
   if (!attr_set) {

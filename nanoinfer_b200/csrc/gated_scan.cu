@@ -303,6 +303,16 @@ extern "C" int nib_short_conv(const float* proj, int ld, int c_off, int Cn, int 
   NIB_LAUNCH_CHECK();
 }
 
+extern "C" int nib_short_conv_state(const float* proj, int ld, int c_off, int Cn, int taps, float* state,
+                                    long long state_stride, const int* entry_start, const int* entry_slot, int n_entries,
+                                    cudaStream_t stream) {
+  if (taps <= 1 || n_entries <= 0 || Cn <= 0) return 0;
+  if (taps > 64 || n_entries > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
+  launch_pdl(short_conv_state_kernel, dim3((Cn + 255) / 256, n_entries), dim3(256), 0, stream, proj, ld, c_off, Cn, taps,
+             state, state_stride, entry_start, entry_slot);
+  NIB_LAUNCH_CHECK();
+}
+
 extern "C" int nib_scan_prepare(const float* proj, int ld, int a_off, int w_off, const float* A_log,
                                 const float* dt_bias, float* cv, int ldc, int q_off, int k_off, int N, int n_head,
                                 int n_kq, int delta, float* coef, int T, cudaStream_t stream) {

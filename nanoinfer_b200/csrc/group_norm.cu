@@ -3,7 +3,8 @@
 //
 //   group_norm       : v = x[rows[r]] (+ add); out[r] = norm(v); with `add`, one vector for all rows, v is also written
 //                      back to x: a looped stack of layers adds such a vector to the stream ahead of each pass, in the
-//                      norm that the pass's first layer starts with.  Without `out` only the sum is made.
+//                      norm that the pass's first layer starts with; `add_rows` is a row of its own for each row, added
+//                      ahead of the vector (the embedding's output, given to every later pass again).  Without `out` only the sum is made.
 //   embed_group_norm : x[t] = norm(table[token_t] * scale): the embedding and the norm that follows it in one pass.
 //
 // A warp owns a (row, part): parts do not see one another, so there is no shared memory and no block barrier.  Parts
@@ -40,6 +41,8 @@ struct StreamSource {
   float* x;
   const int* rows;
   const float* add;
+  const float* add_rows;           // more rows [., C] to add, one a row of the stream (null: none)
+  __device__ __forceinline__ bool adds() const { return add != nullptr || add_rows != nullptr; }
   __device__ __forceinline__ float* row(int r, int C) const { return x + (size_t)(rows ? rows[r] : r) * C; }
 };
 template <typename T>
@@ -81,11 +84,15 @@ group_norm_vec_kernel(Src src, const float* __restrict__ w, OutT* out, int n_row
     if (k < n4) {
       v[i] = gn_load4(p + 4 * k);
       if constexpr (Src::WRITES_BACK) {
+        if (src.add_rows != nullptr) {
+          const float4 b = gn_load4(src.add_rows + (size_t)r * C + c0 + 4 * k);
+          v[i] = make_float4(v[i].x + b.x, v[i].y + b.y, v[i].z + b.z, v[i].w + b.w);
+        }
         if (src.add != nullptr) {
           const float4 a = gn_load4(src.add + c0 + 4 * k);
           v[i] = make_float4(v[i].x + a.x, v[i].y + a.y, v[i].z + a.z, v[i].w + a.w);
-          gn_store4(p + 4 * k, v[i].x, v[i].y, v[i].z, v[i].w);
         }
+        if (src.adds()) gn_store4(p + 4 * k, v[i].x, v[i].y, v[i].z, v[i].w);
       } else {
         v[i] = make_float4(v[i].x * src.scale, v[i].y * src.scale, v[i].z * src.scale, v[i].w * src.scale);
       }
@@ -119,10 +126,9 @@ group_norm_any_kernel(Src src, const float* __restrict__ w, OutT* out, int n_row
   for (int c = lane; c < gs; c += 32) {
     float v = to_float(p[c]);
     if constexpr (Src::WRITES_BACK) {
-      if (src.add != nullptr) {
-        v += src.add[c0 + c];
-        p[c] = v;
-      }
+      if (src.add_rows != nullptr) v += src.add_rows[(size_t)r * C + c0 + c];
+      if (src.add != nullptr) v += src.add[c0 + c];
+      if (src.adds()) p[c] = v;
     } else {
       v *= src.scale;
     }
@@ -159,17 +165,18 @@ static int launch_group_norm(Src src, bool aligned, const float* w, OutT* out, i
 
 using namespace nib;
 
-extern "C" int nib_group_norm(int out_dtype, float* x, const int* rows, const float* add, const float* w, void* out,
+extern "C" int nib_group_norm(int out_dtype, float* x, const int* rows, const float* add, const float* add_rows, const float* w, void* out,
                               int n_rows, int C, int groups, float eps, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (C <= 0 || groups <= 0 || C % groups != 0 || (add != nullptr && rows != nullptr) || (out == nullptr && add == nullptr) ||
+  if (C <= 0 || groups <= 0 || C % groups != 0 || ((add != nullptr || add_rows != nullptr) && rows != nullptr) ||
+      (out == nullptr && add == nullptr && add_rows == nullptr) ||
       (out != nullptr && w == nullptr))
     return NIB_ERR_BAD_ARGUMENT;
-  const bool aligned = (((uintptr_t)x | (uintptr_t)add) & 15) == 0;
+  const bool aligned = (((uintptr_t)x | (uintptr_t)add | (uintptr_t)add_rows) & 15) == 0;
   if (out_dtype == DT_F32)
-    return launch_group_norm(StreamSource<float>{x, rows, add}, aligned, w, (float*)out, n_rows, C, groups, eps, stream);
+    return launch_group_norm(StreamSource<float>{x, rows, add, add_rows}, aligned, w, (float*)out, n_rows, C, groups, eps, stream);
   if (out_dtype == DT_BF16)
-    return launch_group_norm(StreamSource<float>{x, rows, add}, aligned, w, (bf16*)out, n_rows, C, groups, eps, stream);
+    return launch_group_norm(StreamSource<float>{x, rows, add, add_rows}, aligned, w, (bf16*)out, n_rows, C, groups, eps, stream);
   return NIB_ERR_BAD_ARGUMENT;
 }
 

@@ -18,7 +18,8 @@
 // Rotation: pairs (2i, 2i+1) of the first rot_dims values or, with `halves`, value i with value i + rot_dims / 2;
 // angle = position * freq[i]; the angle and its sine and cosine are computed in double precision from a table of frequencies made on the host, the
 // rest in 32-bit.  An output gate per head (optional, logits in 32-bit): the head's output times sigmoid(gate[t, h]),
-// applied to the weighted sum of latents, which the map to the head's values leaves linear.  Scores, softmax and the weighted sums are 32-bit.
+// applied to the weighted sum of latents, which the map to the head's values leaves linear.  A sink per head (optional):
+// exp(sinks[h]) joins the denominator once.  Scores, softmax and the weighted sums are 32-bit.
 #include "api.h"
 #include "common.cuh"
 
@@ -134,7 +135,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32)
 latent_attention_kernel(const TQ* q, const T* cache, T* out, int ldo, const int* __restrict__ block_table,
                         int max_blocks, const int* __restrict__ rows, const int* __restrict__ row_entry,
                         const int* __restrict__ positions, int n_head, int kv_rank, int D, int page_size,
-                        int n_pages, float scale, int window, const float* gate, int ldg, int* status, int n_splits, float* partials) {
+                        int n_pages, float scale, int window, const float* gate, int ldg, const float* sinks, int* status, int n_splits, float* partials) {
   pdl_trigger();
   extern __shared__ float smem[];
   const int Dp = D | 1;
@@ -231,6 +232,7 @@ latent_attention_kernel(const TQ* q, const T* cache, T* out, int ldo, const int*
       if (d < kv_rank) dst[2 + d] = acc[k];
     }
   } else if (live) {
+    if (sinks != nullptr) l += expf(sinks[h] - m);
     float inv = l > 0.0f ? 1.0f / l : 0.0f;
     if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
     T* o = out + (size_t)t * ldo + (size_t)h * kv_rank;
@@ -247,7 +249,7 @@ latent_attention_kernel(const TQ* q, const T* cache, T* out, int ldo, const int*
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* partials, T* out, int ldo, const int* __restrict__ rows,
-                    const int* __restrict__ row_entry, int n_head, int kv_rank, const float* gate, int ldg, int n_splits) {
+                    const int* __restrict__ row_entry, int n_head, int kv_rank, const float* gate, int ldg, const float* sinks, int n_splits) {
   pdl_trigger();
   const int t = rows ? rows[blockIdx.x] : blockIdx.x, h = blockIdx.y;
   if (row_entry[t] < 0) return;
@@ -260,6 +262,7 @@ latent_merge_kernel(const float* partials, T* out, int ldo, const int* __restric
     const float ms = src[(size_t)s * (kv_rank + 2)];
     if (ms != -INFINITY) l += src[(size_t)s * (kv_rank + 2) + 1] * expf(ms - m);
   }
+  if (sinks != nullptr) l += expf(sinks[h] - m);
   float inv = l > 0.0f ? 1.0f / l : 0.0f;
   if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
   for (int d = threadIdx.x; d < kv_rank; d += blockDim.x) {
@@ -276,7 +279,7 @@ template <typename T, typename TQ, int NACC>
 static int launch_latent_attention(const TQ* q, const T* cache, T* out, int ldo, const int* block_table,
                                    int max_blocks, const int* rows, const int* row_entry, const int* positions,
                                    int n_rows, int n_head, int kv_rank, int D, int page_size, int n_pages,
-                                   float scale, int window, const float* gate, int ldg, int* status, int n_splits,
+                                   float scale, int window, const float* gate, int ldg, const float* sinks, int* status, int n_splits,
                                    float* partials, cudaStream_t stream) {
   const size_t smem = ((size_t)LA_TILE * (D | 1) + (size_t)LA_WARPS * D) * sizeof(float);
   if (smem > 200 * 1024) return NIB_ERR_UNSUPPORTED_SIZE;
@@ -284,10 +287,10 @@ static int launch_latent_attention(const TQ* q, const T* cache, T* out, int ldo,
     cudaFuncSetAttribute(latent_attention_kernel<T, TQ, NACC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   launch_pdl(latent_attention_kernel<T, TQ, NACC>, dim3(n_rows, (n_head + LA_WARPS - 1) / LA_WARPS, n_splits),
              dim3(LA_WARPS * 32), smem, stream, q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-             n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status, n_splits, partials);
+             n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, sinks, status, n_splits, partials);
   if (n_splits > 1)
     launch_pdl(latent_merge_kernel<T>, dim3(n_rows, n_head), dim3(128), 0, stream, (const float*)partials, out, ldo,
-               rows, row_entry, n_head, kv_rank, gate, ldg, n_splits);
+               rows, row_entry, n_head, kv_rank, gate, ldg, sinks, n_splits);
   NIB_LAUNCH_CHECK();
 }
 
@@ -295,12 +298,12 @@ template <typename T, typename TQ>
 static int pick_latent_attention(const void* q, const void* cache, void* out, int ldo, const int* block_table,
                                  int max_blocks, const int* rows, const int* row_entry, const int* positions,
                                  int n_rows, int n_head, int kv_rank, int D, int page_size, int n_pages,
-                                 float scale, int window, const float* gate, int ldg, int* status, int n_splits,
+                                 float scale, int window, const float* gate, int ldg, const float* sinks, int* status, int n_splits,
                                  float* partials, cudaStream_t stream) {
 #define NIB_LA(N)                                                                                              \
   return launch_latent_attention<T, TQ, N>((const TQ*)q, (const T*)cache, (T*)out, ldo, block_table, max_blocks, rows,       \
                                        row_entry, positions, n_rows, n_head, kv_rank, D, page_size, n_pages,  \
-                                       scale, window, gate, ldg, status, n_splits, partials, stream)
+                                       scale, window, gate, ldg, sinks, status, n_splits, partials, stream)
   const int n = (kv_rank + 31) / 32;
   if (n <= 2) NIB_LA(2);
   if (n <= 4) NIB_LA(4);
@@ -366,21 +369,21 @@ extern "C" int nib_latent_attention(int dtype, int q_dtype, const void* q, const
                                     const int* block_table, int max_blocks, const int* rows, const int* row_entry,
                                     const int* positions, int n_rows, int n_head, int kv_rank, int D,
                                     int page_size, int n_pages, float scale, int window, const float* gate, int ldg,
-                                    int* status, int n_splits, float* partials, cudaStream_t stream) {
+                                    const float* sinks, int* status, int n_splits, float* partials, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (kv_rank <= 0 || D < kv_rank || n_head <= 0) return NIB_ERR_BAD_ARGUMENT;
   if (n_splits < 1 || n_splits > 65535 || (n_splits > 1 && partials == nullptr)) return NIB_ERR_BAD_ARGUMENT;
   if (dtype == DT_F32 && q_dtype == DT_F32)
     return pick_latent_attention<float, float>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-                                        n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, status,
+                                        n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, sinks, status,
                                         n_splits, partials, stream);
   if (dtype == DT_BF16 && q_dtype == DT_F32)
     return pick_latent_attention<bf16, float>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-                                              n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg,
+                                              n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, sinks,
                                               status, n_splits, partials, stream);
   if (dtype == DT_BF16 && q_dtype == DT_BF16)
     return pick_latent_attention<bf16, bf16>(q, cache, out, ldo, block_table, max_blocks, rows, row_entry, positions,
-                                             n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg,
+                                             n_rows, n_head, kv_rank, D, page_size, n_pages, scale, window, gate, ldg, sinks,
                                              status, n_splits, partials, stream);
   return NIB_ERR_BAD_ARGUMENT;
 }

@@ -1,5 +1,6 @@
 // The product per head of linear_heads.cu on warp-level MMAs (bfloat16 operands, 32-bit sums):
 //   out[t, h, :N] = a[t, h, :K] . w[h]^T,   w [H, N, K],   out bfloat16 or float32,
+// times sigmoid(gate[t, h, n]) where there is a gate (32-bit logits),
 // and, where the heads of `a` hold a rotated part behind the K values (a latent attention's queries [K unrotated | rot_dim
 // rotated]), that part turned by the row's position and written behind the N values of the same head in the same launch:
 // the query of a head over a shared latent.
@@ -35,7 +36,7 @@ struct RotTail {
 template <int BM, typename OutT>
 __global__ void __launch_bounds__(128)
 linear_heads_mma_kernel(const bf16* a, int lda, int a_hs, const bf16* __restrict__ w, OutT* out, int ldo, int o_hs, int M,
-                        int N, int K, RotTail rot) {
+                        int N, int K, RotTail rot, const float* gate, int ldg) {
   pdl_trigger();
   __shared__ __align__(16) bf16 as[2][BM * LH_LD];
   __shared__ __align__(16) bf16 ws[2][LH_BN * LH_LD];
@@ -120,21 +121,23 @@ linear_heads_mma_kernel(const bf16* a, int lda, int a_hs, const bf16* __restrict
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
       const int m = c < 2 ? ra : rb, col = n + (c & 1);
-      if (m < M && col < N) out[(size_t)m * ldo + (size_t)h * o_hs + col] = from_float<OutT>(acc[i][c]);
+      if (m >= M || col >= N) continue;
+      const float y = gate ? acc[i][c] / (1.0f + __expf(-gate[(size_t)m * ldg + (size_t)h * N + col])) : acc[i][c];
+      out[(size_t)m * ldo + (size_t)h * o_hs + col] = from_float<OutT>(y);
     }
   }
 }
 
 template <typename OutT>
 static int launch_linear_heads_mma(const void* a, int lda, int a_hs, const void* w, void* out, int ldo, int o_hs, int M,
-                                   int n_head, int N, int K, RotTail rot, cudaStream_t stream) {
+                                   int n_head, int N, int K, RotTail rot, const float* gate, int ldg, cudaStream_t stream) {
   const int nb = (N + LH_BN - 1) / LH_BN + (rot.rot_dim > 0 ? 1 : 0);
   if (M <= 16)
     launch_pdl(linear_heads_mma_kernel<16, OutT>, dim3(nb, (M + 15) / 16, n_head), dim3(128), 0, stream, (const bf16*)a, lda,
-               a_hs, (const bf16*)w, (OutT*)out, ldo, o_hs, M, N, K, rot);
+               a_hs, (const bf16*)w, (OutT*)out, ldo, o_hs, M, N, K, rot, gate, ldg);
   else
     launch_pdl(linear_heads_mma_kernel<64, OutT>, dim3(nb, (M + 63) / 64, n_head), dim3(128), 0, stream, (const bf16*)a, lda,
-               a_hs, (const bf16*)w, (OutT*)out, ldo, o_hs, M, N, K, rot);
+               a_hs, (const bf16*)w, (OutT*)out, ldo, o_hs, M, N, K, rot, gate, ldg);
   NIB_LAUNCH_CHECK();
 }
 
@@ -152,7 +155,8 @@ extern "C" int nib_linear_heads_mma_supported(const void* a, int lda, int a_head
 // rot_dims values, or halves) goes behind the product's N values.
 extern "C" int nib_linear_heads_mma(int out_dtype, const void* a, int lda, int a_head_stride, const void* w, void* out,
                                     int ldo, int out_head_stride, int M, int n_head, int N, int K, const int* positions,
-                                    const double* freqs, int rot_dim, int rot_dims, int halves, cudaStream_t stream) {
+                                    const double* freqs, int rot_dim, int rot_dims, int halves, const float* gate,
+                                    int ldg, cudaStream_t stream) {
   if (M <= 0 || n_head <= 0 || N <= 0) return 0;
   if (!nib_linear_heads_mma_supported(a, lda, a_head_stride, w, K)) return NIB_ERR_UNSUPPORTED_SIZE;
   if (rot_dim < 0 || rot_dims < 0 || rot_dims > rot_dim || (rot_dims & 1) || (rot_dims > 0 && freqs == nullptr) ||
@@ -161,8 +165,8 @@ extern "C" int nib_linear_heads_mma(int out_dtype, const void* a, int lda, int a
   if ((M + 15) / 16 > 65535 || n_head > 65535) return NIB_ERR_UNSUPPORTED_SIZE;
   const RotTail rot = {positions, freqs, rot_dim, rot_dims, halves};
   if (out_dtype == DT_F32)
-    return launch_linear_heads_mma<float>(a, lda, a_head_stride, w, out, ldo, out_head_stride, M, n_head, N, K, rot, stream);
+    return launch_linear_heads_mma<float>(a, lda, a_head_stride, w, out, ldo, out_head_stride, M, n_head, N, K, rot, gate, ldg, stream);
   if (out_dtype == DT_BF16)
-    return launch_linear_heads_mma<bf16>(a, lda, a_head_stride, w, out, ldo, out_head_stride, M, n_head, N, K, rot, stream);
+    return launch_linear_heads_mma<bf16>(a, lda, a_head_stride, w, out, ldo, out_head_stride, M, n_head, N, K, rot, gate, ldg, stream);
   return NIB_ERR_BAD_ARGUMENT;
 }

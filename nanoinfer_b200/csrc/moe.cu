@@ -1,5 +1,5 @@
 // A routed feed-forward: every row goes through `top` of `n_expert` small two-layer experts.
-//   z = W_router h   (32-bit),  s = softmax(z) over all experts,  the `top` largest s are chosen
+//   z = W_router h (+ bias)   (32-bit),  s = softmax(z) over all experts,  the `top` largest s are chosen
 //   (ties to the lower index), their weights are those s themselves or, with `renorm`, divided by
 //   their sum;  out = sum over the chosen e of s_e * W_down[e] act(W_up[e] h).
 //   moe_route : a block per row -> ids [T, top], weights [T, top]
@@ -42,7 +42,7 @@ constexpr int MOE_WARPS = 4;
 template <typename T>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_expert, int top, int renorm, int score,
-                 const float* __restrict__ choice_bias, int n_real, float* x, int* ids, float* weights) {
+                 const float* __restrict__ logit_bias, const float* __restrict__ choice_bias, int n_real, float* x, int* ids, float* weights) {
   pdl_trigger();
   extern __shared__ float smem[];
   float* row = smem;               // [C]
@@ -59,7 +59,7 @@ moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_exp
     float s = 0.0f;
     for (int c = lane; c < C; c += 32) s += row[c] * to_float(w[c]);
     s = warp_sum(s);
-    if (lane == 0) prob[e] = s;
+    if (lane == 0) prob[e] = logit_bias ? s + logit_bias[e] : s;
   }
   __syncthreads();
   if (score == 0) {   // softmax over all experts (score 1: the logits stay, the chosen ones' sigmoids are the scores)
@@ -391,7 +391,7 @@ extern "C" int nib_moe_grouped(int dtype, int phase, const void* src, int ld_src
 }
 
 extern "C" int nib_moe_route(int dtype, const void* h, int ldh, const void* w_router, int T, int C, int n_expert,
-                             int top, int renorm, int score, const float* choice_bias, int n_real, float* x, int* ids,
+                             int top, int renorm, int score, const float* logit_bias, const float* choice_bias, int n_real, float* x, int* ids,
                              float* weights, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (top <= 0 || top > n_expert || C <= 0 || (score != 0 && score != 1)) return NIB_ERR_BAD_ARGUMENT;
@@ -401,11 +401,11 @@ extern "C" int nib_moe_route(int dtype, const void* h, int ldh, const void* w_ro
   if (dtype == DT_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(moe_route_kernel<float>, dim3(T), dim3(MOE_WARPS * 32), smem, stream, (const float*)h, ldh,
-               (const float*)w_router, C, n_expert, top, renorm, score, choice_bias, n_real, x, ids, weights);
+               (const float*)w_router, C, n_expert, top, renorm, score, logit_bias, choice_bias, n_real, x, ids, weights);
   } else if (dtype == DT_BF16) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(moe_route_kernel<bf16>, dim3(T), dim3(MOE_WARPS * 32), smem, stream, (const bf16*)h, ldh,
-               (const bf16*)w_router, C, n_expert, top, renorm, score, choice_bias, n_real, x, ids, weights);
+               (const bf16*)w_router, C, n_expert, top, renorm, score, logit_bias, choice_bias, n_real, x, ids, weights);
   } else {
     return NIB_ERR_BAD_ARGUMENT;
   }

@@ -351,6 +351,8 @@ class ModelRunner:
             if n_pad:
                 tab[E - n_pad:] = -1
                 tab[E - n_pad:, 0] = self.cache.pad_page[gi]
+                if self.cache.groups[gi].spec.pool > 0:
+                    tab[E - n_pad:, self.cache.pool_column[gi]] = self.cache.pad_page[gi]
         self.last_meta_bytes = 4 * lay.total
         self._meta_dev[:lay.total].copy_(host[:lay.total], non_blocking=True)
         if copied is not None:

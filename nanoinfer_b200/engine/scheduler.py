@@ -133,17 +133,6 @@ class Scheduler:
     def has_work(self) -> bool:
         return bool(self.waiting or self.running)
 
-    def _pages(self, n_tokens: int) -> int:
-        return -(-n_tokens // self.cache.page_size)
-
-    def _free_pages(self) -> int:
-        free = self.cache.pages_free()
-        return min(free) if free else 1 << 30
-
-    def _total_pages(self) -> int:
-        sizes = [g.pool.n_pages for g in self.cache.groups]
-        return min(sizes) if sizes else 1 << 30
-
     def _finish(self, req: Request, reason: str) -> None:
         if req.cache is not None:
             self.cache.close_request(req.cache)
@@ -172,17 +161,20 @@ class Scheduler:
         while self.waiting and len(self.running) < self.max_batch:
             req = self.waiting[0]
             n = len(req.tokens)
-            if self._pages(n + 1) > self._total_pages() or (
+            whole = self.cache.pages_for(n + 1)
+            if any(k > g.pool.n_pages for k, g in zip(whole, self.cache.groups)) or (
                     self.max_positions is not None and n > self.max_positions):
                 self.waiting.popleft()
                 self._finish(req, "too_long")
                 finished.append(req)
                 continue
             # pages already promised to running requests whose prompts are not in the cache yet
-            promised = sum(max(0, self._pages(len(r.prompt) + len(r.output) + 1)
-                               - max((len(b) for b in r.cache.blocks), default=0)) for r in self.running)
-            need = self._pages(n + 1) + self.headroom_pages * len(self.running) + promised
-            if self._free_pages() < need or self.cache.slots.n_free == 0:
+            need = [k + self.headroom_pages * len(self.running) for k in whole]
+            for r in self.running:
+                total = self.cache.pages_for(len(r.prompt) + len(r.output) + 1)
+                for g, (k, b, p) in enumerate(zip(total, r.cache.blocks, r.cache.pooled)):
+                    need[g] += max(0, k - len(b) - len(p))
+            if any(f < k for f, k in zip(self.cache.pages_free(), need)) or self.cache.slots.n_free == 0:
                 break  # head of the line waits; nobody overtakes it
             self.waiting.popleft()
             req.cache = self.cache.open_request()
@@ -196,7 +188,6 @@ class Scheduler:
         """Decide the next step.  Returns the items to run (none if nothing is left to run);
         requests ended without running are in ``self.ended_without_step``."""
         self.ended_without_step: List[Request] = []
-        ps = self.cache.page_size
         while True:
             self._admit(self.ended_without_step)
             free = list(self.cache.pages_free())
@@ -210,8 +201,8 @@ class Scheduler:
                 return True
 
             def max_fit(req: Request) -> int:
-                room = [(len(b) + f) * ps - req.cache.n_tokens for b, f in zip(req.cache.blocks, free)]
-                return min(room) if room else 1 << 30
+                room = self.cache.room(req.cache, free)
+                return 1 << 30 if room is None else room
 
             items: List[ScheduledItem] = []
             portions: List[ScheduledItem] = []

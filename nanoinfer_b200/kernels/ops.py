@@ -58,14 +58,16 @@ _SIGNATURES = {
     "nib_attention_prefill_tc_supported": [_c_int, _c_int],
     "nib_attention_prefill_tc": [_c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr,
                                  _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float, _c_int,
-                                 _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr],
+                                 _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
+                           _c_ptr, _c_ptr],
     "nib_attention_simt": [_c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
                            _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float, _c_int,
-                           _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr],
+                           _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
+                           _c_ptr, _c_ptr],
     "nib_attention_decode": [_c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
                              _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float,
-                             _c_int, _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
-                             _c_ptr, _c_ptr],
+                             _c_int, _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int,
+                             _c_ptr, _c_ptr, _c_ptr],
     "nib_attention_decode_mma_supported": [_c_int, _c_int],
     "nib_attention_decode_mma_clusters": [_c_int, _c_int],
     "nib_attention_decode_mma": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
@@ -74,7 +76,8 @@ _SIGNATURES = {
     "nib_attention_prefill_supported": [_c_int],
     "nib_attention_prefill": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
                               _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_float, _c_int,
-                              _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr],
+                              _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr,
+                           _c_ptr, _c_ptr],
     "nib_convert": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, ctypes.c_longlong, ctypes.c_longlong, _c_int, _c_ptr],
     "nib_argmax": [_c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "nib_sample": [_c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int,
@@ -90,15 +93,15 @@ _SIGNATURES = {
     "nib_rope_heads": [_c_int, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
                        _c_int, _c_int, _c_int, _c_ptr],
     "nib_latent_attention": [_c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int,
-                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr,
+                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr,
                              _c_ptr],
     "nib_linear_heads": [_c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
-                         _c_int, _c_int, _c_ptr],
+                         _c_int, _c_int, _c_ptr, _c_int, _c_ptr],
     "nib_delta_rule": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
                        _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_int,
                        _c_ptr, _c_ptr],
-    "nib_moe_route": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int,
-                      _c_ptr, _c_ptr, _c_ptr, _c_ptr],
+    "nib_moe_route": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr,
+                      _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
     "nib_moe_up": [_c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
                    _c_int, _c_ptr, _c_ptr],
     "nib_moe_gate_scale": [_c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int,
@@ -145,15 +148,16 @@ _SIGNATURES = {
     "nib_attention_wide_tc_supported": [_c_int, _c_int, _c_int, _c_int, _c_int, _c_int],
     "nib_attention_wide_tc": [_c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr,
                               _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
-                              _c_int, _c_float, _c_ptr, _c_int, _c_ptr, _c_ptr],
+                              _c_int, _c_float, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "nib_attention_group_mma_supported": [_c_int, _c_int, _c_int, _c_int, _c_int],
     "nib_attention_group_mma": [_c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float,
-                                _c_ptr, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int, _c_ptr],
+                                _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int,
+                                _c_ptr],
     "nib_linear_heads_mma_supported": [_c_ptr, _c_int, _c_int, _c_ptr, _c_int],
     "nib_linear_heads_mma": [_c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                             _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
-    "nib_group_norm": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_ptr],
+                             _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr],
+    "nib_group_norm": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_ptr],
     "nib_embed_group_norm": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float,
                              _c_ptr],
     "nib_norm_rope_maps_append": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
@@ -161,6 +165,10 @@ _SIGNATURES = {
                                   _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "nib_diff_combine": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int,
                          _c_int, _c_ptr],
+    "nib_conv_pool_append": [_c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int,
+                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
+    "nib_short_conv_state": [_c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr, _c_int, _c_ptr],
     "nib_min_gru": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr,
                     _c_int, _c_int, _c_ptr, _c_int, _c_ptr],
 }
@@ -672,32 +680,37 @@ class AttnExtras:
     sigmoid(gate[t, h]); ``out_scale``: and times this constant; ``span`` > 0: position i sees key j only if
     i // span == j // span (spans count from position 0 of the sequence); ``head_scale`` (float32 [n_head]): the
     scale times head_scale[h]; ``sinks`` (float32 [n_head]): with a sink, its term of the denominator is
-    exp(sinks[h]) instead of exp(0); ``out32``: the output is float32 whatever the dtype of queries and cache;
+    exp(sinks[h]) instead of exp(0); ``gate_dim`` > 0: the gate (float32 [rows, >= n_head * gate_dim]) has a number for each
+    of a head's first gate_dim values; ``pool`` > 0 with ``pool_table``: behind the window every whole block of ``pool``
+    positions is seen as one key and one value, the pooled rows of the cache (``KVCacheView.pool_table``): position i sees
+    block b if (b + 1) pool - 1 <= i - window; ``out32``: the output is float32 whatever the dtype of queries and cache;
     ``layout`` (maps, map size, values): not an option but what is known of the rows: query head h is zero outside the values
     (h % maps) * size .. + size of its key row, and only the first so many values of a result are read."""
 
-    __slots__ = ("softcap", "keep_first", "slopes", "gate", "out_scale", "span", "head_scale", "sinks", "out32", "layout")
+    __slots__ = ("softcap", "keep_first", "slopes", "gate", "out_scale", "span", "head_scale", "sinks", "out32", "layout",
+                 "gate_dim", "pool", "pool_table")
 
     def __init__(self, softcap: float = 0.0, keep_first: int = 0, slopes: Optional[torch.Tensor] = None,
                  gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, span: int = 0,
                  head_scale: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, out32: bool = False,
-                 layout: Optional[tuple] = None):
+                 layout: Optional[tuple] = None, gate_dim: int = 0, pool: int = 0, pool_table: Optional[torch.Tensor] = None):
         self.softcap, self.keep_first, self.slopes = float(softcap), int(keep_first), slopes
         self.gate, self.out_scale = gate, float(out_scale)
         self.span, self.head_scale, self.sinks, self.out32 = int(span), head_scale, sinks, bool(out32)
         self.layout = layout
+        self.gate_dim, self.pool, self.pool_table = int(gate_dim), int(pool), pool_table
 
     @property
     def plain(self) -> bool:
         return not (self.softcap > 0.0 or self.keep_first > 0 or self.slopes is not None or self.gate is not None
                     or self.out_scale != 1.0 or self.span > 0 or self.head_scale is not None or self.sinks is not None
-                    or self.out32)
+                    or self.out32 or self.pool > 0)
 
     @property
     def wide(self) -> bool:
-        """Whether the tcgen05 kernel for wide rows takes the options: a cap, a 32-bit output, no others."""
-        return not (self.keep_first > 0 or self.slopes is not None or self.gate is not None or self.out_scale != 1.0
-                    or self.span > 0 or self.head_scale is not None or self.sinks is not None)
+        """Whether the kernels for wide rows (``attention_wide_tc``, ``attention_group_mma``) take the options."""
+        return not (self.keep_first > 0 or self.slopes is not None or self.out_scale != 1.0 or self.span > 0
+                    or self.head_scale is not None)
 
     def args(self) -> tuple:
         g = self.gate
@@ -708,8 +721,10 @@ class AttnExtras:
                 raise KernelError("attention: the slopes, the heads' scales and the sinks must be contiguous float32")
         if self.span < 0:
             raise KernelError("attention: span must not be negative")
+        if self.pool > 0 and (self.pool_table is None or self.pool_table.dtype != torch.int32):
+            raise KernelError("attention: pooled blocks need the table of their pages")
         return (self.softcap, self.keep_first, _ptr(self.slopes), _ptr(g), g.stride(0) if g is not None else 0,
-                self.out_scale, self.span, _ptr(self.head_scale), _ptr(self.sinks), int(self.out32))
+                self.out_scale, self.span, _ptr(self.head_scale), _ptr(self.sinks), int(self.out32), self.gate_dim, self.pool, _ptr(self.pool_table))
 
 
 _NO_EXTRAS = AttnExtras()
@@ -921,10 +936,12 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, b
 
 def attention_wide_tc(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, out_head: int, block_table: torch.Tensor, ctx,
                       plan, n_head: int, scale: float, window: int, maps: int, map_dim: int, v_cols: int,
-                      softcap: float = 0.0, gate: Optional[torch.Tensor] = None) -> bool:
+                      softcap: float = 0.0, gate: Optional[torch.Tensor] = None, gate_dim: int = 0,
+                      sinks: Optional[torch.Tensor] = None, pool: int = 0, pool_table: Optional[torch.Tensor] = None) -> bool:
     """tcgen05 attention for the step's prompt portions over cached rows of any shape (csrc/attention_wide_tc.cu): ``cache``
     [pages, planes, kv heads, page, row size] in bfloat16, planes 1 where a row is key and value at once; ``q`` heads of a
-    row's size; head h's first ``v_cols`` values go to column h * ``out_head`` of ``out`` (bfloat16 or float32).  False if a
+    row's size; head h's first ``v_cols`` values go to column h * ``out_head`` of ``out`` (bfloat16 or float32).  ``gate``, ``gate_dim``, ``sinks``, ``pool``, ``pool_table``
+    as in ``AttnExtras``.  False if a
     size or an alignment is not taken."""
     n_pages, planes, n_kv_head, page_size, row_dim = cache.shape
     ldq = q.stride(0)
@@ -937,7 +954,8 @@ def attention_wide_tc(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, o
         _ptr(q), ldq, ctx.n_rows, _ptr(cache), planes, _ptr(out), out.stride(0), int(out_head), int(out.dtype == torch.float32),
         _ptr(block_table), block_table.shape[1], _ptr(plan.wide_tiles), plan.n_wide_tiles, _ptr(ctx.entry_start),
         _ptr(ctx.entry_pos0), n_head, n_kv_head, row_dim, maps, map_dim, v_cols, page_size, n_pages, float(scale), int(window),
-        float(softcap), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(ctx.status), _stream()), "attention_wide_tc")
+        float(softcap), _ptr(gate), gate.stride(0) if gate is not None else 0, int(gate_dim), _ptr(sinks), int(pool),
+        _ptr(pool_table), _ptr(ctx.status), _stream()), "attention_wide_tc")
     return True
 
 
@@ -957,12 +975,13 @@ def group_splits(n_rows: int, n_head: int, n_kv_head: int, max_keys: int) -> int
 
 def attention_group_mma(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, out_head: int, block_table: torch.Tensor, ctx,
                         plan, n_head: int, scale: float, window: int, k_cols: int, v_cols: int, softcap: float = 0.0,
-                        gate: Optional[torch.Tensor] = None, diff: Optional[tuple] = None,
-                        n_splits: Optional[int] = None) -> bool:
+                        gate: Optional[torch.Tensor] = None, diff: Optional[tuple] = None, n_splits: Optional[int] = None,
+                        gate_dim: int = 0, sinks: Optional[torch.Tensor] = None, pool: int = 0,
+                        pool_table: Optional[torch.Tensor] = None) -> bool:
     """Attention of the step's single tokens with the heads that share cached rows as the rows of an MMA tile
     (csrc/attention_group_mma.cu); ``cache`` and ``q`` as in ``attention_wide_tc``, ``out`` bfloat16.  ``diff`` (lambda, eps,
     factor): the heads come in pairs, and what is written for pair i, at column i * ``out_head``, is the normed difference of
-    its two results.  False if a size or an alignment is not taken."""
+    its two results.  The other options as in ``attention_wide_tc``.  False if a size or an alignment is not taken."""
     n_pages, planes, n_kv_head, page_size, row_dim = cache.shape
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or q.stride(0) % 8 \
             or q.data_ptr() % 16 or cache.data_ptr() % 16 \
@@ -970,13 +989,15 @@ def attention_group_mma(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor,
         return False
     if n_splits is None:
         keys = plan.max_decode_keys if window <= 0 else min(plan.max_decode_keys, window)
+        if pool > 0:
+            keys += max(0, plan.max_decode_keys - window) // pool
         n_splits = group_splits(plan.n_decode, n_head, n_kv_head, keys)
     lam, eps, mul = diff if diff is not None else (0.0, 0.0, 1.0)
     _check(library().nib_attention_group_mma(
         _ptr(q), q.stride(0), _ptr(cache), planes, _ptr(out), out.stride(0), int(out_head), _ptr(block_table),
         block_table.shape[1], _ptr(plan.decode_rows), _ptr(ctx.row_entry), _ptr(ctx.positions), plan.n_decode, n_head, n_kv_head,
         row_dim, k_cols, v_cols, page_size, n_pages, float(scale), int(window), float(softcap), _ptr(gate),
-        gate.stride(0) if gate is not None else 0, int(diff is not None), float(lam), float(eps), float(mul), _ptr(ctx.status),
+        gate.stride(0) if gate is not None else 0, int(gate_dim), _ptr(sinks), int(pool), _ptr(pool_table), int(diff is not None), float(lam), float(eps), float(mul), _ptr(ctx.status),
         int(n_splits), _stream()), "attention_group_mma")
     return True
 
@@ -1017,7 +1038,7 @@ def attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_tab
             _note_attention(n_portion, plan.prefill_keys, plan.prefill_kv_rows, n_head, n_kv_head, head_dim,
                             q.element_size(), sizes, out.element_size())
         maps, map_dim, v_cols = layout if layout is not None else (1, head_dim, head_dim)
-        if q.dtype == torch.bfloat16 and (layout is not None or head_dim > 64) and not sink and (extras is None or extras.wide) \
+        if q.dtype == torch.bfloat16 and (layout is not None or head_dim > 64) and not sink and (extras is None or (extras.wide and extras.gate is None and extras.pool == 0)) \
                 and attention_wide_tc(q, cache, out, head_dim, block_table, ctx, plan, n_head, scale, window, maps, map_dim,
                                       v_cols, softcap=extras.softcap if extras is not None else 0.0):
             pass
@@ -1261,11 +1282,14 @@ def _latent_keys(ctx, window: int, single: bool) -> int:
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, ctx,
                      n_head: int, kv_rank: int, scale: float, window: int, n_splits: Optional[int] = None,
-                     gate: Optional[torch.Tensor] = None, plan=None) -> None:
+                     gate: Optional[torch.Tensor] = None, plan=None, sinks: Optional[torch.Tensor] = None) -> None:
     """Causal softmax attention of the step's rows over one latent cache layer: q [T, n_head, D] (the absorbed query,
     then the rotated part) in float32 or the cache's dtype, out [T, n_head * kv_rank] the weighted sums of latents.  A step of
     few rows (decoded tokens) cuts every row's keys into ``n_splits`` pieces, merged by a second kernel.  ``gate``
-    (float32 [rows, >= n_head], any row stride): head h's output of row t times sigmoid(gate[t, h])."""
+    (float32 [rows, >= n_head], any row stride): head h's output of row t times sigmoid(gate[t, h]).  ``sinks`` (float32
+    [n_head]): exp(sinks[h]) joins the denominator."""
+    if sinks is not None and (sinks.dtype != torch.float32 or not sinks.is_contiguous() or sinks.numel() != n_head):
+        raise KernelError("latent_attention: the sinks must be contiguous float32 [n_head]")
     if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1):
         raise KernelError("latent_attention: the gate must be float32 with contiguous rows")
     n_pages, _, _, page_size, D = cache.shape
@@ -1273,7 +1297,7 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
         raise KernelError("latent_attention: q must be contiguous, float32 or of the cache's dtype")
     if out.dtype != cache.dtype or out.stride(1) != 1 or q.shape[2] != D:
         raise KernelError("latent_attention: out in the cache's dtype, q [T, heads, D]")
-    gate_args = (_ptr(gate), gate.stride(0) if gate is not None else 0)
+    gate_args = (_ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(sinks))
     if plan is not None and q.dtype == torch.bfloat16 and n_splits is None:
         # on the tensor cores where the sizes allow; what they do not take goes to the general kernel by lists of rows
         e, todo = q.element_size(), []
@@ -1283,14 +1307,16 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
                 keys = _latent_keys(ctx, window, True)
                 _note("attn", "latent_attn", (plan.n_decode, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
                       e * (plan.n_decode * n_head * (D + kv_rank) + keys * D))
-            if not attention_group_mma(q2, cache, out, kv_rank, block_table, ctx, plan, n_head, scale, window, D, kv_rank, gate=gate):
+            if not attention_group_mma(q2, cache, out, kv_rank, block_table, ctx, plan, n_head, scale, window, D, kv_rank, gate=gate,
+                                       sinks=sinks):
                 todo.append((plan.decode_rows, plan.n_decode))
         if plan.n_prefill_rows:
             if tracing():
                 keys = _latent_keys(ctx, window, False)
                 _note("attn", "latent_attn", (plan.n_prefill_rows, keys, n_head * D), keys * n_head * 2.0 * (D + kv_rank),
                       e * (plan.n_prefill_rows * n_head * (D + kv_rank) + plan.prefill_kv_rows * D))
-            if not attention_wide_tc(q2, cache, out, kv_rank, block_table, ctx, plan, n_head, scale, window, 1, D, kv_rank, gate=gate):
+            if not attention_wide_tc(q2, cache, out, kv_rank, block_table, ctx, plan, n_head, scale, window, 1, D, kv_rank, gate=gate,
+                                       sinks=sinks):
                 # (portions alone: all of the step's rows, those of no request among them, which the kernel leaves out)
                 todo.append((plan.prefill_rows, plan.n_prefill_rows if plan.n_decode else ctx.n_rows))
         for rows, n in todo:
@@ -1320,23 +1346,27 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, bl
 
 
 def linear_heads(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
-                 M: int, rot=None) -> None:
+                 M: int, rot=None, gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h * out_head_stride + n] = sum_k a[t, h * a_head_stride + k] * w[h, n, k] for w [heads, N, K].  bfloat16
     runs on warp-level MMAs where the strides allow.  ``rot`` (positions, frequencies, rot_dim, rot_dims, halves): a's heads
     hold ``rot_dim`` more values, which are turned by the rows' positions (as ``rope_heads`` does) and written behind the
-    head's N values in the same launch where that form applies."""
+    head's N values in the same launch where that form applies.  ``gate`` (float32 [rows, >= heads * N], any row stride): the
+    result times sigmoid(gate[t, h * N + n])."""
     H, N, K = w.shape
     if a.dtype != w.dtype or not w.is_contiguous() or a.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("linear_heads: a and w share a dtype, w contiguous [heads, N, K]")
     if tracing():
         _note("matmul", "matmul_heads", (M, K, H * N), 2.0 * M * H * N * K,
               w.numel() * w.element_size() + M * H * (K * a.element_size() + N * out.element_size()))
+    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1 or gate.shape[1] < H * N):
+        raise KernelError("linear_heads: the gate must be float32 [rows, >= heads * N] with contiguous rows")
+    gate_args = (_ptr(gate), gate.stride(0) if gate is not None else 0)
     if a.dtype == torch.bfloat16 and out.dtype in (torch.bfloat16, torch.float32) and \
             _can("nib_linear_heads_mma_supported", 16 + (_ptr(a) & 15), a.stride(0), a_head_stride, 16 + (_ptr(w) & 15), K):
         positions, freqs, rot_dim, rot_dims, halves = rot if rot is not None else (None, None, 0, 0, False)
         _check(library().nib_linear_heads_mma(_dt(out), _ptr(a), a.stride(0), a_head_stride, _ptr(w), _ptr(out), out.stride(0),
                                               out_head_stride, M, H, N, K, _ptr(positions), _ptr(freqs), int(rot_dim),
-                                              int(rot_dims), int(halves), _stream()), "linear_heads_mma")
+                                              int(rot_dims), int(halves), *gate_args, _stream()), "linear_heads_mma")
         return
     if rot is not None:
         positions, freqs, rot_dim, rot_dims, halves = rot
@@ -1344,7 +1374,7 @@ def linear_heads(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torc
             raise KernelError("linear_heads: with a rotated part a's heads are [K | rot_dim] and out is contiguous")
         rope_heads(a, K, rot_dim, rot_dims, freqs, positions, out.view(out.shape[0], H, out_head_stride), N, H, M, halves)
     _check(library().nib_linear_heads(_dt(a), _dt(out), _ptr(a), a.stride(0), a_head_stride, _ptr(w), _ptr(out),
-                                      out.stride(0), out_head_stride, M, H, N, K, _stream()), "linear_heads")
+                                      out.stride(0), out_head_stride, M, H, N, K, *gate_args, _stream()), "linear_heads")
 
 
 # ------------------------------------------------------------------------------ delta rule
@@ -1377,11 +1407,12 @@ def delta_rule(proj: torch.Tensor, offsets, wl: torch.Tensor, w0: torch.Tensor, 
 # ------------------------------------------------------------------------------ routed experts
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, T: int, top: int, renorm: bool, ids: torch.Tensor,
               weights: torch.Tensor, score: str = "softmax", choice_bias: Optional[torch.Tensor] = None,
-              n_real: Optional[int] = None, x: Optional[torch.Tensor] = None) -> None:
+              n_real: Optional[int] = None, x: Optional[torch.Tensor] = None,
+              logit_bias: Optional[torch.Tensor] = None) -> None:
     """Router logits in 32-bit, scores = softmax over all experts (or, ``score`` "sigmoid", each logit's sigmoid),
     the ``top`` largest (ties to the lower index) into ``ids`` int32 [T, top] with their scores in ``weights``
     float32 [T, top] (divided by their sum with ``renorm``).  ``choice_bias`` (float32 [experts]) is added to the
-    scores for the choice only.  The experts from ``n_real`` on have no matrices: a row that chooses one gets
+    scores for the choice only; ``logit_bias`` (float32 [experts]) to the logits themselves.  The experts from ``n_real`` on have no matrices: a row that chooses one gets
     score * h[t] added to ``x`` (float32 [T, C]) right here, and the id -1, which the expert kernels skip."""
     if score not in ("softmax", "sigmoid"):
         raise KernelError("moe_route: score is 'softmax' or 'sigmoid'")
@@ -1390,15 +1421,15 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, T: int, top: int, renorm:
         raise KernelError("moe_route: h and the router share a dtype")
     _i32(ids, "ids"); _f32(weights, "moe_route: weights")
     n_real = E if n_real is None else int(n_real)
-    if choice_bias is not None and (choice_bias.dtype != torch.float32 or choice_bias.numel() != E
-                                    or not choice_bias.is_contiguous()):
-        raise KernelError("moe_route: choice_bias must be contiguous float32 [experts]")
+    for b in (choice_bias, logit_bias):
+        if b is not None and (b.dtype != torch.float32 or b.numel() != E or not b.is_contiguous()):
+            raise KernelError("moe_route: choice_bias and logit_bias must be contiguous float32 [experts]")
     if n_real < E and (x is None or x.dtype != torch.float32 or not x.is_contiguous() or x.shape[1] != C):
         raise KernelError("moe_route: experts without matrices need the 32-bit x [T, C] to add into")
     if tracing():
         _note("matmul", "router", (T, C, E), 2.0 * T * C * E, (E + T) * C * h.element_size() + 8.0 * T * top)
     _check(library().nib_moe_route(_dt(h), _ptr(h), h.stride(0), _ptr(w_router), T, C, E, top, int(renorm),
-                                   int(score == "sigmoid"), _ptr(choice_bias), n_real, _ptr(x) if n_real < E else None, _ptr(ids),
+                                   int(score == "sigmoid"), _ptr(logit_bias), _ptr(choice_bias), n_real, _ptr(x) if n_real < E else None, _ptr(ids),
                                    _ptr(weights), _stream()), "moe_route")
 
 
@@ -1938,10 +1969,12 @@ def selective_scan(dtp: torch.Tensor, x: torch.Tensor, bc: torch.Tensor, b_off: 
 
 # ----------------------------------------------------------------------------- norms in groups
 def group_norm(x: torch.Tensor, weight: Optional[torch.Tensor], groups: int, eps: float, out: Optional[torch.Tensor],
-               n_rows: int, rows: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None) -> None:
+               n_rows: int, rows: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None,
+               add_rows: Optional[torch.Tensor] = None) -> None:
     """out[r] = norm(x[rows[r]]) (rows None: x[r]): the row cut into ``groups`` equal parts, each over its own root mean
     square (``eps`` inside the root), the whole times ``weight``; x is the 32-bit stream.  ``add`` (float32 [C]) is added
-    to the rows first, and x receives the sum; with ``out`` None that is all that happens."""
+    to the rows first (behind ``add_rows``, float32 [., C], a row of its own for each, where given), and x receives the sum;
+    with ``out`` None that is all that happens."""
     C = x.shape[1]
     _f32(x, "group_norm: x")
     if out is not None:
@@ -1954,12 +1987,17 @@ def group_norm(x: torch.Tensor, weight: Optional[torch.Tensor], groups: int, eps
         _f32(add, "group_norm: add")
         if add.numel() != C or rows is not None:
             raise KernelError("group_norm: add is one vector [C], for all rows in order")
+    if add_rows is not None:
+        _f32(add_rows, "group_norm: add_rows")
+        if add_rows.shape[1] != C or add_rows.shape[0] < n_rows or not add_rows.is_contiguous() or rows is not None:
+            raise KernelError("group_norm: add_rows is contiguous [rows, C], for all rows in order")
     if groups <= 0 or C % groups:
         raise KernelError("group_norm: the parts must divide the width")
     if tracing():
         _note("ln", "ln", (n_rows, C, groups), 4.0 * n_rows * C,
-              n_rows * C * (4 + (out.element_size() if out is not None else 0) + (4 if add is not None else 0)) + 4 * C)
-    _check(library().nib_group_norm(_dt(out) if out is not None else 0, _ptr(x), _ptr(rows), _ptr(add), _ptr(weight),
+              n_rows * C * (4 + (out.element_size() if out is not None else 0) + (4 if add is not None else 0)
+                             + (4 if add_rows is not None else 0)) + 4 * C)
+    _check(library().nib_group_norm(_dt(out) if out is not None else 0, _ptr(x), _ptr(rows), _ptr(add), _ptr(add_rows), _ptr(weight),
                                     _ptr(out), n_rows, C, int(groups), float(eps), _stream()), "group_norm")
 
 
@@ -2052,3 +2090,102 @@ def min_gru(proj: torch.Tensor, offsets, width: int, state: torch.Tensor, ctx, o
     _check(library().nib_min_gru(_dt(out), _ptr(proj), proj.stride(0), int(offsets[0]), int(offsets[1]), int(offsets[2]),
                                  int(width), _ptr(state), state.stride(0), _ptr(ctx.entry_start), _ptr(ctx.entry_slot),
                                  ctx.n_entries, ctx.n_rows, _ptr(out), out.stride(0), _stream()), "min_gru")
+
+
+# ----------------------------------------------------------------------------- attention with pooled blocks behind a window
+def conv_pool_append(proj: torch.Tensor, taps: int, w: torch.Tensor, state: Optional[torch.Tensor], n_head: int, n_kv_head: int,
+                     dim: int, norm: bool, eps: float, pool: int, ctx, q_out: torch.Tensor, cache: torch.Tensor,
+                     block_table: torch.Tensor, pool_table: Optional[torch.Tensor]) -> None:
+    """From the 32-bit projection ``proj`` (first n_head query heads, then n_kv_head key heads, of ``dim`` values each): a
+    short convolution over time on every channel (``w`` float32 [taps, channels], the last tap the current row's; what lies
+    before an entry's first row from ``state``, which then moves on), each head over its root mean square (``norm``; ``eps``
+    inside the root), the cast, padding to the cache's head size; queries to ``q_out``, keys to plane 0 of the rows' cache
+    slots and the key heads as they leave the convolution to plane 1.  ``pool`` > 0: a row that ends a block of ``pool``
+    positions also writes the block's mean key and value (of what the cache holds) to its row of the pages in
+    ``pool_table``.  A step in which every entry is one row is one launch."""
+    _f32(w, "conv_pool_append: w")
+    n_pages, two, g, page_size, hd = cache.shape
+    channels = (n_head + n_kv_head) * dim
+    if proj.dtype != torch.float32 or proj.stride(1) != 1 or proj.shape[1] < channels or tuple(w.shape) != (taps, channels) \
+            or not w.is_contiguous():
+        raise KernelError("conv_pool_append: proj float32 [rows, >= channels], w contiguous [taps, channels]")
+    if two != 2 or g != n_kv_head or not cache.is_contiguous() or cache.dtype != q_out.dtype or q_out.stride(1) != 1 \
+            or q_out.shape[1] != n_head * hd:
+        raise KernelError("conv_pool_append: cache contiguous [pages, 2, kv heads, page, head size] of q_out's dtype")
+    if taps > 1 and (state is None or state.dtype != torch.float32 or state.stride(1) != 1):
+        raise KernelError("conv_pool_append: more than one tap needs the requests' state in float32")
+    if pool > 0 and pool_table is None:
+        raise KernelError("conv_pool_append: pooled rows need pages of their own")
+    T = ctx.n_rows
+    alone = T == ctx.n_entries      # (every entry has a row, so as many rows as entries means one each)
+    if tracing():
+        n_out = (n_head + 2 * n_kv_head) * hd
+        _note("kv_write", "norm_kv_write", (T, n_out, taps), (2.0 * taps + 6.0) * T * channels,
+              T * (4.0 * channels + n_out * q_out.element_size()))
+    st = (_ptr(state), state.stride(0) if state is not None else 0)
+    _check(library().nib_conv_pool_append(
+        _dt(q_out), _ptr(proj), proj.stride(0), int(taps), _ptr(w), *st, _ptr(ctx.entry_start), _ptr(ctx.entry_slot),
+        _ptr(ctx.positions), _ptr(ctx.row_entry), n_head, n_kv_head, int(dim), hd, int(bool(norm)), float(eps), _ptr(q_out),
+        q_out.stride(0), _ptr(cache), _ptr(block_table), _ptr(pool_table), block_table.shape[1], page_size, n_pages, int(pool),
+        int(alone), T, _ptr(ctx.status), _stream()), "conv_pool_append")
+    if taps > 1 and not alone:
+        if tracing():
+            _note("other", "conv_state", (ctx.n_entries, channels, taps), 0.0, 8.0 * ctx.n_entries * channels * (taps - 1))
+        _check(library().nib_short_conv_state(_ptr(proj), proj.stride(0), 0, channels, int(taps), *st, _ptr(ctx.entry_start),
+                                              _ptr(ctx.entry_slot), ctx.n_entries, _stream()), "short_conv_state")
+
+
+def _pooled_keys(ctx, window: int, pool: int, single: bool) -> tuple:
+    """(keys seen by the step's single tokens, or by its portions' rows; cached rows that they read, each once an entry)."""
+    keys = rows = 0
+    seen = lambda p: min(p + 1, window) + max(0, p - window + 1) // pool if window > 0 and pool > 0 else \
+        (min(p + 1, window) if window > 0 else p + 1)
+    for e, p0 in enumerate(ctx.host_entry_pos0):
+        n = ctx.host_entry_start[e + 1] - ctx.host_entry_start[e]
+        if (n == 1) == single:
+            keys += sum(seen(p) for p in range(p0, p0 + n))
+            rows += seen(p0 + n - 1) + n - 1
+    return keys, rows
+
+
+def pooled_attention(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, ctx, n_head: int,
+                     dim: int, scale: float, window: int, plan, extras: AttnExtras) -> None:
+    """Attention of the step's rows over the last ``window`` positions (0: all) and, behind them, one key and value a block
+    (``extras.pool``), with learned sinks and a gate per element as ``extras`` has them; heads of ``dim`` values in rows of
+    the cache's size.  bfloat16 runs on the tensor cores (single tokens ``attention_group_mma``, portions
+    ``attention_wide_tc``) where the sizes and options allow; everything else on the general kernels."""
+    row_dim, sink = cache.shape[4], extras.sinks is not None
+    fast = q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and scale > 0.0 and extras.wide
+    options = dict(softcap=extras.softcap, gate=extras.gate, gate_dim=extras.gate_dim, sinks=extras.sinks, pool=extras.pool,
+                   pool_table=extras.pool_table)
+
+    def note(single: bool, n: int) -> None:
+        if tracing():
+            keys, rows = _pooled_keys(ctx, window, extras.pool, single)
+            _note_attention(n, keys, rows, n_head, cache.shape[2], row_dim, q.element_size(), (dim, dim, dim), out.element_size())
+
+    if plan.n_decode:
+        note(True, plan.n_decode)
+        if not (fast and attention_group_mma(q, cache, out, row_dim, block_table, ctx, plan, n_head, scale, window, row_dim,
+                                             row_dim, **options)):
+            _attention_general(q, cache, out, block_table, ctx, n_head, scale, window, plan, sink, extras, True)
+    if plan.n_prefill_rows:
+        note(False, plan.n_prefill_rows)
+        if not (fast and attention_wide_tc(q, cache, out, row_dim, block_table, ctx, plan, n_head, scale, window, 1, row_dim,
+                                           row_dim, **options)):
+            _attention_general(q, cache, out, block_table, ctx, n_head, scale, window, plan, sink, extras, False)
+
+
+def _attention_general(q, cache, out, block_table, ctx, n_head, scale, window, plan, sink, extras, single: bool) -> None:
+    """The step's single tokens, or its portions' rows, on the kernels that take every size and option."""
+    page_size, head_dim = cache.shape[3], cache.shape[4]
+    if single and page_size % 16 == 0 and head_dim % 8 == 0 and head_dim <= 128:
+        keys = plan.max_decode_keys if window <= 0 else min(plan.max_decode_keys, window)
+        attention_decode(q, cache, out, block_table, ctx.row_entry, ctx.positions, plan.n_decode, n_head, scale, window,
+                         ctx.status, keys, ctx.workspace, plan.decode_rows, sink=sink, extras=extras)
+        return
+    # (portions alone: all of the step's rows, those of no request among them, which the kernel leaves out)
+    rows, n = (plan.decode_rows, plan.n_decode) if single else (
+        plan.prefill_rows, plan.n_prefill_rows if plan.n_decode else ctx.n_rows)
+    attention_simt(q, cache, out, block_table, ctx.row_entry, ctx.positions, n, n_head, scale, window, ctx.status, rows,
+                   sink=sink, extras=extras)

@@ -63,6 +63,8 @@ class Model:
         self.stream_vectors = self._build(P.STREAM_VECTORS, spec.stream_vectors, "stream_vectors") \
             if spec.stream_vectors else None
         self.schedule = list(spec.schedule)
+        #: whether a run of the schedule adds the embedding's output to the stream
+        self.keeps_embedding = any(e.add_embedding for e in self.schedule)
         self._check_schedule()
         self.dtype: Optional[torch.dtype] = None
         self.device: Optional[torch.device] = None
@@ -179,6 +181,8 @@ class Model:
         sized for one row per batch entry (what generation asks for); a step that wants more (a
         replay that asks for every position) makes them grow, which drops captured graphs."""
         workspace.reserve("model.residual", limits.max_rows * self.width, torch.float32)
+        if self.keeps_embedding:
+            workspace.reserve("model.embedding", limits.max_rows * self.width, torch.float32)
         n = max(limits.max_entries, 1)
         workspace.reserve("model.final", n * self.width, limits.dtype)
         workspace.reserve("model.logits", n * _round_up(self.vocab_size, 16), torch.float32)
@@ -203,18 +207,23 @@ class Model:
         ws = ctx.workspace
         x = ws.get("model.residual", (ctx.max_rows, self.width), torch.float32)
         self.embedding.forward(ctx, x, self.position)
+        if self.keeps_embedding:      # (made twice: the stream changes in place)
+            start = ws.get("model.embedding", (ctx.max_rows, self.width), torch.float32)
+            self.embedding.forward(ctx, start, self.position)
         for i, e in enumerate(self.schedule):
             owner = i if e.cache_of is None else e.cache_of
             ctx.layer = i
-            # (an arrangement may take the next one's first step ahead, unless a vector is added to the stream in between)
+            # (an arrangement may take the next one's first step ahead, unless something is added to the stream in between)
             nxt = self.schedule[i + 1] if i + 1 < len(self.schedule) else None
-            ctx.next_block = self.layers[nxt.layer] if nxt is not None and nxt.add_vector is None else None
-            if e.add_vector is not None:
-                vector = self.stream_vectors.vector(e.add_vector)
+            plain_next = nxt is not None and nxt.add_vector is None and not nxt.add_embedding
+            ctx.next_block = self.layers[nxt.layer] if plain_next else None
+            if e.add_vector is not None or e.add_embedding:
+                vector = self.stream_vectors.vector(e.add_vector) if e.add_vector is not None else None
+                rows = start if e.add_embedding else None
                 if self.layers[e.layer].adds_vector:
-                    ctx.stream_vector = vector
+                    ctx.stream_vector, ctx.stream_rows = vector, rows
                 else:
-                    ops.group_norm(x, None, 1, 0.0, None, ctx.n_rows, add=vector)
+                    ops.group_norm(x, None, 1, 0.0, None, ctx.n_rows, add=vector, add_rows=rows)
             self.layers[e.layer].forward(x, ctx, caches.get(owner), states.get(i), e.cache_of is None, self.dtype)
         ctx.layer, ctx.next_block = -1, None
         if n_logits <= 0:

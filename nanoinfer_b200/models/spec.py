@@ -54,6 +54,9 @@ class ScheduleEntry:
     cache_of: Optional[int] = None
     #: row of the model's stream vectors that is added to the residual stream ahead of this run; None: nothing
     add_vector: Optional[int] = None
+    #: the embedding's output (the stream as it was ahead of the first run) is added to the stream ahead of this run, and
+    #: ahead of the vector
+    add_embedding: bool = False
 
 
 @dataclass

@@ -57,6 +57,9 @@ class KVCacheSpec:
     planes: int = 2
     #: with a window: the positions 0 .. keep_first - 1 stay readable behind it (their pages are never given back)
     keep_first: int = 0
+    #: with a window: every whole block of so many positions also leaves ONE pooled row (a key and a value) that stays
+    #: readable behind the window; the rows lie in pages of their own (``KVCacheView.pool_table``).  0: none
+    pool: int = 0
 
 
 @dataclass(frozen=True)
@@ -135,7 +138,8 @@ class StepPlan:
 
 
 class Norm(Part):
-    #: True: ``forward`` takes ``add``, a 32-bit vector that is added to the stream first, in the norm's own kernel
+    #: True: ``forward`` takes ``add``, a 32-bit vector that is added to the stream first, in the norm's own kernel, and
+    #: ``add_rows``, a 32-bit row for every row that is added ahead of it
     takes_vector = False
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, n_rows: int,
@@ -215,6 +219,8 @@ class TwoProducts:
     w_in: torch.Tensor
     b_in: Optional[torch.Tensor] = None
     w_out: torch.Tensor
+    #: a bias of the second product (float32 [width]) or None
+    b_out: Optional[torch.Tensor] = None
     n_in = n_inner = 0
 
     def rebase(self, w_in: torch.Tensor, b_in: Optional[torch.Tensor], w_out: torch.Tensor) -> None:
@@ -271,7 +277,7 @@ class TwoProducts:
         ops.linear(xn, self.w_in, self.b_in, proj, T)
         self.inner(proj, out, ctx, cache, state, writes_cache)
         ops.trace_scope(ctx.layer, names[1])
-        ops.linear(out, self.w_out, None, x, T, residual=True)
+        ops.linear(out, self.w_out, self.b_out, x, T, residual=True)
 
 
 class StreamVectors(Part):
@@ -372,6 +378,9 @@ class KVCacheView:
     block_table: torch.Tensor    # int32 [n_entries, max_blocks]; -1 where no page is held
     page_size: int
     window: int
+    #: where the layer keeps pooled rows: the columns of the block table that hold their pages (int32 [n_entries, .], the
+    #: row stride of ``block_table``); the pooled row of block b is row b % page_size of page b // page_size
+    pool_table: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -410,6 +419,8 @@ class StepContext:
     #: float32 [width], to be added to the stream ahead of the run that starts next (None: nothing); an arrangement
     #: that does this itself (``Block.adds_vector``) takes it away
     stream_vector: Optional[torch.Tensor] = None
+    #: float32 [rows, width], to be added to the stream ahead of the vector (None: nothing)
+    stream_rows: Optional[torch.Tensor] = None
     #: int32 [slots]: the token last sampled for each slot, left on the device by the sampler; a
     #: negative entry -(s + 1) of ``tokens`` stands for ``token_feedback[s]``
     token_feedback: Optional[torch.Tensor] = None

@@ -30,7 +30,8 @@ class Block:
     slots: ClassVar[Dict[str, Registry]] = {}
     #: names of ``slots`` that a layer may leave out
     optional: ClassVar[tuple] = ()
-    #: True: ``forward`` adds ``ctx.stream_vector`` to the stream itself before anything else (and takes it away)
+    #: True: ``forward`` adds ``ctx.stream_rows`` and ``ctx.stream_vector`` to the stream itself before anything else (and
+    #: takes them away)
     adds_vector: ClassVar[bool] = False
 
     def __init__(self, width: int, parts: Dict[str, Part]):
@@ -54,6 +55,19 @@ class Block:
     def prepare(self, dtype: torch.dtype, device: torch.device) -> None:
         """Called once after the parts' own ``prepare``."""
 
+    def _first_norm(self, x, xn, ctx) -> None:
+        """``norm_1`` of the stream into ``xn``, behind what is to be added to the stream first: in the norm's own kernel
+        where it takes that."""
+        T, norm = ctx.n_rows, self.norm_1
+        add, rows = ctx.stream_vector, ctx.stream_rows
+        ctx.stream_vector = ctx.stream_rows = None
+        if norm.takes_vector:
+            norm.forward(x, xn, T, add=add, add_rows=rows)
+            return
+        if add is not None or rows is not None:
+            ops.group_norm(x, None, 1, 0.0, None, T, add=add, add_rows=rows)
+        norm.forward(x, xn, T)
+
     def reserve(self, workspace: Workspace, limits: StepLimits) -> None:
         """Size the arrangement's own scratch (the parts size theirs themselves)."""
 
@@ -64,7 +78,18 @@ class Block:
 
 @register_block("pre_norm")
 class PreNormBlock(Block):
+    """A layer may have no feed-forward (and then no ``norm_2``).  What the schedule adds to the stream ahead of the layer is
+    added by the first norm's kernel where it takes that."""
+
     slots = {"norm_1": NORMS, "mixer": MIXERS, "norm_2": NORMS, "feed_forward": FEED_FORWARDS}
+    optional = ("norm_2", "feed_forward")
+    adds_vector = True
+
+    def __init__(self, width: int, parts: Dict[str, Part]):
+        super().__init__(width, parts)
+        if ("norm_2" in parts) != ("feed_forward" in parts):
+            raise ValueError("pre_norm: norm_2 and feed_forward come together or not at all")
+        self.norm_2, self.feed_forward = parts.get("norm_2"), parts.get("feed_forward")
 
     def reserve(self, workspace, limits) -> None:
         workspace.reserve("block.normed", limits.max_rows * self.width, limits.dtype)
@@ -81,8 +106,14 @@ class PreNormBlock(Block):
         return xn
 
     def forward(self, x, ctx, cache, state, writes_cache, dtype) -> None:
-        self.mixer.forward(self._normed(self.norm_1, self.mixer, x, ctx, dtype), x, ctx, cache, state, writes_cache)
-        self.feed_forward.forward(self._normed(self.norm_2, self.feed_forward, x, ctx, dtype), x, ctx)
+        if ctx.stream_vector is not None or ctx.stream_rows is not None:
+            xn = ctx.workspace.get("block.normed", (ctx.max_rows, self.width), dtype)
+            self._first_norm(x, xn, ctx)
+        else:
+            xn = self._normed(self.norm_1, self.mixer, x, ctx, dtype)
+        self.mixer.forward(xn, x, ctx, cache, state, writes_cache)
+        if self.feed_forward is not None:
+            self.feed_forward.forward(self._normed(self.norm_2, self.feed_forward, x, ctx, dtype), x, ctx)
 
 
 @register_block("post_norm_depth_mix")
@@ -340,8 +371,8 @@ class HyperConnectionBlock(Block):
 class ParallelNormBlock(Block):
     """One norm that both sublayers read, and one sum:
         h = norm_1(x);   x <- x + (mixer(h) + feed_forward(h))
-    (a layer may have no feed-forward).  A vector that the schedule adds to the stream ahead of the layer
-    (``ctx.stream_vector``) is added by the norm's kernel.
+    (a layer may have no feed-forward).  What the schedule adds to the stream ahead of the layer is added by the norm's
+    kernel.
 
     The norm is taken once, ahead of both, so both sublayers add their products straight into the stream.  Where both are
     ``TwoProducts`` parts the layer has two products in all: their first matrices lie under one another as one ([mixer's
@@ -355,8 +386,6 @@ class ParallelNormBlock(Block):
     def __init__(self, width: int, parts: Dict[str, Part]):
         super().__init__(width, parts)
         self.feed_forward = parts.get("feed_forward")
-        #: whether the norm's kernel adds a vector to the stream as well
-        self.norm_adds = parts["norm_1"].takes_vector
         self.joint = isinstance(self.mixer, TwoProducts) and isinstance(self.feed_forward, TwoProducts)
         if self.joint:
             m, f = self.mixer, self.feed_forward
@@ -371,6 +400,8 @@ class ParallelNormBlock(Block):
         if not self.joint:
             return
         m, f = self.mixer, self.feed_forward
+        if m.b_out is not None or f.b_out is not None:
+            raise ValueError("parallel_norm: a joint second product takes no bias")
         w_in = torch.zeros(self.n_in, self.width, dtype=dtype, device=device)
         w_in[:m.n_in], w_in[self.ff_row:self.ff_row + f.n_in] = m.w_in, f.w_in
         b_in = None
@@ -394,13 +425,7 @@ class ParallelNormBlock(Block):
     def forward(self, x, ctx, cache, state, writes_cache, dtype) -> None:
         T, ws = ctx.n_rows, ctx.workspace
         xn = ws.get("block.normed", (ctx.max_rows, self.width), dtype)
-        add, ctx.stream_vector = ctx.stream_vector, None
-        if self.norm_adds:
-            self.norm_1.forward(x, xn, T, add=add)
-        else:
-            if add is not None:
-                ops.group_norm(x, None, 1, 0.0, None, T, add=add)
-            self.norm_1.forward(x, xn, T)
+        self._first_norm(x, xn, ctx)
         m, f = self.mixer, self.feed_forward
         if not self.joint:
             m.forward(xn, x, ctx, cache, state, writes_cache)

@@ -14,7 +14,9 @@ W_uv, queries and window.  Rotation: interleaved pairs (2i, 2i+1) of the first `
 rotated part or, with ``rot_layout`` "halves", value i with value i + rot_dims / 2; angle = position *
 rot_base^(-2i / rot_dims).  ``head_gate``: head h's output is multiplied by sigmoid(W_g h)_h, one number per row
 and head; its logits are rows of the down-projections' product (32-bit), and the gate is applied to the head's
-weighted sum of latents.
+weighted sum of latents.  ``element_gate`` instead: W_g has a row for every element of the heads' values, and the heads'
+outputs are multiplied by its sigmoid in the product with W_uv.  ``learned_sink``: a number per head whose exponential joins
+the softmax's denominator (a key without a value, not scaled).
 """
 from __future__ import annotations
 
@@ -32,7 +34,8 @@ from .base import (INIT_ONE_PLUS_NORMAL, MATRIX, VECTOR, KVCacheSpec, KVCacheVie
 class LatentAttention(TwoProducts, Mixer):
     def __init__(self, width: int, n_head: int, nope_dim: int, rot_dim: int, v_dim: int, q_rank: int,
                  kv_rank: int, scale: float, eps: float, window: int = 0, rot_base: float = 10000.0,
-                 rot_dims: Optional[int] = None, own_kv: bool = True, rot_layout: str = "pairs", head_gate: bool = False):
+                 rot_dims: Optional[int] = None, own_kv: bool = True, rot_layout: str = "pairs", head_gate: bool = False,
+                 element_gate: bool = False, learned_sink: bool = False):
         rot_dims = rot_dim if rot_dims is None else rot_dims
         for name, v in (("width", width), ("n_head", n_head), ("v_dim", v_dim), ("q_rank", q_rank),
                         ("kv_rank", kv_rank)):
@@ -51,11 +54,15 @@ class LatentAttention(TwoProducts, Mixer):
         self.latent_dim = self.kv_rank + self.rot_dim
         if rot_layout not in ("pairs", "halves"):
             raise ValueError(f"latent_attention: rot_layout {rot_layout!r} is not 'pairs' or 'halves'")
+        if head_gate and element_gate:
+            raise ValueError("latent_attention: a gate per head or per element, not both")
         self.halves, self.head_gate = rot_layout == "halves", bool(head_gate)
+        self.element_gate, self.learned_sink = bool(element_gate), bool(learned_sink)
+        self.n_gate = self.n_head if self.head_gate else self.n_head * self.v_dim if self.element_gate else 0
         #: columns of the down-projections' product: the query latent, the key/value latent and the rotated part (not
         #: in a layer on another's cache), the gate's logits
         self.gate_off = self.q_rank + (self.latent_dim if self.own_kv else 0)
-        self.n_in = self.gate_off + (self.n_head if self.head_gate else 0)
+        self.n_in = self.gate_off + self.n_gate
         self.n_inner = self.n_head * self.v_dim
 
     def param_specs(self) -> List[ParamSpec]:
@@ -69,8 +76,10 @@ class LatentAttention(TwoProducts, Mixer):
         specs += [ParamSpec("k_up", (H * self.nope_dim, self.kv_rank), MATRIX),
                   ParamSpec("v_up", (H * self.v_dim, self.kv_rank), MATRIX),
                   ParamSpec("out_weight", (self.width, H * self.v_dim), MATRIX)]
-        if self.head_gate:
-            specs.append(ParamSpec("gate_weight", (H, self.width), MATRIX))
+        if self.n_gate:
+            specs.append(ParamSpec("gate_weight", (self.n_gate, self.width), MATRIX))
+        if self.learned_sink:
+            specs.append(ParamSpec("sink", (H,), VECTOR))
         return specs
 
     def kv_spec(self) -> Optional[KVCacheSpec]:
@@ -86,7 +95,7 @@ class LatentAttention(TwoProducts, Mixer):
         super().prepare(dtype, device)
         p, H = self.params, self.n_head
         # the down-projections and the gate read the same rows: one product
-        keys = ["q_down"] + (["kv_down"] if self.own_kv else []) + (["gate_weight"] if self.head_gate else [])
+        keys = ["q_down"] + (["kv_down"] if self.own_kv else []) + (["gate_weight"] if self.n_gate else [])
         self.w_in = torch.cat([p[k] for k in keys], 0).contiguous()
         self.w_out, at = p["out_weight"], 0
         for k in keys:
@@ -144,6 +153,8 @@ class LatentAttention(TwoProducts, Mixer):
                                                                  device=proj.device)
         lat = ws.get("latent.out", (n, H * self.kv_rank), self.dtype)
         ops.latent_attention(qf, cache.layer, lat, cache.block_table, ctx, H, self.kv_rank, self.scale, self.window,
-                             gate=proj[:, self.gate_off:self.gate_off + H] if self.head_gate else None, plan=plan)
+                             gate=proj[:, self.gate_off:self.gate_off + H] if self.head_gate else None, plan=plan,
+                             sinks=p.get("sink"))
         ops.trace_scope(ctx.layer, "v_up")
-        ops.linear_heads(lat, self.kv_rank, self.v_up, out, self.v_dim, T)
+        ops.linear_heads(lat, self.kv_rank, self.v_up, out, self.v_dim, T,
+                         gate=proj[:, self.gate_off:self.gate_off + self.n_gate] if self.element_gate else None)

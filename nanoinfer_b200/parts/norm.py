@@ -85,18 +85,26 @@ class ScalarRMSNorm(RMSNorm):
 class GroupedRMSNorm(Norm):
     """An RMS norm in groups: the vector is cut into ``groups`` equal consecutive parts, each part is divided by its own
     sqrt(mean(part^2) + eps), and the whole is multiplied by one weight of the vector's size; statistics in 32-bit.  One
-    group is the plain RMS norm.  ``add`` (a 32-bit vector) is added to the stream first, in the same kernel."""
+    group is the plain RMS norm.  ``add`` (a 32-bit vector) and ``add_rows`` (a 32-bit row for each) are added to the stream
+    first, in the same kernel.  ``one_plus``: as in ``rmsnorm``."""
 
     takes_vector = True
 
-    def __init__(self, width: int, eps: float, groups: int = 1):
+    def __init__(self, width: int, eps: float, groups: int = 1, one_plus: bool = False):
         if groups <= 0 or width % groups:
             raise ValueError(f"grouped_rmsnorm: {groups} groups do not divide a width of {width}")
-        self.width, self.eps, self.groups = int(width), float(eps), int(groups)
+        self.width, self.eps, self.groups, self.one_plus = int(width), float(eps), int(groups), bool(one_plus)
+        self._shifted = False
 
     def param_specs(self) -> List[ParamSpec]:
-        return [ParamSpec("weight", (self.width,), VECTOR, INIT_ONE_PLUS_NORMAL)]
+        return [ParamSpec("weight", (self.width,), VECTOR, INIT_NORMAL if self.one_plus else INIT_ONE_PLUS_NORMAL)]
+
+    def prepare(self, dtype, device) -> None:
+        super().prepare(dtype, device)
+        if self.one_plus and not self._shifted:
+            self.params["weight"] = self.params["weight"] + 1.0
+            self._shifted = True
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, n_rows: int, rows: Optional[torch.Tensor] = None,
-                add: Optional[torch.Tensor] = None) -> None:
-        ops.group_norm(x, self.params["weight"], self.groups, self.eps, out, n_rows, rows, add)
+                add: Optional[torch.Tensor] = None, add_rows: Optional[torch.Tensor] = None) -> None:
+        ops.group_norm(x, self.params["weight"], self.groups, self.eps, out, n_rows, rows, add, add_rows)

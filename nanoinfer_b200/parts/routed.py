@@ -13,7 +13,8 @@ expert; gate and value rows are interleaved into one matrix at load, so that one
 experts is not the same as scaling the output (the first product is linear, so the kernels scale its results
 before the activation); ``shared_row_gate``: the shared expert's output times sigmoid(w_sg . h), one number a row
 (its row rides in the shared expert's first product); ``choice_bias``: a learned number per expert that is added
-to the scores for the CHOICE only (the weights stay the scores); ``n_identity`` > 0: the router has that many outputs
+to the scores for the CHOICE only (the weights stay the scores); ``router_bias``: a learned number per expert that is
+added to the LOGITS, for choice and weights alike; ``n_identity`` > 0: the router has that many outputs
 more than there are experts with matrices, and a row that chooses one of them gets its own input back, times the
 score (the routing kernel adds it, the expert kernels skip the choice); activation "swiglu_capped" (gated experts):
 g' = min(g, act_limit), u' = clamp(u, -act_limit, act_limit), g' sigmoid(1.702 g') (u' + 1).
@@ -37,7 +38,7 @@ class RoutedExperts(FeedForward):
     def __init__(self, width: int, n_expert: int, top: int, inner: int, activation: str = "erf",
                  renorm: bool = False, shared_inner: int = 0, shared_activation: str = "erf",
                  score: str = "softmax", gated: bool = False, weight_on: str = "output", shared_row_gate: bool = False,
-                 choice_bias: bool = False, n_identity: int = 0, act_limit: float = 0.0):
+                 choice_bias: bool = False, n_identity: int = 0, act_limit: float = 0.0, router_bias: bool = False):
         if n_identity < 0 or not 0 < top <= n_expert + n_identity:
             raise ValueError(f"routed_experts: top {top} must be between 1 and the number of experts {n_expert} "
                              f"(+ {n_identity} without matrices)")
@@ -67,6 +68,7 @@ class RoutedExperts(FeedForward):
         self.last_ids: Optional[torch.Tensor] = None
         self.shared_row_gate = bool(shared_row_gate)
         self.choice_bias, self.n_identity, self.act_limit = bool(choice_bias), int(n_identity), float(act_limit)
+        self.router_bias = bool(router_bias)
         #: outputs of the router: the experts with matrices, then those without
         self.n_routes = self.n_expert + self.n_identity
 
@@ -74,6 +76,8 @@ class RoutedExperts(FeedForward):
         specs = [ParamSpec("router", (self.n_routes, self.width), MATRIX)]
         if self.choice_bias:
             specs.append(ParamSpec("choice_bias", (self.n_routes,), VECTOR))
+        if self.router_bias:
+            specs.append(ParamSpec("router_bias", (self.n_routes,), VECTOR))
         for e in range(self.n_expert):
             if self.gated:
                 specs.append(ParamSpec(f"expert{e}_gate", (self.inner, self.width), MATRIX))
@@ -148,7 +152,7 @@ class RoutedExperts(FeedForward):
         weights = ws.get("moe.weights", (n, self.top), torch.float32)
         ops.trace_scope(ctx.layer, "router")
         ops.moe_route(xn, p["router"], T, self.top, self.renorm, ids, weights, score=self.score,
-                      choice_bias=p.get("choice_bias"), n_real=self.n_expert, x=x)
+                      choice_bias=p.get("choice_bias"), n_real=self.n_expert, x=x, logit_bias=p.get("router_bias"))
         inner = ws.get("moe.inner", (n * self.top, self.inner), self.dtype)
         ops.trace_scope(ctx.layer, "experts")
         ops.moe_experts(xn, self.w_up, self.w_down, ids, weights, inner, x, T, self.top,

@@ -96,5 +96,10 @@ def _register_builtin() -> None:
 
     register_architecture("Dedunex", DedunexConfig, build_dedunex_spec)
 
+    from .config.pasopel import PasopelConfig
+    from .models.pasopel import build_pasopel_spec
+
+    register_architecture("Pasopel", PasopelConfig, build_pasopel_spec)
+
 
 _register_builtin()

@@ -522,6 +522,28 @@ def dedunex_like(width: int, n_layer: int, vocab: int, window: int = 512) -> dic
                 loop=dict(start=0, stop=n_layer, times=1), layers=layers)
 
 
+def pasopel_like(width: int, n_layer: int, vocab: int, window: int = 512, pool: int = 16) -> dict:
+    """A Pasopel configuration whose layers have the sizes of a GPT-2 of ``width``: by turns attention over a window with
+    pooled blocks of 16 behind it (heads of 64, a key head for about four query heads, four taps; a window of half of
+    ``window``, so that a context of twice that has blocks to see) with a dense feed-forward of 4 x width, attention through a
+    latent of 256 + 32 (heads of 64, a window of ``window``) with eight gated experts of the model's width of which a row
+    visits two beside a shared one, pooled attention with such experts, and latent attention with a dense feed-forward; the
+    stack runs once, with its vector."""
+    heads = width // 64
+    kv_heads = max(d for d in range(1, max(1, heads // 4) + 1) if heads % d == 0)
+    att = dict(heads=heads, kv_heads=kv_heads, dim=64, vdim=64, conv=4, scale=0.125, mask=dict(size=window // 2, pool=pool))
+    lat = dict(heads=heads, dim=64, rot_dim=32, vdim=64, q_rank=width // 2, kv_rank=256, scale=96 ** -0.5,
+               mask=dict(size=window), rot=dict(base=10000.0, dims=32))
+    moe = dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=width), shared=dict(ff=width))
+    dense = dict(kind="dense", ff=4 * width)
+    layers = []
+    for i in range(n_layer):
+        kind, m = (("attention", att), ("latent_attention", lat))[i % 2]
+        layers.append(dict(type=kind, mixer=json.loads(json.dumps(m)), mlp=json.loads(json.dumps((dense, moe, moe, dense)[i % 4]))))
+    return dict(architecture="Pasopel", vocab=vocab, width=width, norm=dict(eps=1e-6), logit_softcap=30.0,
+                loop=dict(start=0, stop=n_layer, times=1), layers=layers)
+
+
 def folder_of(raw: dict, seed: int, dtype: torch.dtype) -> str:
     """A folder with seeded random weights of the configuration ``raw`` (made once, in the temporary folder)."""
     from .config.base import architecture_name
@@ -577,7 +599,7 @@ def profile_forward(eng, prompt, batch: int, repeats: int = 3):
 
 def compare_designs(widths=(768, 1024, 1600), n_layer: int = 4, batch: int = 8, context: int = 1024,
                     steps: int = 64, warmup: int = 8, designs=("vadonex", "gpt2")) -> List[dict]:
-    """The ``designs`` (of "dedunex", "nagilix", "kemuzen", "mulavik", "vadonex", "gpt2") side by side at equal width, depth, vocabulary and
+    """The ``designs`` (of "pasopel", "dedunex", "nagilix", "kemuzen", "mulavik", "vadonex", "gpt2") side by side at equal width, depth, vocabulary and
     context (random weights, bfloat16): one prompt of ``context - steps - warmup`` tokens in one step, decode at
     ``batch``, and where the time of each goes op by op with every op's fraction of its roofline (measured
     peaks)."""
@@ -591,7 +613,8 @@ def compare_designs(widths=(768, 1024, 1600), n_layer: int = 4, batch: int = 8, 
                 "mulavik": lambda: mulavik_like(width, n_layer, 50257),
                 "kemuzen": lambda: kemuzen_like(width, n_layer, 50257),
                 "nagilix": lambda: nagilix_like(width, n_layer, 50257, context),
-                "dedunex": lambda: dedunex_like(width, n_layer, 50257)}
+                "dedunex": lambda: dedunex_like(width, n_layer, 50257),
+                "pasopel": lambda: pasopel_like(width, n_layer, 50257)}
         for name in designs:
             raw = made[name]()
             d = folder_of(raw, 1234, torch.bfloat16)

@@ -309,12 +309,16 @@ class CacheManager:
         """How many tokens the request could append with so many free pages per group (None: any number)."""
         most = None
         for g, blocks, pooled, f in zip(self.groups, req.blocks, req.pooled, free):
-            k = f                # pages for positions; what is left must do for the pooled rows
-            while k > 0 and k + max(0, self._pool_pages(g, (len(blocks) + k) * self.page_size) - len(pooled)) > f:
-                k -= 1
-            n = (len(blocks) + k) * self.page_size - req.n_tokens
-            while n > 0 and self._pool_pages(g, req.n_tokens + n) - len(pooled) > f - k:
-                n -= 1
+            n = (len(blocks) + f) * self.page_size - req.n_tokens      # if the pooled rows took no page
+            if g.spec.pool > 0:
+                def fits(k: int) -> bool:
+                    end = req.n_tokens + k
+                    return max(0, -(-end // self.page_size) - len(blocks)) + max(0, self._pool_pages(g, end) - len(pooled)) <= f
+                lo, hi = 0, max(0, n)
+                while lo < hi:
+                    mid = (lo + hi + 1) // 2
+                    lo, hi = (mid, hi) if fits(mid) else (lo, mid - 1)
+                n = lo
             most = n if most is None else min(most, n)
         return most
 

@@ -5,6 +5,7 @@ from .kemuzen import KemuzenConfig
 from .mulavik import MulavikConfig
 from .nagilix import NagilixConfig
 from .dedunex import DedunexConfig
+from .pasopel import PasopelConfig
 
 __all__ = ["ConfigError", "ModelConfig", "field", "read_config_json", "architecture_name", "GPT2Config", "VadonexConfig",
-           "MulavikConfig", "KemuzenConfig", "NagilixConfig", "DedunexConfig"]
+           "MulavikConfig", "KemuzenConfig", "NagilixConfig", "DedunexConfig", "PasopelConfig"]

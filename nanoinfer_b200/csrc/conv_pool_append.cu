@@ -121,7 +121,7 @@ conv_pool_append_kernel(const ConvPoolParams<T> prm) {
           const float r = head_row(H + g, pos - p, v);
 #pragma unroll
           for (int n = 0; n < ND; ++n) {
-            ks[n] += to_float(from_float<T>(v[n] * r));
+            ks[n] += to_float(from_float<T>(__fmul_rn(v[n], r)));   // (the cached value: no multiply-add across it)
             vs[n] += to_float(from_float<T>(v[n]));
           }
         } else {

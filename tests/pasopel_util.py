@@ -66,10 +66,12 @@ def write_model(cfg_dict, out_dir, dtype=torch.float32, seed=1, sharpen=3.0):
     for name, t in tensors.items():
         leaf = name.split(".", 1)[1] if name.startswith("l") and name[1].isdigit() else name
         if name == "embed":
-            t.copy_(rn(t, 0.8))
+            t.copy_(rn(t, 0.5))
         elif name == "loop.step":
-            t.copy_(rn(t, 0.7))
-        elif leaf in ("norm1", "norm2", "final.norm"):
+            t.copy_(rn(t, 0.3))
+        elif name == "final.norm":
+            t.copy_(rn(t) - 1.0)      # (signs of its own: the tied table does not give every token back at once)
+        elif leaf in ("norm1", "norm2"):
             t.copy_(1.2 * ru(t) - 0.6)
         elif leaf in ("mix.dq.norm", "mix.dkv.norm"):
             t.copy_(0.5 + ru(t))
@@ -92,3 +94,16 @@ def write_model(cfg_dict, out_dir, dtype=torch.float32, seed=1, sharpen=3.0):
         json.dump(cfg.to_dict(), fh)
     write_safetensors(os.path.join(out_dir, "model.safetensors"), {k: v.to(dtype) for k, v in tensors.items()})
     return out_dir
+
+
+#: a router whose choice hangs on less than this (of logits of size one) may choose otherwise in bfloat16
+CLOSE_CALL = 0.05
+
+
+def assert_close_where_routing_is_clear(errs, margins, dtype, what=""):
+    """``assert_close``; in bfloat16 over the positions at which no router's choice is a close call."""
+    if dtype != "float32":
+        clear = margins >= CLOSE_CALL
+        assert int(clear.sum()) * 4 >= len(clear), f"{what}: too few positions with a clear choice to say anything"
+        errs = errs[clear.to(errs.device)]
+    assert_close(errs, dtype, what)

@@ -141,6 +141,12 @@ def router_choice(h: torch.Tensor, w: Tensors, p: str, top: int):
     return best.indices, torch.softmax(best.values, dim=1)
 
 
+def router_margin(h: torch.Tensor, w: Tensors, p: str, top: int) -> torch.Tensor:
+    """How far the last chosen expert's logit lies above the first one left out, per row (a large number: none is)."""
+    z = (h @ w[p + "router"].T + w[p + "router.b"]).sort(dim=1, descending=True).values
+    return z[:, top - 1] - z[:, top] if z.shape[1] > top else torch.full((h.shape[0],), math.inf, dtype=torch.float64)
+
+
 def routed_feed_forward(h: torch.Tensor, w: Tensors, p: str, m: dict) -> torch.Tensor:
     ids, s = router_choice(h, w, p, m["router"]["top"])
     out = torch.zeros_like(h)
@@ -168,8 +174,10 @@ def run_order(cfg: dict) -> List[tuple]:
     return order + [(i, None) for i in range(b, n)]
 
 
-def forward(cfg: dict, w: Tensors, tokens: Sequence[int], layers_out: Optional[list] = None) -> torch.Tensor:
-    """Logits [n, vocab] of a whole sequence.  ``layers_out`` receives the stream after every layer run."""
+def forward(cfg: dict, w: Tensors, tokens: Sequence[int], layers_out: Optional[list] = None,
+            margins_out: Optional[list] = None) -> torch.Tensor:
+    """Logits [n, vocab] of a whole sequence.  ``layers_out`` receives the stream after every layer run, ``margins_out``
+    every router's margin per position."""
     w = {k: v.to(torch.float64) for k, v in w.items()}
     eps = cfg["norm"]["eps"]
     start = x = w["embed"][torch.tensor(list(tokens), dtype=torch.long)]
@@ -183,6 +191,8 @@ def forward(cfg: dict, w: Tensors, tokens: Sequence[int], layers_out: Optional[l
         mlp = layer.get("mlp")
         if mlp is not None:
             h = norm_around_zero(x, w[p + "norm2"], eps)
+            if margins_out is not None and mlp["kind"] == "moe":
+                margins_out.append(router_margin(h, w, p + "mlp.", mlp["router"]["top"]))
             x = x + (dense_feed_forward(h, w, p + "mlp.") if mlp["kind"] == "dense"
                      else routed_feed_forward(h, w, p + "mlp.", mlp))
         if layers_out is not None:
@@ -213,6 +223,12 @@ class PlainPasopel:
 
     def logits(self, tokens: Sequence[int], layers_out: Optional[list] = None) -> torch.Tensor:
         return forward(self.cfg, self.w, tokens, layers_out)
+
+    def margins(self, tokens: Sequence[int]) -> torch.Tensor:
+        """The smallest margin of any router, per position (infinite in a model without routers)."""
+        out: List[torch.Tensor] = []
+        forward(self.cfg, self.w, tokens, None, out)
+        return torch.stack(out).min(dim=0).values if out else torch.full((len(tokens),), math.inf, dtype=torch.float64)
 
     def greedy(self, prompt: Sequence[int], n: int) -> List[int]:
         """The ``n`` tokens that greedy decoding appends to ``prompt`` (ties to the lower index)."""

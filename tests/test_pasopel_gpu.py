@@ -10,7 +10,7 @@ import random
 import pytest
 import torch
 
-from pasopel_util import TOL, assert_close, config, dense, latent_layer, moe, pooled_layer, rel_err, row_errs, write_model
+from pasopel_util import TOL, assert_close_where_routing_is_clear, config, dense, latent_layer, moe, pooled_layer, rel_err, row_errs, write_model
 from test_dedunex_gpu import _latent_cache
 from test_mulavik_gpu import step_ctx, toks
 
@@ -349,7 +349,7 @@ class Harness:
         return torch.cat(rows)
 
     def check(self, got, tokens, what=""):
-        assert_close(row_errs(got, self.plain.logits(tokens)), self.dtype, what)
+        assert_close_where_routing_is_clear(row_errs(got, self.plain.logits(tokens)), self.plain.margins(tokens), self.dtype, what)
 
 
 ONE_LAYER = {
@@ -620,7 +620,8 @@ def test_random_configuration_cut_at_random(case, dtype, tmp_path):
     want = [h.plain.logits(t) for t in prompts]
     keys = sorted(got)
     errs = row_errs(torch.stack([got[k] for k in keys]), torch.stack([want[i][p] for i, p in keys]))
-    assert_close(errs, dtype, f"case {case} {json.dumps(cfg)} at (request, position) {keys}")
+    sure = [h.plain.margins(t) for t in prompts]
+    assert_close_where_routing_is_clear(errs, torch.stack([sure[i][p] for i, p in keys]), dtype, f"case {case} {json.dumps(cfg)} at (request, position) {keys}")
 
 
 def test_greedy_generation_through_the_engine_and_its_scheduler(tmp_path):

@@ -78,6 +78,9 @@ int nib_linear_tc_supported(const void* a, int lda, const void* w, int ldw, int 
 int nib_linear_tc(int out_dtype, const void* a, int lda, const void* w, int ldw, const float* bias,
                   void* out, int ldo, int M, int N, int K, int act, int residual, int* status,
                   cudaStream_t stream);
+// w [K / seg_k, N, seg_k]: stacked matrices, one product whose K walks them (seg_k a multiple of 64)
+int nib_linear_tc_segments(int out_dtype, const void* a, int lda, const void* w, int seg_k, const float* bias, void* out,
+                           int ldo, int M, int N, int K, int act, int residual, int* status, cudaStream_t stream);
 
 // The general tensor-core product for steps of at most 128 rows, with three options: activations made
 // in the kernel by LayerNorm of the 32-bit residual stream (ln_x), keys and values written straight

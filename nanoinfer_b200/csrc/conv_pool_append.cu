@@ -8,10 +8,12 @@
 //            means of what the cache holds, as row (position / pool) of the request's pooled pages (same cache)
 // in one kernel, and in a step whose entries are one row each the convolution's state as well.
 //
-// A block owns a row and eight heads, a warp a head.  The keys of a pooled block that came with this step may not be in the
-// cache yet (other blocks of the launch write them): they are made again from the projection, with the same rounding; those
-// of earlier steps are read from the cache.  The eight warps share a block's positions (by index modulo eight) and add up in
-// warp order, so a mean does not depend on how the prompt was cut.
+// A block owns a row and eight heads, a warp a head; the pooled rows are made by blocks of their own (a row and a key head,
+// which leave at once where the row ends no block) unless every entry is one row, where the block that owns the key head does
+// it.  The keys of a pooled block that came with this step may not be in the cache yet (other blocks of the launch write them):
+// they are made again from the projection, with the same rounding; those of earlier steps are read from the cache.  The eight
+// warps share a block's positions (by index modulo eight) and add up in warp order, so a mean does not depend on how the
+// prompt was cut.  The usual numbers of taps are compiled in, so that all of a head's loads travel together.
 #include "api.h"
 #include "common.cuh"
 
@@ -38,10 +40,11 @@ struct ConvPoolParams {
   const int* block_table;
   const int* pool_table;
   int max_blocks, page_size, n_pages, pool, shift_state;
+  int head_blocks;             // blocks of eight heads a row; behind them, a block a key head for the pooled rows
   int* status;
 };
 
-template <typename T, int ND>
+template <typename T, int ND, int TAPS>
 __global__ void __launch_bounds__(CP_WARPS * 32)
 conv_pool_append_kernel(const ConvPoolParams<T> prm) {
   pdl_trigger();
@@ -50,7 +53,9 @@ conv_pool_append_kernel(const ConvPoolParams<T> prm) {
   const int entry = prm.row_entry[t];
   if (entry < 0) return;                           // a row of no request
   const int pos = prm.positions[t], i = t - prm.entry_start[entry];
-  const int dim = prm.dim, hd = prm.hd, taps = prm.taps, H = prm.n_head, G = prm.n_kv_head;
+  const int dim = prm.dim, hd = prm.hd, taps = TAPS > 0 ? TAPS : prm.taps, H = prm.n_head, G = prm.n_kv_head;
+  const bool pools = (int)blockIdx.y >= prm.head_blocks, ends = prm.pool > 0 && (pos + 1) % prm.pool == 0;
+  if (pools && !ends) return;
   const int channels = (H + G) * dim;
   float* st = prm.state + (size_t)prm.entry_slot[entry] * prm.state_stride;
   const int* table = prm.block_table + (size_t)entry * prm.max_blocks;
@@ -74,11 +79,21 @@ conv_pool_append_kernel(const ConvPoolParams<T> prm) {
       const int d = lane + 32 * n, c = unit * dim + d;
       float acc = 0.0f;
       if (d < dim) {
-        for (int j = 0; j < taps; ++j) {
+        auto at = [&](int j) -> const float* {
           const int src = i - back - (taps - 1 - j);
-          const float x = src >= 0 ? prm.proj[(size_t)(t - back - (taps - 1 - j)) * prm.ld + c]
-                                   : st[(size_t)(taps - 1 + src) * channels + c];
-          acc = fmaf(prm.w[(size_t)j * channels + c], x, acc);
+          return src >= 0 ? prm.proj + (size_t)(t - back - (taps - 1 - j)) * prm.ld + c : st + (size_t)(taps - 1 + src) * channels + c;
+        };
+        if constexpr (TAPS > 0) {
+          float x[TAPS], w[TAPS];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) {
+            x[j] = *at(j);
+            w[j] = prm.w[(size_t)j * channels + c];
+          }
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], x[j], acc);
+        } else {
+          for (int j = 0; j < taps; ++j) acc = fmaf(prm.w[(size_t)j * channels + c], *at(j), acc);
         }
       }
       v[n] = acc;
@@ -88,7 +103,7 @@ conv_pool_append_kernel(const ConvPoolParams<T> prm) {
   };
 
   const int u0 = blockIdx.y * CP_WARPS, unit = u0 + warp;
-  if (unit < H + G) {
+  if (!pools && unit < H + G) {
     float v[ND];
     const float r = head_row(unit, 0, v);
     if (unit < H) {
@@ -109,9 +124,11 @@ conv_pool_append_kernel(const ConvPoolParams<T> prm) {
       }
     }
   }
-  if (prm.pool > 0 && (pos + 1) % prm.pool == 0) {
+  if (ends && (pools || prm.shift_state)) {
     const int P = prm.pool, first = pos + 1 - P;
-    for (int g = max(u0 - H, 0); g < min(u0 + CP_WARPS - H, G); ++g) {
+    const int g0 = pools ? (int)blockIdx.y - prm.head_blocks : max(u0 - H, 0);
+    const int g1 = pools ? g0 + 1 : min(u0 + CP_WARPS - H, G);
+    for (int g = g0; g < g1; ++g) {
       float ks[ND], vs[ND];
 #pragma unroll
       for (int n = 0; n < ND; ++n) ks[n] = vs[n] = 0.0f;
@@ -164,14 +181,24 @@ conv_pool_append_kernel(const ConvPoolParams<T> prm) {
   }
 }
 
-template <typename T>
+template <typename T, int TAPS>
 static int launch_conv_pool_append(const ConvPoolParams<T>& prm, int n_rows, cudaStream_t stream) {
-  const dim3 grid(n_rows, (prm.n_head + prm.n_kv_head + CP_WARPS - 1) / CP_WARPS);
+  const dim3 grid(n_rows, prm.head_blocks + (prm.pool > 0 && !prm.shift_state ? prm.n_kv_head : 0)), block(CP_WARPS * 32);
   const size_t smem = prm.pool > 0 ? (size_t)CP_WARPS * 2 * prm.hd * sizeof(float) : 0;
-  if (prm.hd <= 64) launch_pdl(conv_pool_append_kernel<T, 2>, grid, dim3(CP_WARPS * 32), smem, stream, prm);
-  else if (prm.hd <= 128) launch_pdl(conv_pool_append_kernel<T, 4>, grid, dim3(CP_WARPS * 32), smem, stream, prm);
-  else launch_pdl(conv_pool_append_kernel<T, 8>, grid, dim3(CP_WARPS * 32), smem, stream, prm);
+  if (prm.hd <= 64) launch_pdl(conv_pool_append_kernel<T, 2, TAPS>, grid, block, smem, stream, prm);
+  else if (prm.hd <= 128) launch_pdl(conv_pool_append_kernel<T, 4, TAPS>, grid, block, smem, stream, prm);
+  else launch_pdl(conv_pool_append_kernel<T, 8, TAPS>, grid, block, smem, stream, prm);
   NIB_LAUNCH_CHECK();
+}
+template <typename T>
+static int pick_conv_pool_append(const ConvPoolParams<T>& prm, int n_rows, cudaStream_t stream) {
+  switch (prm.taps) {
+    case 1: return launch_conv_pool_append<T, 1>(prm, n_rows, stream);
+    case 2: return launch_conv_pool_append<T, 2>(prm, n_rows, stream);
+    case 3: return launch_conv_pool_append<T, 3>(prm, n_rows, stream);
+    case 4: return launch_conv_pool_append<T, 4>(prm, n_rows, stream);
+  }
+  return launch_conv_pool_append<T, 0>(prm, n_rows, stream);
 }
 
 }  // namespace nib
@@ -189,7 +216,7 @@ extern "C" int nib_conv_pool_append(int dtype, const float* proj, int ld, int ta
                                     const int* pool_table, int max_blocks, int page_size, int n_pages, int pool,
                                     int shift_state, int T, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (taps < 1 || taps > 64 || dim <= 0 || dim > hd || hd > 256 || (n_head + n_kv_head) > CP_WARPS * 65535)
+  if (taps < 1 || taps > 64 || dim <= 0 || dim > hd || hd > 256 || n_head + 2 * n_kv_head > 65535)
     return NIB_ERR_UNSUPPORTED_SIZE;
   if (n_head <= 0 || n_kv_head <= 0 || page_size <= 0 || pool < 0 || (pool > 0 && pool_table == nullptr) || cache == nullptr ||
       (taps > 1 && state == nullptr))
@@ -201,18 +228,19 @@ extern "C" int nib_conv_pool_append(int dtype, const float* proj, int ld, int ta
     prm->ldq = ldq; prm->block_table = block_table; prm->pool_table = pool_table; prm->max_blocks = max_blocks;
     prm->page_size = page_size; prm->n_pages = n_pages; prm->pool = pool; prm->shift_state = shift_state;
     prm->status = status;
+    prm->head_blocks = (n_head + n_kv_head + CP_WARPS - 1) / CP_WARPS;
   };
   if (dtype == DT_F32) {
     ConvPoolParams<float> prm;
     fill(&prm);
     prm.q_out = (float*)q_out; prm.cache = (float*)cache;
-    return launch_conv_pool_append(prm, T, stream);
+    return pick_conv_pool_append(prm, T, stream);
   }
   if (dtype == DT_BF16) {
     ConvPoolParams<bf16> prm;
     fill(&prm);
     prm.q_out = (bf16*)q_out; prm.cache = (bf16*)cache;
-    return launch_conv_pool_append(prm, T, stream);
+    return pick_conv_pool_append(prm, T, stream);
   }
   return NIB_ERR_BAD_ARGUMENT;
 }

@@ -45,6 +45,9 @@ struct TcParams {
   int bq;            // rows of the Q tile = MMA N (multiple of 16, at most 256)
   int stages;
   int k_sub;         // 64-wide K blocks per pipeline stage (1 or 2)
+  // Optional (plain orientation only): the weights lie as segments of K one after another, seg_rows rows of seg_k values each
+  // (a multiple of 64; 0: one matrix), so that one product sums over matrices that are stacked, not side by side
+  int seg_k, seg_rows;
   int kb_per_split;  // 64-wide K blocks per split of K (grid.z splits; their tiles are summed by reduce-add)
   int swap;          // 0: P = activations (out[p, q]); 1: P = weights (out[q, p])
   void* out;
@@ -161,6 +164,12 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constan
     // barriers and buffers, so the lanes run in lockstep).
     const int L = stages < 4 ? stages : 4;
     const bool weights_are_p = prm.swap != 0;
+    // a tile of the N side; with segments, block kx of K is block kx % seg_k of segment kx / seg_k (past the end of K stays
+    // past the end: zeros)
+    auto load_q = [&](uint8_t* dst, uint64_t* bar, int kx) {
+      if (prm.seg_k > 0 && kx < prm.K) tma_load_2d(dst, &map_q, bar, kx % prm.seg_k, q0 + kx / prm.seg_k * prm.seg_rows);
+      else tma_load_2d(dst, &map_q, bar, kx, q0);
+    };
     // first round (the stages are all free): the weight tiles now, the activation tiles after the wait
     const int first_round = num_kb < stages ? num_kb : stages;
     if (lane < L) {
@@ -171,7 +180,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constan
           const int kb64 = kb_begin + kb * k_sub + sub;
           const int kx = (kb64 < kb_end ? kb64 : (prm.K + TC_BK - 1) / TC_BK) * TC_BK;
           if (weights_are_p) tma_load_2d(sp + sub * p_bytes, &map_p, &full_bar[kb], kx, p0);
-          else tma_load_2d(sp + k_sub * p_bytes + sub * q_bytes, &map_q, &full_bar[kb], kx, q0);
+          else load_q(sp + k_sub * p_bytes + sub * q_bytes, &full_bar[kb], kx);
         }
       }
     }
@@ -199,7 +208,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constan
           const int kb64 = kb_begin + kb * k_sub + sub;
           const int kx = (kb64 < kb_end ? kb64 : (prm.K + TC_BK - 1) / TC_BK) * TC_BK;
           tma_load_2d(sp + sub * p_bytes, &map_p, &full_bar[s], kx, p0);
-          if (!ln) tma_load_2d(sp + k_sub * p_bytes + sub * q_bytes, &map_q, &full_bar[s], kx, q0);
+          if (!ln) load_q(sp + k_sub * p_bytes + sub * q_bytes, &full_bar[s], kx);
         }
       }
     }
@@ -545,15 +554,19 @@ constexpr int TC_LN_MAX_Q_BYTES = 96 * 1024;  // resident normalised activations
 
 static int launch_tc(int out_dtype, const void* a, int lda, const void* w, int ldw, const float* bias, void* out,
                      int ldo, int M, int N, int K, int act, int residual, const LnSource* ln, const KvTarget* kv,
-                     const FixScratch* fix, int* status, cudaStream_t stream) {
+                     const FixScratch* fix, int* status, cudaStream_t stream, int seg_k = 0) {
   if (M <= 0 || N <= 0) return 0;
   if (ln != nullptr) a = nullptr;
   if (ln == nullptr && a == nullptr) return NIB_ERR_BAD_ARGUMENT;
   if (!nib_linear_tc_supported(a, lda, w, ldw, K)) return NIB_ERR_UNSUPPORTED_SIZE;
+  if (seg_k != 0 && (seg_k < 0 || seg_k % TC_BK || K % seg_k || ldw != seg_k || ln != nullptr || kv != nullptr || fix != nullptr))
+    return NIB_ERR_UNSUPPORTED_SIZE;
   if (residual && out_dtype != DT_F32) return NIB_ERR_BAD_ARGUMENT;
   if (ln != nullptr && M > 128) return NIB_ERR_UNSUPPORTED_SIZE;
   TcParams prm;
   prm.K = K;
+  prm.seg_k = seg_k;
+  prm.seg_rows = N;
   prm.out = out;
   prm.ldo = ldo;
   prm.out_f32 = out_dtype == DT_F32;
@@ -584,7 +597,7 @@ static int launch_tc(int out_dtype, const void* a, int lda, const void* w, int l
   // 128-feature tiles alone fill the device (the head); else activations on the M side even for 17 to 128
   // rows (one row tile, padded): the swapped product has N / 128 blocks, 38 for GPT-2 XL's q/k/v, the other
   // N / 64 and a split of K for the residual, and a step of an 80-token prompt takes 4.3 ms instead of 5.3.
-  prm.swap = M <= 128 && (M <= 16 || kv != nullptr || ln != nullptr || fix != nullptr || (N + TC_BP - 1) / TC_BP >= 148);
+  prm.swap = seg_k == 0 && M <= 128 && (M <= 16 || kv != nullptr || ln != nullptr || fix != nullptr || (N + TC_BP - 1) / TC_BP >= 148);
   const int esz = prm.out_f32 ? 4 : 2;
   // TMA can store the tile if the output's rows are 16-byte multiples (it also clips a store at the
   // tensor's edge in 16-byte pieces, so the row length must be a multiple too)
@@ -690,7 +703,8 @@ static int launch_tc(int out_dtype, const void* a, int lda, const void* w, int l
   CUtensorMap map_p, map_q, map_o;
   if (!make_map(&map_p, p_base, false, prm.p_rows, K, p_ld, TC_BP, TC_BK, true)) return NIB_ERR_DRIVER;
   if (ln == nullptr) {
-    if (!make_map(&map_q, q_base, false, prm.q_rows, K, q_ld, prm.bq, TC_BK, true)) return NIB_ERR_DRIVER;
+    const int map_rows = seg_k > 0 ? N * (K / seg_k) : prm.q_rows, map_k = seg_k > 0 ? seg_k : K;
+    if (!make_map(&map_q, q_base, false, map_rows, map_k, q_ld, prm.bq, TC_BK, true)) return NIB_ERR_DRIVER;
   } else {
     map_q = map_p;  // unused
   }
@@ -738,6 +752,16 @@ extern "C" int nib_linear_tc(int out_dtype, const void* a, int lda, const void* 
                              cudaStream_t stream) {
   return launch_tc(out_dtype, a, lda, w, ldw, bias, out, ldo, M, N, K, act, residual, nullptr, nullptr, nullptr,
                    status, stream);
+}
+
+// The same with the weights as segments of K: w [K / seg_k, N, seg_k] contiguous (matrices that are stacked), a [M, K]:
+// out = sum over the segments s of a[:, s seg_k .. + seg_k] . w[s]^T.  seg_k a multiple of 64.
+extern "C" int nib_linear_tc_segments(int out_dtype, const void* a, int lda, const void* w, int seg_k, const float* bias,
+                                      void* out, int ldo, int M, int N, int K, int act, int residual, int* status,
+                                      cudaStream_t stream) {
+  if (seg_k <= 0) return NIB_ERR_BAD_ARGUMENT;
+  return launch_tc(out_dtype, a, lda, w, seg_k, bias, out, ldo, M, N, K, act, residual, nullptr, nullptr, nullptr, status,
+                   stream, seg_k);
 }
 
 // The general form for steps of at most 128 rows.  Any of three options may be on:

@@ -7,9 +7,9 @@
 //                      ahead of the vector (the embedding's output, given to every later pass again).  Without `out` only the sum is made.
 //   embed_group_norm : x[t] = norm(table[token_t] * scale): the embedding and the norm that follows it in one pass.
 //
-// A warp owns a (row, part): parts do not see one another, so there is no shared memory and no block barrier.  Parts
-// whose size is a multiple of 4 (up to 2048) live in registers as 16-byte pieces; others are read twice.  A part's sum
-// runs in the same order whatever the number of rows.
+// A warp owns a (row, part): parts do not see one another, so there is no shared memory and no block barrier (one group and
+// at most 64 rows: a block a row).  Parts
+// whose size is a multiple of 4 (up to 2048) live in registers as 16-byte pieces; others are read twice.
 #include "api.h"
 #include "common.cuh"
 
@@ -111,6 +111,58 @@ group_norm_vec_kernel(Src src, const float* __restrict__ w, OutT* out, int n_row
   }
 }
 
+// The same with one group and a block a row, a 16-byte piece a thread: steps of few rows, where a warp's row is a chain of
+// loads and stores that nothing else fills.
+template <typename Src, typename OutT, int NV>
+__global__ void __launch_bounds__(256)
+group_norm_row_kernel(Src src, const float* __restrict__ w, OutT* out, int n_rows, int C, float eps) {
+  pdl_trigger();
+  __shared__ float sums[32];
+  const int r = blockIdx.x, n4 = C >> 2;
+  float4 ww[NV];
+  if (out != nullptr) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int k = threadIdx.x + blockDim.x * i;
+      if (k < n4) ww[i] = gn_load4(w + 4 * k);
+    }
+  }
+  pdl_wait();
+  auto* p = src.row(r, C);
+  float4 v[NV];
+  float q = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int k = threadIdx.x + blockDim.x * i;
+    if (k < n4) {
+      v[i] = gn_load4(p + 4 * k);
+      if constexpr (Src::WRITES_BACK) {
+        if (src.add_rows != nullptr) {
+          const float4 b = gn_load4(src.add_rows + (size_t)r * C + 4 * k);
+          v[i] = make_float4(v[i].x + b.x, v[i].y + b.y, v[i].z + b.z, v[i].w + b.w);
+        }
+        if (src.add != nullptr) {
+          const float4 a = gn_load4(src.add + 4 * k);
+          v[i] = make_float4(v[i].x + a.x, v[i].y + a.y, v[i].z + a.z, v[i].w + a.w);
+        }
+        if (src.adds()) gn_store4(p + 4 * k, v[i].x, v[i].y, v[i].z, v[i].w);
+      } else {
+        v[i] = make_float4(v[i].x * src.scale, v[i].y * src.scale, v[i].z * src.scale, v[i].w * src.scale);
+      }
+      q += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+  }
+  if (out == nullptr) return;
+  const float rstd = 1.0f / sqrtf(block_sum(q, sums) / (float)C + eps);
+  OutT* o = out + (size_t)r * C;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int k = threadIdx.x + blockDim.x * i;
+    if (k < n4)
+      gn_store4(o + 4 * k, v[i].x * rstd * ww[i].x, v[i].y * rstd * ww[i].y, v[i].z * rstd * ww[i].z, v[i].w * rstd * ww[i].w);
+  }
+}
+
 template <typename Src, typename OutT>
 __global__ void __launch_bounds__(256)
 group_norm_any_kernel(Src src, const float* __restrict__ w, OutT* out, int n_rows, int C, int groups, float eps) {
@@ -151,6 +203,12 @@ static int launch_group_norm(Src src, bool aligned, const float* w, OutT* out, i
   const long long units = (long long)n_rows * groups;
   const dim3 grid((unsigned)((units + 7) / 8));
   const bool vec = aligned && (gs & 3) == 0 && gs <= 2048 && (((uintptr_t)w | (uintptr_t)out) & 15) == 0;
+  if (vec && groups == 1 && C >= 256 && n_rows <= 64) {
+    const int n4 = C >> 2, threads = n4 >= 256 ? 256 : (n4 + 31) / 32 * 32;
+    if (n4 <= 256) launch_pdl(group_norm_row_kernel<Src, OutT, 1>, dim3(n_rows), dim3(threads), 0, stream, src, w, out, n_rows, C, eps);
+    else launch_pdl(group_norm_row_kernel<Src, OutT, 2>, dim3(n_rows), dim3(threads), 0, stream, src, w, out, n_rows, C, eps);
+    NIB_LAUNCH_CHECK();
+  }
 #define NIB_GN(NV) launch_pdl(group_norm_vec_kernel<Src, OutT, NV>, grid, dim3(256), 0, stream, src, w, out, n_rows, C, groups, eps)
   if (vec && gs <= 256) NIB_GN(2);
   else if (vec && gs <= 512) NIB_GN(4);

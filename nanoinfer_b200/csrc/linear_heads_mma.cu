@@ -90,6 +90,29 @@ linear_heads_mma_kernel(const bf16* a, int lda, int a_hs, const bf16* __restrict
   load_a(0, 0);
   cp_async_commit();
   const int n_k = (K + LH_KC - 1) / LH_KC;
+  float gates[NT][4];                                       // (asked for here, they travel while the products are made)
+  if (gate != nullptr) {
+    const int ga = m0 + (BM == 64 ? warp * 16 : 0) + (lane >> 2), gc = n0 + (BM == 64 ? 0 : warp * 16) + (lane & 3) * 2;
+    const bool pairs = ((uintptr_t)gate & 7) == 0 && (ldg & 1) == 0 && (N & 1) == 0;
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+      for (int c = 0; c < 4; c += 2) {
+        const int m = ga + (c < 2 ? 0 : 8), col = gc + i * 8;
+        const float* g = gate + (size_t)m * ldg + (size_t)h * N + col;
+        gates[i][c] = gates[i][c + 1] = 0.0f;
+        if (m < M && col < N) {
+          if (pairs) {
+            const float2 v = *reinterpret_cast<const float2*>(g);
+            gates[i][c] = v.x;
+            gates[i][c + 1] = v.y;
+          } else {
+            gates[i][c] = g[0];
+            if (col + 1 < N) gates[i][c + 1] = g[1];
+          }
+        }
+      }
+  }
   const int arow = BM == 64 ? warp * 16 : 0, bcol = BM == 64 ? 0 : warp * 16;
   for (int kc = 0; kc < n_k; ++kc) {
     const int buf = kc & 1;
@@ -122,7 +145,7 @@ linear_heads_mma_kernel(const bf16* a, int lda, int a_hs, const bf16* __restrict
     for (int c = 0; c < 4; ++c) {
       const int m = c < 2 ? ra : rb, col = n + (c & 1);
       if (m >= M || col >= N) continue;
-      const float y = gate ? acc[i][c] / (1.0f + __expf(-gate[(size_t)m * ldg + (size_t)h * N + col])) : acc[i][c];
+      const float y = gate ? acc[i][c] / (1.0f + __expf(-gates[i][c])) : acc[i][c];
       out[(size_t)m * ldo + (size_t)h * o_hs + col] = from_float<OutT>(y);
     }
   }

@@ -37,15 +37,16 @@
 
 namespace nib {
 
-constexpr int MOE_WARPS = 4;
+constexpr int MOE_WARPS = 4, MOE_R_WARPS = 8;   // (of the routing kernel: an expert's logit a warp)
 
 template <typename T>
-__global__ void __launch_bounds__(MOE_WARPS * 32)
+__global__ void __launch_bounds__(MOE_R_WARPS * 32)
 moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_expert, int top, int renorm, int score,
                  const float* __restrict__ logit_bias, const float* __restrict__ choice_bias, int n_real, float* x, int* ids, float* weights) {
   pdl_trigger();
-  extern __shared__ float smem[];
+  extern __shared__ __align__(16) float smem[];
   float* row = smem;               // [C]
+  const bool wide = (C * sizeof(T)) % 16 == 0 && ((uintptr_t)wr & 15) == 0;
   float* prob = smem + C;          // [n_expert]
   __shared__ float scratch[32];
   __shared__ float pass_on;        // the summed scores of the chosen experts that hand their input on
@@ -54,10 +55,27 @@ moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_exp
   pdl_wait();
   for (int c = threadIdx.x; c < C; c += blockDim.x) row[c] = to_float(h[(size_t)t * ldh + c]);
   __syncthreads();
-  for (int e = warp; e < n_expert; e += MOE_WARPS) {
+  for (int e = warp; e < n_expert; e += MOE_R_WARPS) {
     const T* w = wr + (size_t)e * C;
     float s = 0.0f;
-    for (int c = lane; c < C; c += 32) s += row[c] * to_float(w[c]);
+    if (wide) {                                    // 16 bytes a lane and load
+      constexpr int VN = 16 / sizeof(T);
+#pragma unroll 4
+      for (int c = lane * VN; c < C; c += 32 * VN) {
+        const uint4 u = *reinterpret_cast<const uint4*>(w + c);
+        const T* v = reinterpret_cast<const T*>(&u);
+#pragma unroll
+        for (int i = 0; i < VN; i += 4) {
+          const float4 r = *reinterpret_cast<const float4*>(row + c + i);
+          s = fmaf(r.x, to_float(v[i]), s);
+          s = fmaf(r.y, to_float(v[i + 1]), s);
+          s = fmaf(r.z, to_float(v[i + 2]), s);
+          s = fmaf(r.w, to_float(v[i + 3]), s);
+        }
+      }
+    } else {
+      for (int c = lane; c < C; c += 32) s += row[c] * to_float(w[c]);
+    }
     s = warp_sum(s);
     if (lane == 0) prob[e] = logit_bias ? s + logit_bias[e] : s;
   }
@@ -312,6 +330,48 @@ moe_gate_scale_kernel(const TI* pre, T* inner, const int* ids, const float* weig
   inner[i] = from_float<T>(v);
 }
 
+// Four outputs a thread (F a multiple of 4): what a row did not choose is written as zeros and not read.
+template <typename TI, typename T>
+__global__ void __launch_bounds__(256)
+moe_gate_scale4_kernel(const TI* pre, T* inner, const int* ids, const float* weights, int n_expert, int F, int top,
+                       int act, float act_prm, int on_input) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.y, per = F >> 2;
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n_expert * per) return;
+  const int e = i / per;
+  float s = 0.0f;
+  bool chosen = false;
+  for (int k = 0; k < top; ++k)
+    if (ids[(size_t)t * top + k] == e) { s = weights[(size_t)t * top + k]; chosen = true; }
+  float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+  const size_t at = ((size_t)t * n_expert * per + i) * 4;
+  if (chosen) {
+    float p[8];
+    if constexpr (sizeof(TI) == 4) {
+      const float4 a = reinterpret_cast<const float4*>(pre + 2 * at)[0], b = reinterpret_cast<const float4*>(pre + 2 * at)[1];
+      p[0] = a.x; p[1] = a.y; p[2] = a.z; p[3] = a.w; p[4] = b.x; p[5] = b.y; p[6] = b.z; p[7] = b.w;
+    } else {
+      const uint4 u = *reinterpret_cast<const uint4*>(pre + 2 * at);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) p[j] = to_float(reinterpret_cast<const TI*>(&u)[j]);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      v[j] = on_input ? gated_act(s * p[2 * j], s * p[2 * j + 1], act, act_prm) : s * gated_act(p[2 * j], p[2 * j + 1], act, act_prm);
+  }
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(inner + at) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<uint32_t*>(&lo);
+    u.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(inner + at) = u;
+  }
+}
+
 __global__ void __launch_bounds__(256) moe_combine_kernel(const float* parts, const int* ids, float* x, int C, int top,
                                                           size_t n) {
   pdl_trigger();
@@ -400,11 +460,11 @@ extern "C" int nib_moe_route(int dtype, const void* h, int ldh, const void* w_ro
   if (smem > 200 * 1024) return NIB_ERR_UNSUPPORTED_SIZE;
   if (dtype == DT_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_pdl(moe_route_kernel<float>, dim3(T), dim3(MOE_WARPS * 32), smem, stream, (const float*)h, ldh,
+    launch_pdl(moe_route_kernel<float>, dim3(T), dim3(MOE_R_WARPS * 32), smem, stream, (const float*)h, ldh,
                (const float*)w_router, C, n_expert, top, renorm, score, logit_bias, choice_bias, n_real, x, ids, weights);
   } else if (dtype == DT_BF16) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_pdl(moe_route_kernel<bf16>, dim3(T), dim3(MOE_WARPS * 32), smem, stream, (const bf16*)h, ldh,
+    launch_pdl(moe_route_kernel<bf16>, dim3(T), dim3(MOE_R_WARPS * 32), smem, stream, (const bf16*)h, ldh,
                (const bf16*)w_router, C, n_expert, top, renorm, score, logit_bias, choice_bias, n_real, x, ids, weights);
   } else {
     return NIB_ERR_BAD_ARGUMENT;
@@ -463,6 +523,21 @@ extern "C" int nib_moe_gate_scale(int pre_dtype, int dtype, const void* pre, voi
                                   int on_input, cudaStream_t stream) {
   if (T <= 0) return 0;
   const size_t n = (size_t)T * n_expert * F;
+  if ((F & 3) == 0 && T <= 65535 && (((uintptr_t)pre | (uintptr_t)inner) & 15) == 0) {
+    const dim3 grid4((unsigned)((n_expert * (F >> 2) + 255) / 256), T);
+    if (pre_dtype == DT_F32 && dtype == DT_F32)
+      launch_pdl(moe_gate_scale4_kernel<float, float>, grid4, dim3(256), 0, stream, (const float*)pre, (float*)inner, ids,
+                 weights, n_expert, F, top, act, act_prm, on_input);
+    else if (pre_dtype == DT_F32 && dtype == DT_BF16)
+      launch_pdl(moe_gate_scale4_kernel<float, bf16>, grid4, dim3(256), 0, stream, (const float*)pre, (bf16*)inner, ids,
+                 weights, n_expert, F, top, act, act_prm, on_input);
+    else if (pre_dtype == DT_BF16 && dtype == DT_BF16)
+      launch_pdl(moe_gate_scale4_kernel<bf16, bf16>, grid4, dim3(256), 0, stream, (const bf16*)pre, (bf16*)inner, ids,
+                 weights, n_expert, F, top, act, act_prm, on_input);
+    else
+      return NIB_ERR_BAD_ARGUMENT;
+    NIB_LAUNCH_CHECK();
+  }
   const dim3 grid((unsigned)((n + 255) / 256));
   if (pre_dtype == DT_F32 && dtype == DT_F32)
     launch_pdl(moe_gate_scale_kernel<float, float>, grid, dim3(256), 0, stream, (const float*)pre, (float*)inner, ids,

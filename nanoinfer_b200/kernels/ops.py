@@ -43,6 +43,8 @@ _SIGNATURES = {
     "nib_linear_tc_supported": [_c_ptr, _c_int, _c_ptr, _c_int, _c_int],
     "nib_linear_tc": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                       _c_int, _c_int, _c_ptr, _c_ptr],
+    "nib_linear_tc_segments": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
+                               _c_int, _c_int, _c_ptr, _c_ptr],
     "nib_linear_tc_small": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                             _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_ptr,
                             _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr,
@@ -392,6 +394,21 @@ def linear_tc(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], ou
     _check(library().nib_linear_tc(_dt(out), _ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(bias), _ptr(out),
                                    out.stride(0), M, N, K, act, int(residual), _ptr(status_word()), _stream()),
            "linear_tc")
+
+
+def linear_segments(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, residual: bool = False) -> bool:
+    """out[:M] (+)= sum_s a[:M, s F : (s + 1) F] . w[s]^T for stacked bfloat16 matrices w [segments, N, F], as ONE product on
+    the tensor cores whose K walks the segments.  False if a size or an alignment is not taken."""
+    S, N, F = w.shape
+    if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or F % 64 or not w.is_contiguous() or a.shape[1] != S * F \
+            or a.stride(1) != 1 or a.stride(0) % 8 or a.data_ptr() % 16 or w.data_ptr() % 16 or out.stride(1) != 1 \
+            or out.shape[1] != N or (residual and out.dtype != torch.float32):
+        return False
+    if tracing():
+        _note("matmul", "matmul", (M, S * F, N), 2.0 * M * S * F * N, w.numel() * 2 + M * S * F * 2 + M * N * out.element_size() * (2 if residual else 1))
+    _check(library().nib_linear_tc_segments(_dt(out), _ptr(a), a.stride(0), _ptr(w), F, None, _ptr(out), out.stride(0), M, N,
+                                            S * F, ACT_NONE, int(residual), _ptr(status_word()), _stream()), "linear_tc_segments")
+    return True
 
 
 _capability: dict = {}
@@ -1357,7 +1374,7 @@ def linear_heads(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torc
         raise KernelError("linear_heads: a and w share a dtype, w contiguous [heads, N, K]")
     if tracing():
         _note("matmul", "matmul_heads", (M, K, H * N), 2.0 * M * H * N * K,
-              w.numel() * w.element_size() + M * H * (K * a.element_size() + N * out.element_size()))
+              w.numel() * w.element_size() + M * H * (K * a.element_size() + N * out.element_size() + (4 * N if gate is not None else 0)))
     if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1 or gate.shape[1] < H * N):
         raise KernelError("linear_heads: the gate must be float32 [rows, >= heads * N] with contiguous rows")
     gate_args = (_ptr(gate), gate.stride(0) if gate is not None else 0)
@@ -1511,7 +1528,8 @@ def moe_experts(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: 
     """x[t] += sum_k weights[t, k] * W_down[ids[t, k]] . act(W_up[ids[t, k]] . h[t]) with w_up [experts, F, C] and
     w_down [experts, C, F].  Steps of few rows: row by row.  Steps of many rows: all experts through the engine's
     own products with the unchosen ones scaled to zero in between (``moe_dense_pays``: the first matrices as one
-    product, the second ones a product an expert, all adding into the stream), else expert by expert (weights
+    product, the second ones one product that walks the experts, or a product an expert where their width is no multiple of 64,
+    adding into the stream), else expert by expert (weights
     staged in shared memory, a fixed order of additions)."""
     E, F, C = w_up.shape
     if gated:
@@ -1536,6 +1554,8 @@ def moe_experts(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: 
             linear(h, w_up.view(E * F, C), None, inner_all, T, act=act)
             moe_scale(inner_all, ids, weights, T, E, F, top)
         trace_scope(_rec.layer if _rec is not None else -1, "experts_down")
+        if linear_segments(inner_all, w_down, x, T, residual=True):
+            return
         for e in range(E):
             linear(inner_all[:, e * F:(e + 1) * F], w_down[e], None, x, T, residual=True)
         return

@@ -283,13 +283,13 @@ def test_product_per_head_with_a_gate_per_element(H, N, K, M, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("E,top", [(5, 2), (16, 4), (40, 1), (3, 3)])
-def test_routing_by_biased_logits(E, top, dtype):
+@pytest.mark.parametrize("E,top,C", [(5, 2, 72), (16, 4, 1000), (40, 1, 45), (3, 3, 768), (7, 2, 2056)])
+def test_routing_by_biased_logits(E, top, C, dtype):
     from nanoinfer_b200.kernels import ops
 
     torch.manual_seed(E)
-    dt, T, C = DT[dtype], 30, 72
-    h, w, b = torch.randn(T, C, device=DEV).to(dt), (torch.randn(E, C, device=DEV) / 8).to(dt), torch.randn(E, device=DEV)
+    dt, T = DT[dtype], 30
+    h, w, b = torch.randn(T, C, device=DEV).to(dt), (torch.randn(E, C, device=DEV) / C ** 0.5).to(dt), torch.randn(E, device=DEV)
     ids, weights = torch.zeros(T, top, dtype=torch.int32, device=DEV), torch.zeros(T, top, device=DEV)
     ops.moe_route(h, w, T, top, True, ids, weights, logit_bias=b)
     z = h.double() @ w.double().T + b.double()
@@ -298,8 +298,53 @@ def test_routing_by_biased_logits(E, top, dtype):
     assert float((weights.double() - torch.softmax(best.values, 1)).abs().max()) < 1e-5
 
 
+@pytest.mark.parametrize("M", [17, 128, 130, 700])
+@pytest.mark.parametrize("S,N,F", [(3, 64, 64), (8, 768, 128), (5, 72, 192), (16, 200, 64), (2, 1600, 1600), (1, 48, 320)])
+def test_one_product_over_stacked_matrices(S, N, F, M):
+    """The K of one product walks matrices that lie one after another (tcgen05, TMA coordinates by segment), stored and added."""
+    from nanoinfer_b200.kernels import ops
+
+    torch.manual_seed(M + N)
+    a = torch.randn(M + 3, S * F, device=DEV).to(torch.bfloat16)
+    w = (torch.randn(S, N, F, device=DEV) / (S * F) ** 0.5).to(torch.bfloat16)
+    want = sum(a[:M, s * F:(s + 1) * F].double() @ w[s].double().T for s in range(S))
+    x0 = torch.randn(M + 3, N, device=DEV)
+    for residual in (True, False):
+        x = x0.clone()
+        assert ops.linear_segments(a, w, x, M, residual=residual)
+        assert int(ops.status_word()) == 0
+        ref = want + (x0[:M].double() if residual else 0.0)
+        assert float((x[:M].double() - ref).abs().max()) < 1e-3 and torch.equal(x[M:], x0[M:])
+
+
+@pytest.mark.parametrize("F", [64, 24, 30])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("C,groups", [(40, 1), (264, 2), (30, 3), (1536, 1)])
+def test_gated_experts_all_at_once(F, dtype):
+    """A step of many rows: all experts through the engine's products, what a row did not choose zeroed and not read (what
+    lies there is not a number), by the four-a-thread kernel and the plain one."""
+    from nanoinfer_b200.kernels import ops
+
+    torch.manual_seed(F)
+    dt, T, E, top = DT[dtype], 21, 6, 2
+    pre = torch.randn(T, E * 2 * F, device=DEV)
+    ids = torch.stack([torch.randperm(E, device=DEV)[:top] for _ in range(T)]).to(torch.int32)
+    weights = torch.rand(T, top, device=DEV)
+    want = torch.zeros(T, E, F, dtype=torch.float64, device=DEV)
+    p = pre.double().view(T, E, F, 2)
+    chosen = torch.zeros(T, E, dtype=torch.bool, device=DEV)
+    for k in range(top):
+        r = torch.arange(T, device=DEV)
+        g, u = p[r, ids[:, k].long(), :, 0], p[r, ids[:, k].long(), :, 1]
+        want[r, ids[:, k].long()] = weights[:, k:k + 1].double() * g * torch.sigmoid(g) * u
+        chosen[r, ids[:, k].long()] = True
+    pre.view(T, E, 2 * F)[~chosen] = float("nan")
+    out = torch.full((T, E * F), 7.0, device=DEV, dtype=dt)
+    ops.moe_gate_scale(pre, out, ids, weights, T, E, F, top, ops.ACT_SILU, False)
+    assert float((out.double() - want.view(T, -1)).abs().max()) < (1e-5 if dtype == "float32" else 3e-2)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("C,groups", [(40, 1), (264, 2), (30, 3), (1536, 1), (768, 1), (2048, 1)])
 def test_norm_with_rows_and_a_vector_added_first(C, groups, dtype):
     from nanoinfer_b200.kernels import ops
 

@@ -367,8 +367,8 @@ int nib_group_norm(int out_dtype, float* x, const int* rows, const float* add, c
 // ---- short convolution, norm per head, cache write and pooled rows of an attention whose values are its keys
 // (conv_pool_append.cu)
 int nib_conv_pool_append(int dtype, const float* proj, int ld, int taps, const float* w, float* state,
-                         long long state_stride, const int* entry_start, const int* entry_slot, const int* positions,
-                         const int* row_entry, int n_head, int n_kv_head, int dim, int hd, int norm, float eps, void* q_out,
+                         long long state_stride, const int* entry_start, const int* entry_pos0, const int* entry_slot,
+                         int n_entries, const int* positions, const int* row_entry, int n_head, int n_kv_head, int dim, int hd, int norm, float eps, void* q_out,
                          int ldq, void* cache, const int* block_table, const int* pool_table, int max_blocks,
                          int page_size, int n_pages, int pool, int shift_state, int T, int* status, cudaStream_t stream);
 // The state of a short convolution behind a step (the second half of nib_short_conv on its own).

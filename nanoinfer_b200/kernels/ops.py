@@ -167,7 +167,8 @@ _SIGNATURES = {
                                   _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "nib_diff_combine": [_c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr, _c_int,
                          _c_int, _c_ptr],
-    "nib_conv_pool_append": [_c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+    "nib_conv_pool_append": [_c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr, _c_ptr, _c_int,
+                             _c_ptr, _c_ptr,
                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int,
                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "nib_short_conv_state": [_c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, ctypes.c_longlong, _c_ptr, _c_ptr, _c_int, _c_ptr],
@@ -2144,8 +2145,8 @@ def conv_pool_append(proj: torch.Tensor, taps: int, w: torch.Tensor, state: Opti
               T * (4.0 * channels + n_out * q_out.element_size()))
     st = (_ptr(state), state.stride(0) if state is not None else 0)
     _check(library().nib_conv_pool_append(
-        _dt(q_out), _ptr(proj), proj.stride(0), int(taps), _ptr(w), *st, _ptr(ctx.entry_start), _ptr(ctx.entry_slot),
-        _ptr(ctx.positions), _ptr(ctx.row_entry), n_head, n_kv_head, int(dim), hd, int(bool(norm)), float(eps), _ptr(q_out),
+        _dt(q_out), _ptr(proj), proj.stride(0), int(taps), _ptr(w), *st, _ptr(ctx.entry_start),
+        _ptr(ctx.entry_pos0), _ptr(ctx.entry_slot), ctx.n_entries, _ptr(ctx.positions), _ptr(ctx.row_entry), n_head, n_kv_head, int(dim), hd, int(bool(norm)), float(eps), _ptr(q_out),
         q_out.stride(0), _ptr(cache), _ptr(block_table), _ptr(pool_table), block_table.shape[1], page_size, n_pages, int(pool),
         int(alone), T, _ptr(ctx.status), _stream()), "conv_pool_append")
     if taps > 1 and not alone:

@@ -38,7 +38,7 @@ struct SkinnyParams {
   const float* ln_x;    // residual stream, normalised here
   int ln_ldx;
   const float* ln_gamma;
-  const float* ln_beta;
+  const float* ln_beta;   // null: an RMS norm (nothing is taken off, nothing added)
   const int* ln_rows;
   float ln_eps;
   const bf16* w;        // [N, K]
@@ -134,7 +134,8 @@ linear_skinny_kernel(const SkinnyParams prm) {
   if (prm.ln_x != nullptr) {
     for (int i = threadIdx.x; i < prm.K / 4; i += blockDim.x) {
       reinterpret_cast<float4*>(ln_gb)[i] = reinterpret_cast<const float4*>(prm.ln_gamma)[i];
-      reinterpret_cast<float4*>(ln_gb + prm.K)[i] = reinterpret_cast<const float4*>(prm.ln_beta)[i];
+      reinterpret_cast<float4*>(ln_gb + prm.K)[i] =
+          prm.ln_beta != nullptr ? reinterpret_cast<const float4*>(prm.ln_beta)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   }
   // What the epilogue needs and the kernel ahead does not write: the first tile's bias, and for the
@@ -200,7 +201,7 @@ linear_skinny_kernel(const SkinnyParams prm) {
         *reinterpret_cast<float4*>(mine + k) = t;
         sum += (t.x + t.y) + (t.z + t.w);
       }
-      const float mean = warp_sum(sum) / (float)K;
+      const float mean = prm.ln_beta != nullptr ? warp_sum(sum) / (float)K : 0.0f;   // (no shift: an RMS norm)
       float sq = 0.0f;
       for (int k = lane * 4; k < K; k += 128) {   // (a lane reads back what it wrote)
         const float4 t = *reinterpret_cast<const float4*>(mine + k);
@@ -234,7 +235,7 @@ linear_skinny_kernel(const SkinnyParams prm) {
         v[4 * j] = t.x; v[4 * j + 1] = t.y; v[4 * j + 2] = t.z; v[4 * j + 3] = t.w;
         sum += (t.x + t.y) + (t.z + t.w);
       }
-      const float mean = warp_sum(sum) / (float)K;
+      const float mean = prm.ln_beta != nullptr ? warp_sum(sum) / (float)K : 0.0f;   // (no shift: an RMS norm)
       float sq = 0.0f;
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
@@ -558,7 +559,7 @@ extern "C" int nib_linear_skinny_supported(int M, int K, int ldw, int ln, const 
 
 // The product for steps of at most 128 rows (bfloat16 weights and activations; out bfloat16 or
 // float32).  Options as for nib_linear_tc_small: ln_x != null folds the LayerNorm before the product
-// in (`a` ignored); cache != null sends the features from q_dim on to the paged
+// in (`a` ignored; ln_beta null: an RMS norm); cache != null sends the features from q_dim on to the paged
 // cache.  split: blocks of a cluster that split K (0: chosen here; 1, 2, 4 or 8).
 extern "C" int nib_linear_skinny(int out_dtype, const void* a, int lda, const void* w, int ldw, const float* bias,
                                  void* out, int ldo, int M, int N, int K, int act, int residual, const float* ln_x,

@@ -562,7 +562,7 @@ static int launch_tc(int out_dtype, const void* a, int lda, const void* w, int l
   if (seg_k != 0 && (seg_k < 0 || seg_k % TC_BK || K % seg_k || ldw != seg_k || ln != nullptr || kv != nullptr || fix != nullptr))
     return NIB_ERR_UNSUPPORTED_SIZE;
   if (residual && out_dtype != DT_F32) return NIB_ERR_BAD_ARGUMENT;
-  if (ln != nullptr && M > 128) return NIB_ERR_UNSUPPORTED_SIZE;
+  if (ln != nullptr && (M > 128 || ln->beta == nullptr)) return NIB_ERR_UNSUPPORTED_SIZE;   // (a LayerNorm only)
   TcParams prm;
   prm.K = K;
   prm.seg_k = seg_k;

@@ -39,6 +39,43 @@ namespace nib {
 
 constexpr int MOE_WARPS = 4, MOE_R_WARPS = 8;   // (of the routing kernel: an expert's logit a warp)
 
+// This lane's part of the products of a row in shared memory with NW rows of weights `stride` elements apart: 16 bytes a lane
+// and load where `wide` (K and the weights' address allow it), one element otherwise.
+template <int NW, typename T>
+__device__ __forceinline__ void moe_dot(const float* row, const T* w, size_t stride, int K, int lane, bool wide, float* s) {
+#pragma unroll
+  for (int n = 0; n < NW; ++n) s[n] = 0.0f;
+  if (wide) {
+    constexpr int VN = 16 / sizeof(T);
+#pragma unroll 4
+    for (int c = lane * VN; c < K; c += 32 * VN) {
+      uint4 u[NW];
+#pragma unroll
+      for (int n = 0; n < NW; ++n) u[n] = *reinterpret_cast<const uint4*>(w + n * stride + c);
+#pragma unroll
+      for (int i = 0; i < VN; i += 4) {
+        const float4 r = *reinterpret_cast<const float4*>(row + c + i);
+#pragma unroll
+        for (int n = 0; n < NW; ++n) {
+          const T* v = reinterpret_cast<const T*>(&u[n]) + i;
+          s[n] = fmaf(r.x, to_float(v[0]), s[n]);
+          s[n] = fmaf(r.y, to_float(v[1]), s[n]);
+          s[n] = fmaf(r.z, to_float(v[2]), s[n]);
+          s[n] = fmaf(r.w, to_float(v[3]), s[n]);
+        }
+      }
+    }
+  } else {
+    for (int c = lane; c < K; c += 32)
+#pragma unroll
+      for (int n = 0; n < NW; ++n) s[n] += row[c] * to_float(w[n * stride + c]);
+  }
+}
+template <typename T>
+__device__ __forceinline__ bool moe_wide(const T* w, int K) {
+  return (K * sizeof(T)) % 16 == 0 && ((uintptr_t)w & 15) == 0;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(MOE_R_WARPS * 32)
 moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_expert, int top, int renorm, int score,
@@ -46,7 +83,7 @@ moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_exp
   pdl_trigger();
   extern __shared__ __align__(16) float smem[];
   float* row = smem;               // [C]
-  const bool wide = (C * sizeof(T)) % 16 == 0 && ((uintptr_t)wr & 15) == 0;
+  const bool wide = moe_wide(wr, C);
   float* prob = smem + C;          // [n_expert]
   __shared__ float scratch[32];
   __shared__ float pass_on;        // the summed scores of the chosen experts that hand their input on
@@ -57,25 +94,8 @@ moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_exp
   __syncthreads();
   for (int e = warp; e < n_expert; e += MOE_R_WARPS) {
     const T* w = wr + (size_t)e * C;
-    float s = 0.0f;
-    if (wide) {                                    // 16 bytes a lane and load
-      constexpr int VN = 16 / sizeof(T);
-#pragma unroll 4
-      for (int c = lane * VN; c < C; c += 32 * VN) {
-        const uint4 u = *reinterpret_cast<const uint4*>(w + c);
-        const T* v = reinterpret_cast<const T*>(&u);
-#pragma unroll
-        for (int i = 0; i < VN; i += 4) {
-          const float4 r = *reinterpret_cast<const float4*>(row + c + i);
-          s = fmaf(r.x, to_float(v[i]), s);
-          s = fmaf(r.y, to_float(v[i + 1]), s);
-          s = fmaf(r.z, to_float(v[i + 2]), s);
-          s = fmaf(r.w, to_float(v[i + 3]), s);
-        }
-      }
-    } else {
-      for (int c = lane; c < C; c += 32) s += row[c] * to_float(w[c]);
-    }
+    float s;
+    moe_dot<1>(row, w, 0, C, lane, wide, &s);
     s = warp_sum(s);
     if (lane == 0) prob[e] = logit_bias ? s + logit_bias[e] : s;
   }
@@ -136,7 +156,7 @@ moe_route_kernel(const T* h, int ldh, const T* __restrict__ wr, int C, int n_exp
   }
 }
 
-constexpr int MOE_PER_WARP = 2;   // outputs a warp makes one after the other (few: a step of few rows is bound by the
+constexpr int MOE_PER_WARP = 2;   // outputs a warp makes, their loads side by side (few: a step of few rows is bound by the
                                   // latency of each weight row's loads, so it wants many warps at once)
 
 template <typename T>
@@ -144,7 +164,8 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_up_kernel(const T* h, int ldh, const T* __restrict__ w_up, const int* ids, T* inner, int C, int F, int top,
               int act, float act_prm, int gated, const float* in_weights) {
   pdl_trigger();
-  extern __shared__ float row[];   // [C]
+  extern __shared__ __align__(16) float row[];   // [C]
+  const bool wide = moe_wide(w_up, C);
   const int p = blockIdx.x, t = p / top, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
   const int e = ids[p];
@@ -154,23 +175,25 @@ moe_up_kernel(const T* h, int ldh, const T* __restrict__ w_up, const int* ids, T
   const int f0 = (blockIdx.y * MOE_WARPS + warp) * MOE_PER_WARP;
   if (gated) {   // rows 2f and 2f + 1 of the expert's matrix are output f's gate and value
     const float ws = in_weights ? in_weights[p] : 1.0f;
-    for (int f = f0; f < min(F, f0 + MOE_PER_WARP); ++f) {
-      const T* w = w_up + ((size_t)e * F + f) * 2 * C;
-      float g = 0.0f, u = 0.0f;
-      for (int c = lane; c < C; c += 32) {
-        g += row[c] * to_float(w[c]);
-        u += row[c] * to_float(w[C + c]);
-      }
-      g = warp_sum(g);
-      u = warp_sum(u);
-      if (lane == 0) inner[(size_t)p * F + f] = from_float<T>(gated_act(ws * g, ws * u, act, act_prm));
+    if (f0 >= F) return;
+    const bool two = f0 + 1 < F;
+    float s[4];
+    if (two) {
+      moe_dot<4>(row, w_up + ((size_t)e * F + f0) * 2 * C, (size_t)C, C, lane, wide, s);
+    } else {
+      moe_dot<2>(row, w_up + ((size_t)e * F + f0) * 2 * C, (size_t)C, C, lane, wide, s);
+      s[2] = s[3] = 0.0f;
     }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) s[n] = warp_sum(s[n]);
+    if (lane == 0) inner[(size_t)p * F + f0] = from_float<T>(gated_act(ws * s[0], ws * s[1], act, act_prm));
+    if (lane == 0 && two) inner[(size_t)p * F + f0 + 1] = from_float<T>(gated_act(ws * s[2], ws * s[3], act, act_prm));
     return;
   }
   for (int f = f0; f < min(F, f0 + MOE_PER_WARP); ++f) {
     const T* w = w_up + ((size_t)e * F + f) * C;
-    float s = 0.0f;
-    for (int c = lane; c < C; c += 32) s += row[c] * to_float(w[c]);
+    float s;
+    moe_dot<1>(row, w, 0, C, lane, wide, &s);
     s = warp_sum(s);
     if (lane == 0) inner[(size_t)p * F + f] = from_float<T>(apply_act(s, act));
   }
@@ -181,26 +204,28 @@ __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_down_kernel(const T* inner, const T* __restrict__ w_down, const int* ids, const float* weights, float* x, int C,
                 int F, int top) {
   pdl_trigger();
-  extern __shared__ float rows[];  // [top][F]
+  extern __shared__ __align__(16) float rows[];  // [top][F]
+  const bool wide = moe_wide(w_down, F);   // (then every choice's row of F values starts on a 16-byte boundary, too)
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_wait();
   for (int i = threadIdx.x; i < top * F; i += blockDim.x)
     rows[i] = ids[(size_t)t * top + i / F] < 0 ? 0.0f : to_float(inner[(size_t)t * top * F + i]);
   __syncthreads();
+  static_assert(MOE_PER_WARP == 2, "a warp's two outputs are made side by side");
   const int c0 = (blockIdx.y * MOE_WARPS + warp) * MOE_PER_WARP;
-  for (int c = c0; c < min(C, c0 + MOE_PER_WARP); ++c) {
-    float total = 0.0f;
-    for (int k = 0; k < top; ++k) {
-      const int e = ids[(size_t)t * top + k];
-      if (e < 0) continue;
-      const T* w = w_down + ((size_t)e * C + c) * F;
-      const float* r = rows + k * F;
-      float s = 0.0f;
-      for (int f = lane; f < F; f += 32) s += r[f] * to_float(w[f]);
-      total += (weights ? weights[(size_t)t * top + k] : 1.0f) * warp_sum(s);
-    }
-    if (lane == 0) x[(size_t)t * C + c] += total;
+  if (c0 >= C) return;
+  float total[2] = {0.0f, 0.0f};
+  for (int k = 0; k < top; ++k) {
+    const int e = ids[(size_t)t * top + k];
+    if (e < 0) continue;
+    float s[2];
+    // (behind the last output the same row is read twice)
+    moe_dot<2>(rows + (size_t)k * F, w_down + ((size_t)e * C + c0) * F, c0 + 1 < C ? (size_t)F : 0, F, lane, wide, s);
+    const float wgt = weights ? weights[(size_t)t * top + k] : 1.0f;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) total[n] += wgt * warp_sum(s[n]);
   }
+  if (lane < 2 && c0 + lane < C) x[(size_t)t * C + c0 + lane] += lane == 0 ? total[0] : total[1];
 }
 
 constexpr int MOE_G_WARPS = 4, MOE_G_OUT = 32, MOE_G_ROWS = 4;

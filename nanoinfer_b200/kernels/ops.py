@@ -465,19 +465,22 @@ def _note_linear(a, norm, w, bias, out, M, residual) -> None:
 
 
 class NormInput:
-    """Activations given as the 32-bit residual stream plus the parameters of the LayerNorm that
-    stands before the product: ``linear`` normalises ``x[rows[m]]`` (or ``x[m]``) itself, inside the
-    tensor-core kernel where the step is small enough, else with the LayerNorm kernel into scratch
+    """Activations given as the 32-bit residual stream plus the parameters of the LayerNorm (``beta`` None:
+    of the RMS norm) that stands before the product: ``linear`` normalises ``x[rows[m]]`` (or ``x[m]``) itself, inside the
+    tensor-core kernel where the step is small enough, else with the norm's kernel into scratch
     taken from ``workspace``."""
 
-    def __init__(self, x: torch.Tensor, gamma: torch.Tensor, beta: torch.Tensor, eps: float, workspace,
+    def __init__(self, x: torch.Tensor, gamma: torch.Tensor, beta: Optional[torch.Tensor], eps: float, workspace,
                  dtype: torch.dtype, rows: Optional[torch.Tensor] = None, max_rows: int = 0):
         self.x, self.gamma, self.beta, self.eps = x, gamma, beta, float(eps)
         self.workspace, self.dtype, self.rows, self.max_rows = workspace, dtype, rows, max_rows
 
     def materialise(self, M: int) -> torch.Tensor:
         out = self.workspace.get("norm.fallback", (max(M, self.max_rows), self.x.shape[1]), self.dtype)
-        layernorm(self.x, self.gamma, self.beta, self.eps, out, M, self.rows)
+        if self.beta is None:
+            group_norm(self.x, self.gamma, 1, self.eps, out, M, self.rows)
+        else:
+            layernorm(self.x, self.gamma, self.beta, self.eps, out, M, self.rows)
         return out
 
 
@@ -617,7 +620,8 @@ def _linear_small(a, norm, w, bias, out, M, act, residual, kv=None) -> bool:
         # (rows wider than SKINNY_LN_REGISTER_WIDTH are normalised through a buffer per warp in shared memory, which
         # leaves room for one block an SM from 9 rows on: GPT-2 XL at batch 12 to 32 is 2 to 7 % faster with the
         # norm as a kernel of its own there)
-        if norm is not None and (M > SKINNY_LN_MAX_ROWS or (K > SKINNY_LN_REGISTER_WIDTH and M > 8)):
+        # (an RMS norm of its own is a few microseconds: wide rows take that at any M)
+        if norm is not None and (M > SKINNY_LN_MAX_ROWS or (K > SKINNY_LN_REGISTER_WIDTH and (M > 8 or norm.beta is None))):
             a, norm = norm.materialise(M), None
         if linear_skinny(a, norm, w, bias, out, M, act, residual, kv):
             return True
@@ -635,11 +639,11 @@ def _linear_small(a, norm, w, bias, out, M, act, residual, kv=None) -> bool:
 def linear(a: Optional[torch.Tensor], w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, M: int,
            act: int = ACT_NONE, residual: bool = False, norm: Optional[NormInput] = None) -> None:
     """The matrix product of the model: out[:M] = act(a[:M] . w^T + bias), added to the 32-bit
-    ``out`` with ``residual``.  With ``norm`` the activations are LayerNorm of the residual stream
+    ``out`` with ``residual``.  With ``norm`` the activations are a norm of the residual stream
     (``a`` is then None).  bfloat16 runs on the tensor cores where shape and alignment allow (rows
     of 16-byte multiples), else on the CUDA cores; float32 always runs on the CUDA cores in true
     32-bit arithmetic."""
-    if _linear_small(a, norm, w, bias, out, M, act, residual):
+    if w.dtype == torch.bfloat16 and _linear_small(a, norm, w, bias, out, M, act, residual):
         return
     if norm is not None:
         a = norm.materialise(M)   # (scratch: a second call for the same rows rewrites the same values)

@@ -54,10 +54,17 @@ def weight_bytes_per_step(model) -> int:
     return sum(t.numel() * t.element_size() for t, streamed in _unique_tensors(model).values() if streamed)
 
 
+def rows_seen(n: float, window: int, pool: int) -> float:
+    """Cached rows that a query seeing ``n`` positions reads: those of the window, and one a block of ``pool`` behind it."""
+    if not window:
+        return n
+    return min(n, window) + (max(0.0, n - window) // pool if pool else 0.0)
+
+
 def kv_bytes_per_position(cache) -> List[tuple]:
-    """(bytes per cached position over all layers of the group, window) for every cache group."""
+    """(bytes per cached position over all layers of the group, window, pool) for every cache group."""
     itemsize = torch.empty(0, dtype=cache.dtype).element_size()
-    return [(g.bytes_per_page(itemsize) // cache.page_size, g.spec.window) for g in cache.groups]
+    return [(g.bytes_per_page(itemsize) // cache.page_size, g.spec.window, g.spec.pool) for g in cache.groups]
 
 
 def kv_bytes(cache, contexts: Iterable[float]) -> float:
@@ -65,8 +72,8 @@ def kv_bytes(cache, contexts: Iterable[float]) -> float:
     total = 0.0
     groups = kv_bytes_per_position(cache)
     for n in contexts:
-        for per_pos, window in groups:
-            total += per_pos * (min(n, window) if window else n)
+        for per_pos, window, pool in groups:
+            total += per_pos * rows_seen(n, window, pool)
     return total
 
 
@@ -88,7 +95,7 @@ def step_flops(model, row_contexts: Sequence[int], n_logit_rows: int) -> float:
     for e in model.schedule:
         mixer = model.layers[e.layer].mixer
         if mixer is not None:
-            w = mixer.kv_spec().window if mixer.kv_spec() is not None else 0
-            k = float(sum(min(c, w) for c in row_contexts)) if w else keys
+            spec = mixer.kv_spec()
+            k = float(sum(rows_seen(c, spec.window, spec.pool) for c in row_contexts)) if spec is not None and spec.window else keys
             flops += mixer.flops_per_key() * k
     return flops

@@ -216,6 +216,8 @@ class TwoProducts:
     ``inner`` is what lies between: it reads the first product's result ``proj`` (float32 [rows, n_in], any row stride)
     and leaves the second's input in ``out`` ([rows, n_inner], the engine's dtype, any row stride)."""
 
+    #: (``run_alone`` hands a foldable norm to the first product)
+    takes_norm_input = True
     w_in: torch.Tensor
     b_in: Optional[torch.Tensor] = None
     w_out: torch.Tensor
@@ -268,13 +270,12 @@ class TwoProducts:
                   state: Optional[torch.Tensor] = None, writes_cache: bool = True, names=("in", "out")) -> None:
         from ..kernels import ops
 
-        if isinstance(xn, ops.NormInput):
-            xn = xn.materialise(ctx.n_rows)
+        xn, norm = (None, xn) if isinstance(xn, ops.NormInput) else (xn, None)
         T, ws = ctx.n_rows, ctx.workspace
         proj = ws.get("two_products.proj", (ctx.max_rows, self.n_in), torch.float32)
         out = ws.get("two_products.inner", (ctx.max_rows, self.n_inner), self.dtype)
         ops.trace_scope(ctx.layer, names[0])
-        ops.linear(xn, self.w_in, self.b_in, proj, T)
+        ops.linear(xn, self.w_in, self.b_in, proj, T, norm=norm)
         self.inner(proj, out, ctx, cache, state, writes_cache)
         ops.trace_scope(ctx.layer, names[1])
         ops.linear(out, self.w_out, self.b_out, x, T, residual=True)

@@ -105,6 +105,17 @@ class GroupedRMSNorm(Norm):
             self.params["weight"] = self.params["weight"] + 1.0
             self._shifted = True
 
+    def reserve(self, workspace, limits) -> None:
+        if self.groups == 1:      # (what ``as_input`` falls back to)
+            workspace.reserve("norm.fallback", limits.max_rows * self.width, limits.dtype)
+
+    def as_input(self, x: torch.Tensor, ctx, dtype: torch.dtype, rows: Optional[torch.Tensor] = None):
+        """One group: this norm in the form a matrix product can take as its activations."""
+        if self.groups != 1:
+            return None
+        return ops.NormInput(x, self.params["weight"], None, self.eps, ctx.workspace, dtype, rows=rows,
+                             max_rows=0 if rows is not None else ctx.max_rows)
+
     def forward(self, x: torch.Tensor, out: torch.Tensor, n_rows: int, rows: Optional[torch.Tensor] = None,
                 add: Optional[torch.Tensor] = None, add_rows: Optional[torch.Tensor] = None) -> None:
         ops.group_norm(x, self.params["weight"], self.groups, self.eps, out, n_rows, rows, add, add_rows)

@@ -260,7 +260,7 @@ def run_serving(model_dir: str, dtype: str = "bfloat16", requests: int = 128, ma
     run_continuous(eng, reqs[:min(len(reqs), 4)], **sampling)   # warm up: kernels built, first graphs captured
     peaks = measured_peaks()
     weights = weight_bytes_per_step(eng.model)
-    page_bytes = sum(per_pos for per_pos, _ in kv_bytes_per_position(eng.cache)) * page
+    page_bytes = sum(per_pos for per_pos, _, _ in kv_bytes_per_position(eng.cache)) * page
     out = []
     for name in policies:
         o = (run_static if name == "static" else run_continuous)(eng, reqs, **sampling)

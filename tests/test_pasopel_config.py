@@ -200,6 +200,17 @@ def test_truncation_gives_pooled_pages_back():
     m.check()
 
 
+def test_bytes_and_operations_count_the_window_and_the_blocks_behind_it():
+    from nanoinfer_b200 import measure
+
+    assert [measure.rows_seen(n, 10, 4) for n in (3, 10, 13, 14, 18, 19)] == [3, 10, 10, 11, 12, 12]
+    assert measure.rows_seen(50, 0, 0) == 50 and measure.rows_seen(50, 20, 0) == 20
+    m = _manager(10, 4, max_tokens=64)
+    m.dtype = torch.float32
+    per = 2 * 2 * 16 * 4
+    assert measure.kv_bytes(m, [18]) == per * 12 + 2 * 32 * 4 * 18
+
+
 @pytest.mark.parametrize("seed", range(4))
 def test_scheduler_over_pooled_rows_and_a_small_pool(seed):
     """Requests through a pool too small for all of them: portions are cut to the pages that are left, nothing starves, and

@@ -298,6 +298,29 @@ def test_routing_by_biased_logits(E, top, C, dtype):
     assert float((weights.double() - torch.softmax(best.values, 1)).abs().max()) < 1e-5
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("M", [1, 8, 9, 16, 40, 130])
+@pytest.mark.parametrize("N,K", [(96, 48), (200, 768), (64, 1600), (33, 100)])
+def test_product_of_an_rms_norm_of_the_stream(N, K, M, dtype):
+    """The norm folded into the product of few rows (no shift, nothing taken off), or run ahead of it; rows picked."""
+    from nanoinfer_b200.kernels import ops
+    from nanoinfer_b200.parts.base import Workspace
+
+    torch.manual_seed(N + M)
+    dt, eps = DT[dtype], 1e-4
+    x, g = torch.randn(M + 5, K, device=DEV) + 0.7, torch.rand(K, device=DEV) + 0.5
+    w, b = (torch.randn(N, K, device=DEV) / K ** 0.5).to(dt), torch.randn(N, device=DEV)
+    rows = torch.randperm(M + 5, device=DEV)[:M].to(torch.int32)
+    for r in (None, rows):
+        norm = ops.NormInput(x, g, None, eps, Workspace(torch.device(DEV)), dt, rows=r)
+        out = torch.full((M, N), 7.0, device=DEV)
+        ops.linear(None, w, b, out, M, norm=norm)
+        xr = (x[:M] if r is None else x[r.long()]).double()
+        y = (xr / torch.sqrt((xr ** 2).mean(-1, keepdim=True) + eps) * g.double()).to(dt).double()
+        want = y @ w.double().T + b.double()
+        assert float((out.double() - want).abs().max()) < (1e-5 if dtype == "float32" else 3e-2)
+
+
 @pytest.mark.parametrize("M", [17, 128, 130, 700])
 @pytest.mark.parametrize("S,N,F", [(3, 64, 64), (8, 768, 128), (5, 72, 192), (16, 200, 64), (2, 1600, 1600), (1, 48, 320)])
 def test_one_product_over_stacked_matrices(S, N, F, M):
